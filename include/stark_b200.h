@@ -419,6 +419,11 @@ stark_b200_status stark_b200_cancel(stark_b200_model *model);
 /* Feeds token_ids; logits of the last row are available afterwards (asynchronous until a read-out
  * or drain).  hybrid::Model::ingest_prefix + step (mod.rs:897-1018). */
 stark_b200_status stark_b200_prefill(stark_b200_model *model, const uint32_t *token_ids, size_t count);
+/* The same for a portion of a prompt, with the logits of chosen rows of it: `wanted` are ascending indices into
+ * token_ids, dst receives [wanted_count, vocab] f32 on the host.  Every family serves it; a family without a several-rows
+ * read-out cuts the portion behind each wanted row.  UNSUPPORTED with a draft head. */
+stark_b200_status stark_b200_prefill_rows(stark_b200_model *model, const uint32_t *token_ids, size_t count,
+                                          const uint32_t *wanted, size_t wanted_count, float *dst);
 stark_b200_status stark_b200_step(stark_b200_model *model, uint32_t token_id);
 /* Full-vocabulary logits of the last row, f32 (stark_glm_readout_f32). */
 stark_b200_status stark_b200_readout_f32(stark_b200_model *model, float *dst, size_t count);

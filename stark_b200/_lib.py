@@ -166,6 +166,7 @@ def load() -> C.CDLL:
         "stark_b200_drain": (u32, [vp]),
         "stark_b200_cancel": (u32, [vp]),
         "stark_b200_prefill": (u32, [vp, vp, sz]),
+        "stark_b200_prefill_rows": (u32, [vp, vp, sz, vp, sz, vp]),
         "stark_b200_step": (u32, [vp, u32]),
         "stark_b200_readout_f32": (u32, [vp, vp, sz]),
         "stark_b200_readout_bf16": (u32, [vp, vp, sz]),

@@ -1,9 +1,5 @@
-// Dense Qwen3-shaped decode engine: one recorded launch sequence (CUDA graph with programmatic
-// dependent launch between its kernels) per token, replayed with the position and token read from
-// device memory.  Mirrors the reference's decode pass
-//   crates/stark-engine/src/engine/language_model/stream/stream.rs:787-1217 (one submission per token,
-//   on-device token chaining) and its layer wiring
-//   crates/stark-engine/src/encodable_block/transformer_layer.rs:549-659.
+// Dense Qwen3-shaped decoder: what one token launches, its tensors, and its hooks into the shared token loop
+// (token_loop.cu).  Layer wiring: crates/stark-engine/src/encodable_block/transformer_layer.rs:549-659.
 //
 // Per layer the sequence is five kernels:
 //   qkv    = W_qkv  rmsnorm(h)                      matvec, norm fused in the prologue
@@ -26,13 +22,6 @@ namespace sb {
 
 namespace {
 
-template <typename T>
-stark_b200_status dmalloc(T **p, size_t count) {
-    *p = nullptr;
-    SB_CUDA(cudaMalloc(p, count * sizeof(T) ? count * sizeof(T) : 1));
-    return STARK_B200_OK;
-}
-
 // Size of the token id space: the embedding table's rows (under tensor parallelism cfg.vocab is the
 // read-out shard of this rank).
 uint32_t input_vocab(const Model *m) { return m->tp.size > 1u ? m->tp_vocab_total : m->cfg.vocab; }
@@ -48,80 +37,6 @@ uint32_t default_attn_splits(uint32_t kv_heads) {
 
 }  // namespace
 
-Model::~Model() {
-    if (step_graph) cudaGraphExecDestroy(step_graph);
-    if (ingest_graph) cudaGraphExecDestroy(ingest_graph);
-    for (auto &L : layers) {
-        qmatrix_free(L.qkv);
-        qmatrix_free(L.o);
-        qmatrix_free(L.upgate);
-        qmatrix_free(L.down);
-        qmatrix_free(L.o_rows);
-        qmatrix_free(L.down_rows);
-        cudaFree(L.attn_norm);
-        cudaFree(L.mlp_norm);
-        cudaFree(L.attn_norm_b16);
-        cudaFree(L.mlp_norm_b16);
-        cudaFree(L.q_norm);
-        cudaFree(L.k_norm);
-        cudaFree(L.kv.keys);
-        cudaFree(L.kv.values);
-    }
-    mtp_destroy(this);
-    if (lm_head != embed) qmatrix_free(lm_head);
-    qmatrix_free(embed);
-    cudaFree(final_norm);
-    cudaFree(final_norm_b16);
-    cudaFree(block_table);
-    cudaFree(rope_cos);
-    cudaFree(rope_sin);
-    cudaFree(state);
-    cudaFree(pending);
-    cudaFree(generated);
-    cudaFree(trace);
-    cudaFree(tp_staged);
-    cudaFree(mega_ops);
-    cudaFree(mega_ingest_ops);
-    cudaFree(mega_done);
-    cudaFree(mega_scratch);
-    cudaFree(h);
-    cudaFree(h_alt);
-    cudaFree(qkv);
-    cudaFree(attn);
-    cudaFree(act);
-    cudaFree(logits);
-    cudaFree(attn_scratch);
-    cudaFree(attn_counters);
-    cudaFree(partial_max);
-    cudaFree(partial_index);
-    if (tp_connected)
-        for (uint32_t r = 0; r < tp.size; ++r)
-            if (r != tp.rank && tp.base[r]) {
-                if (tp_stand_ins) cudaFree(tp.base[r]);
-                else cudaIpcCloseMemHandle(tp.base[r]);
-            }
-    if (tp_rows_connected)
-        for (uint32_t r = 0; r < tp_rows.size; ++r)
-            if (r != tp_rows.rank && tp_rows.base[r]) cudaIpcCloseMemHandle(tp_rows.base[r]);
-    cudaFree(chunk_tokens);
-    if (!tp_rows_local) {  // under tensor parallelism these two live inside the rows region
-        cudaFree(chunk_h);
-        cudaFree(chunk_act);
-    }
-    cudaFree(chunk_x);
-    cudaFree(chunk_qkv);
-    cudaFree(chunk_attn);
-    cudaFree(tp_rows_local);
-    cudaFree(tp_rows_arrive);
-    cudaFree(rows_attn_partials);
-    cudaFree(tp_local);
-    cudaFree(sample_scratch);
-    cudaFree(tp_seq);
-    if (host_state) cudaFreeHost(host_state);
-    if (host_logits) cudaFreeHost(host_logits);
-    if (stream) cudaStreamDestroy(stream);
-}
-
 stark_b200_status model_create(const stark_b200_dense_config &c, Model **out) {
     *out = nullptr;
     if (c.layers == 0 || c.hidden == 0 || c.hidden % 64u != 0 || c.head_dim != kHeadDim || c.kv_heads == 0 ||
@@ -135,17 +50,15 @@ stark_b200_status model_create(const stark_b200_dense_config &c, Model **out) {
         delete m;
         return STARK_B200_INVALID_ARGUMENT;
     }
-    cudaGetDevice(&m->device);
     m->layers.resize(c.layers + c.reserved);  // the draft head's layer (with its own cache) comes last
     stark_b200_status st = STARK_B200_OK;
     auto fail = [&](stark_b200_status s) {
         delete m;
         return s;
     };
-    if (cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking) != cudaSuccess) return fail(STARK_B200_DEVICE_FAILURE);
+    m->family = &kDenseFamily;
+    if ((st = model_create_session(m, false)) != STARK_B200_OK) return fail(st);
 
-    // KV pages: identity block table sized for the context (rounded up to whole pages).
-    m->num_blocks = (c.context_tokens + kPageTokens - 1u) / kPageTokens;
     const size_t page_elems = (size_t)c.kv_heads * kPageTokens * kHeadDim;
     for (auto &L : m->layers) {
         if ((st = dmalloc(&L.kv.keys, m->num_blocks * page_elems)) != STARK_B200_OK) return fail(st);
@@ -154,12 +67,6 @@ stark_b200_status model_create(const stark_b200_dense_config &c, Model **out) {
             cudaMemset(L.kv.values, 0, m->num_blocks * page_elems * 2) != cudaSuccess)
             return fail(STARK_B200_DEVICE_FAILURE);
     }
-    std::vector<int32_t> table(m->num_blocks);
-    for (uint32_t i = 0; i < m->num_blocks; ++i) table[i] = (int32_t)i;
-    if ((st = dmalloc(&m->block_table, m->num_blocks)) != STARK_B200_OK) return fail(st);
-    if (cudaMemcpy(m->block_table, table.data(), table.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess)
-        return fail(STARK_B200_DEVICE_FAILURE);
-
     // RoPE tables on the host with the reference's formulas and operation order
     // (crates/stark-engine/src/encodable_block/mixer/attention/rope.rs:346-440, UnscaledRoPEConfig).
     {
@@ -190,33 +97,22 @@ stark_b200_status model_create(const stark_b200_dense_config &c, Model **out) {
     // splits than that start cold.
     m->attn_splits = default_attn_splits(c.kv_heads);
     if (tunables().attn_splits) m->attn_splits = tunables().attn_splits;  // tuning: CTAs per KV head
-    if ((st = dmalloc(&m->state, 1)) != STARK_B200_OK) return fail(st);
-    if ((st = dmalloc(&m->pending, (size_t)c.context_tokens + 1u)) != STARK_B200_OK) return fail(st);
-    if ((st = dmalloc(&m->generated, (size_t)c.context_tokens + 1u)) != STARK_B200_OK) return fail(st);
     if ((st = dmalloc(&m->h, c.hidden)) != STARK_B200_OK) return fail(st);
     if ((st = dmalloc(&m->h_alt, c.hidden)) != STARK_B200_OK) return fail(st);
     if ((st = dmalloc(&m->qkv, qkv_n)) != STARK_B200_OK) return fail(st);
     if ((st = dmalloc(&m->attn, c.q_heads * kHeadDim)) != STARK_B200_OK) return fail(st);
     if ((st = dmalloc(&m->act, c.inter)) != STARK_B200_OK) return fail(st);
-    if ((st = dmalloc(&m->logits, c.vocab)) != STARK_B200_OK) return fail(st);
     if ((st = dmalloc(&m->attn_scratch, attention_scratch_floats(c.q_heads, c.kv_heads, kMaxAttnSplits))) !=
         STARK_B200_OK)
         return fail(st);
     if ((st = dmalloc(&m->attn_counters, c.kv_heads)) != STARK_B200_OK) return fail(st);
-    if ((st = dmalloc(&m->partial_max, 1024)) != STARK_B200_OK) return fail(st);
-    if ((st = dmalloc(&m->partial_index, 1024)) != STARK_B200_OK) return fail(st);
     if (const char *e = getenv("STARK_B200_TRACE")) {
         if (e[0] == '1') {  // one slot per launch
             m->trace_slots = 1u + 7u * c.layers + 3u;  // up to 7 launches per layer with tensor-parallel reductions
             if ((st = dmalloc(&m->trace, m->trace_slots)) != STARK_B200_OK) return fail(st);
         }
     }
-    if (cudaMemset(m->attn_counters, 0, c.kv_heads * 4) != cudaSuccess ||
-        cudaMemset(m->state, 0, sizeof(StepState)) != cudaSuccess)
-        return fail(STARK_B200_DEVICE_FAILURE);
-    if (cudaMallocHost(&m->host_state, sizeof(StepState)) != cudaSuccess ||
-        cudaMallocHost(&m->host_logits, (size_t)c.vocab * 2u) != cudaSuccess)
-        return fail(STARK_B200_OUT_OF_MEMORY);
+    if (cudaMemset(m->attn_counters, 0, c.kv_heads * 4) != cudaSuccess) return fail(STARK_B200_DEVICE_FAILURE);
     if (c.reserved == 1u && (st = mtp_create(m)) != STARK_B200_OK) return fail(st);
     *out = m;
     return STARK_B200_OK;
@@ -612,31 +508,6 @@ static stark_b200_status build_mega(Model *m) {
     return STARK_B200_OK;
 }
 
-// One token on the model's stream: the recorded launch sequence, or the persistent kernel.
-static stark_b200_status launch_token(Model *m, bool full) {
-    if (m->use_mega) {
-        SB_CUDA(cudaMemsetAsync(m->mega_done, 0, (m->mega_num_ops + 1u) * sizeof(unsigned long long), m->stream));
-        return mega_launch(full ? m->mega_full : m->mega_ingest, m->mega_grid, m->mega_smem, m->stream);
-    }
-    SB_CUDA(cudaGraphLaunch(full ? m->step_graph : m->ingest_graph, m->stream));
-    return STARK_B200_OK;
-}
-
-static stark_b200_status capture(Model *m, bool full, cudaGraphExec_t *exec, uint32_t *launches) {
-    SB_CUDA(cudaStreamBeginCapture(m->stream, cudaStreamCaptureModeThreadLocal));
-    stark_b200_status st = issue_token(m, full, launches);
-    cudaGraph_t g = nullptr;
-    cudaError_t e = cudaStreamEndCapture(m->stream, &g);
-    if (st != STARK_B200_OK) {
-        if (g) cudaGraphDestroy(g);
-        return st;
-    }
-    if (e != cudaSuccess) return cuda_status(e);
-    e = cudaGraphInstantiate(exec, g, 0);
-    cudaGraphDestroy(g);
-    return cuda_status(e);
-}
-
 stark_b200_status model_tp_init(Model *m, uint32_t rank, uint32_t size, uint32_t vocab_offset, uint32_t vocab_total,
                                 uint8_t *handle_out) {
     static_assert(sizeof(cudaIpcMemHandle_t) == 64, "handle size is part of the interface");
@@ -742,29 +613,31 @@ stark_b200_status model_tp_connect_unanswered(Model *m) {
     return STARK_B200_OK;
 }
 
-stark_b200_status model_finalize(Model *m) {
-    if (m->finalized) return STARK_B200_INVALID_STATE;
+// ---- what the shared token loop asks of the dense family
+
+static stark_b200_status dense_ready(Model *m) {
     if (!m->embed || !m->lm_head || !m->final_norm) return STARK_B200_INVALID_STATE;
     if (m->tp.size > 1u && !m->tp_connected) return STARK_B200_INVALID_STATE;
     for (auto &L : m->layers)
         if (!L.qkv || !L.o || !L.upgate || !L.down || !L.attn_norm || !L.mlp_norm || !L.q_norm || !L.k_norm)
             return STARK_B200_INVALID_STATE;
-    // One eager pass first (function attributes and lazily created library state must exist before
-    // a recording), on a scratch position; then record both sequences.
-    stark_b200_status st = model_reset(m);
-    if (st != STARK_B200_OK) return st;
-    // Tensor parallel: this first pass is where every rank's kernels are loaded, and on a machine that has not run
-    // the library yet one rank can take seconds longer over that than another.  That is start-up skew, not a peer
-    // that left: the first pass waits a minute for its peers; the recorded sequences keep the configured limit.
+    return STARK_B200_OK;
+}
+
+// Tensor parallel: this first pass is where every rank's kernels are loaded, and on a machine that has not run
+// the library yet one rank can take seconds longer over that than another.  That is start-up skew, not a peer
+// that left: the first pass waits a minute for its peers; the recorded sequences keep the configured limit.
+static stark_b200_status dense_first_pass(Model *m) {
     const unsigned long long configured_wait = m->tp.wait_ns;
     if (m->tp.size > 1u && !m->tp_stand_ins) m->tp.wait_ns = std::max<unsigned long long>(configured_wait, 60000000000ull);
-    st = issue_token(m, true, nullptr);
+    stark_b200_status st = issue_token(m, true, nullptr);
     if (st == STARK_B200_OK) st = issue_token(m, false, nullptr);
     m->tp.wait_ns = configured_wait;
-    if (st != STARK_B200_OK) return st;
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    if ((st = capture(m, true, &m->step_graph, &m->step_launches)) != STARK_B200_OK) return st;
-    if ((st = capture(m, false, &m->ingest_graph, &m->ingest_launches)) != STARK_B200_OK) return st;
+    return st;
+}
+
+static stark_b200_status dense_recorded(Model *m) {
+    stark_b200_status st;
     if (const char *e = getenv("STARK_B200_MEGA")) m->use_mega = e[0] == '1' && m->tp.size <= 1u;
     if (m->use_mega) {
         if (m->trace) {  // one slot per operator instead of one per launch
@@ -777,240 +650,133 @@ stark_b200_status model_finalize(Model *m) {
         m->step_launches = 1;
         m->ingest_launches = 1;
     }
-    if ((st = mtp_finalize(m)) != STARK_B200_OK) return st;
-    m->finalized = true;
-    return model_reset(m);
+    return mtp_finalize(m);
 }
 
-// Records both launch sequences again with the current launch-shape settings.  Cache and position are kept.
-stark_b200_status model_recapture(Model *m) {
-    if (!m->finalized || m->fenced) return STARK_B200_INVALID_STATE;
-    if (m->use_mega) return STARK_B200_UNSUPPORTED;
-    SB_CUDA(cudaStreamSynchronize(m->stream));
+static stark_b200_status dense_launch_persistent(Model *m, bool full) {
+    SB_CUDA(cudaMemsetAsync(m->mega_done, 0, (m->mega_num_ops + 1u) * sizeof(unsigned long long), m->stream));
+    return mega_launch(full ? m->mega_full : m->mega_ingest, m->mega_grid, m->mega_smem, m->stream);
+}
+
+static void dense_retune(Model *m) {
     m->attn_splits = tunables().attn_splits ? tunables().attn_splits : default_attn_splits(m->cfg.kv_heads);
-    // one eager pass on a scratch copy of the step state (first use of a kernel instance sets its attributes)
-    StepState saved;
-    SB_CUDA(cudaMemcpy(&saved, m->state, sizeof(StepState), cudaMemcpyDeviceToHost));
-    stark_b200_status st;
-    if ((st = issue_token(m, true, nullptr)) != STARK_B200_OK) return st;
-    if ((st = issue_token(m, false, nullptr)) != STARK_B200_OK) return st;
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    SB_CUDA(cudaMemcpy(m->state, &saved, sizeof(StepState), cudaMemcpyHostToDevice));
-    cudaGraphExec_t step = nullptr, ingest = nullptr;
-    uint32_t step_n = 0, ingest_n = 0;
-    if ((st = capture(m, true, &step, &step_n)) != STARK_B200_OK) return st;
-    if ((st = capture(m, false, &ingest, &ingest_n)) != STARK_B200_OK) {
-        cudaGraphExecDestroy(step);
-        return st;
-    }
-    cudaGraphExecDestroy(m->step_graph);
-    cudaGraphExecDestroy(m->ingest_graph);
-    m->step_graph = step;
-    m->ingest_graph = ingest;
-    m->step_launches = step_n;
-    m->ingest_launches = ingest_n;
-    m->has_logits = false;
-    return STARK_B200_OK;
 }
 
-stark_b200_status model_reset(Model *m) {
-    SB_CUDA(cudaMemsetAsync(m->state, 0, sizeof(StepState), m->stream));
+static stark_b200_status dense_reset(Model *m) {
     SB_CUDA(cudaMemsetAsync(m->attn_counters, 0, m->cfg.kv_heads * 4, m->stream));
     if (m->mega_done)
         SB_CUDA(cudaMemsetAsync(m->mega_done, 0, (m->mega_num_ops + 1u) * sizeof(unsigned long long), m->stream));
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    m->position = 0;
-    m->has_logits = false;
     return mtp_reset(m);
 }
 
-stark_b200_status model_rewind(Model *m, uint64_t position) {
-    if (position > m->position) return STARK_B200_INVALID_ARGUMENT;
+static stark_b200_status dense_rewind(Model *m, uint64_t position) {
     // the draft head's cache would need the hidden row before the cut, which is not kept
     if (m->mtp.enabled && position != 0) return STARK_B200_UNSUPPORTED;
-    if (m->mtp.enabled) mtp_reset(m);
-    const uint32_t pos = (uint32_t)position;
-    SB_CUDA(cudaMemcpyAsync(&m->state->position, &pos, 4, cudaMemcpyHostToDevice, m->stream));
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    m->position = position;
-    m->has_logits = false;
-    return STARK_B200_OK;
+    return m->mtp.enabled ? mtp_reset(m) : STARK_B200_OK;
 }
 
-// Feeds `count` tokens; the last one runs the full sequence so that logits and the greedy token
-// are available afterwards (hybrid::Model: ingest all but the last, then step the last;
-// crates/stark-score/src/scoring.rs:453-489).
-stark_b200_status model_prefill(Model *m, const uint32_t *ids, size_t count) {
-    if (!m->finalized || m->fenced || m->mtp.open_rows) return STARK_B200_INVALID_STATE;
-    if (count == 0) return STARK_B200_INVALID_ARGUMENT;
-    if (m->position + count > m->cfg.context_tokens) return STARK_B200_CONTEXT_LIMIT;
-    for (size_t i = 0; i < count; ++i)
-        if (ids[i] >= input_vocab(m)) return STARK_B200_INVALID_ARGUMENT;
-    // All rows but the last only fill the cache: enough of them go through the batched path (tensor-core
-    // contraction over whole chunks), after which the last row is an ordinary token at its position.
-    const bool batched = tunables().prefill_batch && model_batched_prefill_ready(m);
-    if (m->mtp.enabled && (!batched || (m->position > 0 && !m->mtp.has_pending))) return STARK_B200_UNSUPPORTED;
-    if (batched && (m->mtp.enabled || count - 1 >= tunables().prefill_min_rows)) {
-        if (m->mtp.enabled && m->position > 0) {
-            // a continued prompt: the pair (first new token, hidden of the last row so far) enters the head's cache
-            SB_CUDA(cudaMemcpyAsync(m->chunk_tokens, ids, 4, cudaMemcpyHostToDevice, m->stream));
-            stark_b200_status ps = mtp_prime_continue(m);
-            if (ps != STARK_B200_OK) return ps;
-        }
-        stark_b200_status bs = model_prefill_batched(m, ids, count - 1, count);
-        if (bs == STARK_B200_CANCELLED) {
-            m->cancel_requested = false;
-            cudaStreamSynchronize(m->stream);
-            model_reset(m);
-            return bs;
-        }
-        if (bs != STARK_B200_OK) return bs;
-        StepState last{};
-        last.position = (uint32_t)(m->position + count - 1);
-        last.token = ids[count - 1];
-        SB_CUDA(cudaMemcpyAsync(m->state, &last, sizeof(last), cudaMemcpyHostToDevice, m->stream));
-        stark_b200_status ls = launch_token(m, true);
-        if (ls != STARK_B200_OK) return ls;
-        m->position += count;
-        m->has_logits = true;
-        m->launches_issued += m->step_launches;
-        return mtp_after_prompt(m);
-    }
-    // pending[0 .. count-2] = ids[1 ..]; the ingest-advance kernel pops one per row
-    if (count > 1) SB_CUDA(cudaMemcpyAsync(m->pending, ids + 1, (count - 1) * 4, cudaMemcpyHostToDevice, m->stream));
-    StepState hs{};
-    hs.position = (uint32_t)m->position;
-    hs.token = ids[0];
-    hs.next_token = 0;
-    hs.cursor = 0;
-    SB_CUDA(cudaMemcpyAsync(m->state, &hs, sizeof(hs), cudaMemcpyHostToDevice, m->stream));
-    for (size_t i = 0; i + 1 < count; ++i) {
-        if (m->cancel_requested) {
-            m->cancel_requested = false;
-            cudaStreamSynchronize(m->stream);
-            m->fenced = false;
-            model_reset(m);
-            return STARK_B200_CANCELLED;
-        }
-        stark_b200_status ls = launch_token(m, false);
-        if (ls != STARK_B200_OK) return ls;
-    }
-    {
-        stark_b200_status ls = launch_token(m, true);
-        if (ls != STARK_B200_OK) return ls;
-    }
-    m->position += count;
-    m->has_logits = true;
-    m->launches_issued += (count - 1) * m->ingest_launches + m->step_launches;
-    return STARK_B200_OK;
+static stark_b200_status dense_prompt_begin(Model *m, const uint32_t *ids) {
+    if (!m->mtp.enabled || m->position == 0) return STARK_B200_OK;
+    // a continued prompt: the pair (first new token, hidden of the last row so far) enters the head's cache
+    SB_CUDA(cudaMemcpyAsync(m->chunk_tokens, ids, 4, cudaMemcpyHostToDevice, m->stream));
+    return mtp_prime_continue(m);
 }
 
-stark_b200_status model_step(Model *m, uint32_t token, bool chained) {
-    if (!m->finalized || m->fenced || m->mtp.open_rows) return STARK_B200_INVALID_STATE;
-    if (m->position + 1 > m->cfg.context_tokens) return STARK_B200_CONTEXT_LIMIT;
-    if (!chained) {
-        if (token >= input_vocab(m)) return STARK_B200_INVALID_ARGUMENT;
-        SB_CUDA(cudaMemcpyAsync(&m->state->token, &token, 4, cudaMemcpyHostToDevice, m->stream));
+static stark_b200_status dense_rows_done(Model *m, uint32_t mrows, uint32_t pairs, uint32_t first_pos) {
+    return m->mtp.enabled ? mtp_prime_rows(m, mrows, pairs, first_pos) : STARK_B200_OK;
+}
+
+static void dense_sizes(const Model *m, uint64_t *weight_bytes, uint64_t *kv_bytes_per_token) {
+    uint64_t wb = 0;
+    for (auto &L : m->layers)
+        for (QMatrix *q : {L.qkv, L.o, L.upgate, L.down})
+            if (q) wb += q->bytes;
+    if (m->embed) wb += m->embed->bytes;
+    if (m->lm_head && m->lm_head != m->embed) wb += m->lm_head->bytes;
+    *weight_bytes = wb;
+    *kv_bytes_per_token = (uint64_t)m->cfg.layers * 2u * m->cfg.kv_heads * kHeadDim * 2u;
+}
+
+static void dense_destroy(Model *m) {
+    for (auto &L : m->layers) {
+        qmatrix_free(L.qkv);
+        qmatrix_free(L.o);
+        qmatrix_free(L.upgate);
+        qmatrix_free(L.down);
+        qmatrix_free(L.o_rows);
+        qmatrix_free(L.down_rows);
+        cudaFree(L.attn_norm);
+        cudaFree(L.mlp_norm);
+        cudaFree(L.attn_norm_b16);
+        cudaFree(L.mlp_norm_b16);
+        cudaFree(L.q_norm);
+        cudaFree(L.k_norm);
+        cudaFree(L.kv.keys);
+        cudaFree(L.kv.values);
     }
-    {
-        stark_b200_status ls = launch_token(m, true);
-        if (ls != STARK_B200_OK) return ls;
+    mtp_destroy(m);
+    if (m->lm_head != m->embed) qmatrix_free(m->lm_head);
+    qmatrix_free(m->embed);
+    cudaFree(m->final_norm);
+    cudaFree(m->final_norm_b16);
+    cudaFree(m->rope_cos);
+    cudaFree(m->rope_sin);
+    cudaFree(m->tp_staged);
+    cudaFree(m->mega_ops);
+    cudaFree(m->mega_ingest_ops);
+    cudaFree(m->mega_done);
+    cudaFree(m->mega_scratch);
+    cudaFree(m->h);
+    cudaFree(m->h_alt);
+    cudaFree(m->qkv);
+    cudaFree(m->attn);
+    cudaFree(m->act);
+    cudaFree(m->attn_scratch);
+    cudaFree(m->attn_counters);
+    if (m->tp_connected)
+        for (uint32_t r = 0; r < m->tp.size; ++r)
+            if (r != m->tp.rank && m->tp.base[r]) {
+                if (m->tp_stand_ins) cudaFree(m->tp.base[r]);
+                else cudaIpcCloseMemHandle(m->tp.base[r]);
+            }
+    if (m->tp_rows_connected)
+        for (uint32_t r = 0; r < m->tp_rows.size; ++r)
+            if (r != m->tp_rows.rank && m->tp_rows.base[r]) cudaIpcCloseMemHandle(m->tp_rows.base[r]);
+    if (!m->tp_rows_local) {  // under tensor parallelism these two live inside the rows region
+        cudaFree(m->chunk_h);
+        cudaFree(m->chunk_act);
     }
-    m->position += 1;
-    m->has_logits = true;
-    m->launches_issued += m->step_launches;
-    return STARK_B200_OK;
+    cudaFree(m->chunk_x);
+    cudaFree(m->chunk_qkv);
+    cudaFree(m->chunk_attn);
+    cudaFree(m->tp_rows_local);
+    cudaFree(m->tp_rows_arrive);
+    cudaFree(m->rows_attn_partials);
+    cudaFree(m->tp_local);
+    cudaFree(m->tp_seq);
 }
 
-static stark_b200_status check_device_error(Model *m) {
-    DeviceContext *ctx = device_context();
-    if (!ctx) return STARK_B200_DEVICE_FAILURE;
-    uint32_t word = 0;
-    SB_CUDA(cudaMemcpyAsync(&word, ctx->error_word, 4, cudaMemcpyDeviceToHost, m->stream));
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    if (word) {
-        m->fenced = true;
-        return STARK_B200_DEVICE_FAILURE;
-    }
-    return STARK_B200_OK;
+static ModelFamily make_dense_family() {
+    ModelFamily f{};
+    f.name = "dense";
+    f.input_vocab = input_vocab;
+    f.ready = dense_ready;
+    f.issue_token = issue_token;
+    f.first_pass = dense_first_pass;
+    f.recorded = dense_recorded;
+    f.launch_token = dense_launch_persistent;
+    f.retune = dense_retune;
+    f.rows_ready = model_batched_prefill_ready;
+    f.rows_pass = model_rows_pass;
+    f.prompt_begin = dense_prompt_begin;
+    f.rows_done = dense_rows_done;
+    f.prompt_end = mtp_after_prompt;
+    f.reset = dense_reset;
+    f.rewind = dense_rewind;
+    f.sizes = dense_sizes;
+    f.destroy = dense_destroy;
+    return f;
 }
-
-stark_b200_status model_drain(Model *m) {
-    cudaError_t e = cudaStreamSynchronize(m->stream);
-    if (e != cudaSuccess) {
-        m->fenced = true;
-        return cuda_status(e);
-    }
-    return check_device_error(m);
-}
-
-stark_b200_status model_next_token(Model *m, uint32_t *out) {
-    if (!m->has_logits) return STARK_B200_INVALID_STATE;
-    SB_CUDA(cudaMemcpyAsync(m->host_state, m->state, sizeof(StepState), cudaMemcpyDeviceToHost, m->stream));
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    *out = m->host_state->next_token;
-    return STARK_B200_OK;
-}
-
-stark_b200_status model_readout_bf16(Model *m, uint16_t *dst, size_t count) {
-    if (!m->has_logits) return STARK_B200_INVALID_STATE;
-    if (count != m->cfg.vocab) return STARK_B200_INVALID_ARGUMENT;
-    SB_CUDA(cudaMemcpyAsync(m->host_logits, m->logits, count * 2, cudaMemcpyDeviceToHost, m->stream));
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    memcpy(dst, m->host_logits, count * 2);
-    return STARK_B200_OK;
-}
-
-stark_b200_status model_readout_f32(Model *m, float *dst, size_t count) {
-    if (!m->has_logits) return STARK_B200_INVALID_STATE;
-    if (count != m->cfg.vocab) return STARK_B200_INVALID_ARGUMENT;
-    SB_CUDA(cudaMemcpyAsync(m->host_logits, m->logits, count * 2, cudaMemcpyDeviceToHost, m->stream));
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    for (size_t i = 0; i < count; ++i) dst[i] = bf16_bits_to_f32(m->host_logits[i]);
-    return STARK_B200_OK;
-}
-
-// Greedy decode of `steps` tokens chained on the device: the step sequence writes its own next
-// input.  Token ids come back through one small device-to-host copy per step, all asynchronous;
-// the host synchronises once at the end.
-stark_b200_status model_generate_greedy(Model *m, uint32_t steps, uint32_t *out_tokens) {
-    if (!m->finalized || m->fenced || !m->has_logits) return STARK_B200_INVALID_STATE;
-    if (m->position + steps > m->cfg.context_tokens) return STARK_B200_CONTEXT_LIMIT;
-    uint32_t *pinned = nullptr;
-    SB_CUDA(cudaMallocHost(&pinned, (size_t)(steps + 1u) * 4u));
-    // out[0] is the token sampled from the logits already present (the prompt's last row); the
-    // rest are appended to the device-side list by each step and fetched in one copy at the end.
-    const uint32_t window[2] = {0u, steps};
-    cudaError_t e = cudaMemcpyAsync(&pinned[0], &m->state->next_token, 4, cudaMemcpyDeviceToHost, m->stream);
-    if (e == cudaSuccess) e = cudaMemcpyAsync(&m->state->gen_cursor, window, 8, cudaMemcpyHostToDevice, m->stream);
-    for (uint32_t i = 0; i < steps && e == cudaSuccess; ++i) {
-        if (launch_token(m, true) != STARK_B200_OK) e = last_cuda_error() != cudaSuccess ? last_cuda_error() : cudaErrorUnknown;
-    }
-    if (e == cudaSuccess && steps)
-        e = cudaMemcpyAsync(&pinned[1], m->generated, (size_t)steps * 4u, cudaMemcpyDeviceToHost, m->stream);
-    const uint32_t closed[2] = {0u, 0u};
-    if (e == cudaSuccess) e = cudaMemcpyAsync(&m->state->gen_cursor, closed, 8, cudaMemcpyHostToDevice, m->stream);
-    if (e == cudaSuccess) e = cudaStreamSynchronize(m->stream);
-    if (e == cudaSuccess) memcpy(out_tokens, pinned, (size_t)(steps + 1u) * 4u);
-    cudaFreeHost(pinned);
-    if (e != cudaSuccess) {
-        m->fenced = true;
-        return cuda_status(e);
-    }
-    m->position += steps;
-    m->launches_issued += (uint64_t)steps * m->step_launches;
-    return check_device_error(m);
-}
-
-// Copies out the timeline slots of the launches issued since the last call and re-arms them.
-stark_b200_status model_read_trace(Model *m, unsigned long long *dst, size_t count) {
-    if (!m->trace) return STARK_B200_UNSUPPORTED;
-    if (count != (size_t)m->trace_slots * kTraceFields) return STARK_B200_INVALID_ARGUMENT;
-    SB_CUDA(cudaStreamSynchronize(m->stream));
-    SB_CUDA(cudaMemcpy(dst, m->trace, count * 8u, cudaMemcpyDeviceToHost));
-    std::vector<TraceSlot> init(m->trace_slots, TraceSlot{~0ull, ~0ull, 0ull, 0ull, 0ull, 0ull});
-    SB_CUDA(cudaMemcpy(m->trace, init.data(), count * 8u, cudaMemcpyHostToDevice));
-    return STARK_B200_OK;
-}
+const ModelFamily kDenseFamily = make_dense_family();
 
 }  // namespace sb

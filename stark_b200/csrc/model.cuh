@@ -48,8 +48,47 @@ struct MtpHead {
     bool has_pending = false;
 };
 
+struct Model;
+struct LayeredState;  // layered.cuh
+
+// What a family of decoders supplies to the shared token loop (token_loop.cu).  Optional entries may be nullptr.
+struct ModelFamily {
+    const char *name;
+    uint32_t min_rows = UINT32_MAX;                 // fewest cache-only rows worth a batched pass (capped by the tunable)
+    uint32_t (*input_vocab)(const Model *);         // token ids are below this
+    stark_b200_status (*ready)(Model *);            // INVALID_STATE while a tensor is missing
+    // Issues the kernels of one token on m->stream.  full == false: cache only, the next token from the pending list.
+    stark_b200_status (*issue_token)(Model *, bool full, uint32_t *launches);
+    stark_b200_status (*first_pass)(Model *);       // optional: the eager pass before recording
+    stark_b200_status (*recorded)(Model *);         // optional: after the sequences are recorded
+    stark_b200_status (*launch_token)(Model *, bool full);  // optional: the persistent form of a token
+    void (*retune)(Model *);                        // optional: picks up changed launch-shape settings
+    bool (*rows_ready)(Model *);                    // batched passes serve this model (m->chunk_tokens exists then)
+    stark_b200_status (*rows_pass)(Model *, const uint32_t *tokens_device, uint32_t mrows, uint32_t first_pos);
+    // optional: logits of rows of the last pass, [count, vocab] on the host
+    stark_b200_status (*rows_logits)(Model *, const uint32_t *rows, uint32_t count, uint32_t mrows, float *dst);
+    stark_b200_status (*prompt_begin)(Model *, const uint32_t *ids);                                     // optional
+    stark_b200_status (*rows_done)(Model *, uint32_t mrows, uint32_t pairs, uint32_t first_pos);  // optional
+    stark_b200_status (*prompt_end)(Model *);                                                            // optional
+    stark_b200_status (*reset)(Model *);                                                                 // optional
+    stark_b200_status (*rewind)(Model *, uint64_t position);                                      // optional
+    void (*sizes)(const Model *, uint64_t *weight_bytes, uint64_t *kv_bytes_per_token);
+    void (*destroy)(Model *);                       // frees what the family allocated
+};
+extern const ModelFamily kDenseFamily;
+constexpr uint32_t kLogitsPartials = 1024;  // CTAs of a read-out matvec, at most
+
+template <typename T>
+inline stark_b200_status dmalloc(T **p, size_t count) {
+    *p = nullptr;
+    SB_CUDA(cudaMalloc(p, count * sizeof(T) ? count * sizeof(T) : 1));
+    return STARK_B200_OK;
+}
+
 struct Model {
-    stark_b200_dense_config cfg{};
+    stark_b200_dense_config cfg{};  // other families fill the sizes the token loop uses
+    const ModelFamily *family = nullptr;
+    LayeredState *layered = nullptr;
     int device = 0;
     cudaStream_t stream = nullptr;
     QMatrix *embed = nullptr, *lm_head = nullptr;
@@ -66,6 +105,7 @@ struct Model {
     uint32_t trace_slots = 0;
     uint16_t *h_alt = nullptr;      // second residual-stream buffer (tensor parallel only)
     uint16_t *h = nullptr, *qkv = nullptr, *attn = nullptr, *act = nullptr, *logits = nullptr;
+    float *logits_f32 = nullptr;    // instead of `logits` where the family reads out in f32
     float *attn_scratch = nullptr;
     uint32_t *attn_counters = nullptr;
     float *partial_max = nullptr;
@@ -111,6 +151,7 @@ struct Model {
     ~Model();
 };
 
+stark_b200_status model_create_session(Model *m, bool f32_logits);
 stark_b200_status model_create(const stark_b200_dense_config &cfg, Model **out);
 stark_b200_status model_set_matrix(Model *m, uint32_t layer, uint32_t which, QMatrix *q);  // takes ownership
 stark_b200_status model_set_vector(Model *m, uint32_t layer, uint32_t which, const float *data, uint32_t count);
@@ -131,9 +172,10 @@ stark_b200_status model_reset(Model *m);
 stark_b200_status model_recapture(Model *m);
 stark_b200_status model_rewind(Model *m, uint64_t position);
 stark_b200_status model_prefill(Model *m, const uint32_t *ids, size_t count);
+stark_b200_status model_prefill_rows(Model *m, const uint32_t *ids, size_t count, const uint32_t *wanted, size_t wanted_count,
+                                     float *dst);
 stark_b200_status model_step(Model *m, uint32_t token, bool chained);
 bool model_batched_prefill_ready(Model *m);
-stark_b200_status model_prefill_batched(Model *m, const uint32_t *ids, size_t rows, size_t ids_total);
 stark_b200_status model_rows_pass(Model *m, const uint32_t *tokens_device, uint32_t mrows, uint32_t first_pos);
 stark_b200_status ensure_chunk_buffers(Model *m);
 stark_b200_status model_drain(Model *m);

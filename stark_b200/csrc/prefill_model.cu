@@ -205,22 +205,4 @@ stark_b200_status model_rows_pass(Model *m, const uint32_t *tokens_device, uint3
     return STARK_B200_OK;
 }
 
-// Ingests `rows` prompt rows starting at position m->position (cache only: no logits).  The caller has checked
-// ids and the context limit.  With a draft head loaded, every chunk also primes the head's cache with the pairs
-// (next prompt token, this row's normalized hidden): dense_mtp.rs:462-584.
-stark_b200_status model_prefill_batched(Model *m, const uint32_t *ids, size_t rows, size_t ids_total) {
-    stark_b200_status st;
-    for (size_t done = 0; done < rows; done += kPrefillBatchRows) {
-        if (m->cancel_requested) return STARK_B200_CANCELLED;
-        const uint32_t mrows = (uint32_t)std::min<size_t>(kPrefillBatchRows, rows - done);
-        const uint32_t first_pos = (uint32_t)(m->position + done);
-        // one extra id when there is one: the head's pairs need the token after each row
-        const size_t upload = std::min<size_t>((size_t)mrows + 1u, ids_total - done);
-        SB_CUDA(cudaMemcpyAsync(m->chunk_tokens, ids + done, upload * 4u, cudaMemcpyHostToDevice, m->stream));
-        if ((st = model_rows_pass(m, m->chunk_tokens, mrows, first_pos)) != STARK_B200_OK) return st;
-        if (m->mtp.enabled && (st = mtp_prime_rows(m, mrows, (uint32_t)(upload - 1u), first_pos)) != STARK_B200_OK) return st;
-    }
-    return STARK_B200_OK;
-}
-
 }  // namespace sb
