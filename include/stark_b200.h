@@ -644,6 +644,74 @@ stark_b200_status stark_b200_moe_model_launches_per_token(const stark_b200_moe_m
 stark_b200_status stark_b200_moe_model_stream(const stark_b200_moe_model *model, void **out_stream);
 stark_b200_status stark_b200_moe_model_destroy(stark_b200_moe_model **model);
 
+/* ------------------------------------------------------------------------------------------
+ * Layered decoders: a model whose configuration lists every layer's mixer and feed-forward with sizes of their own
+ * (Guvulorn), over bf16 weights.  Nothing in the reference corresponds to it.  Built empty from its description,
+ * filled tensor by tensor, finalized; from then on the handle is an ordinary stark_b200_model: prefill, prefill_rows,
+ * step, read-outs, sample, generate_greedy, rewind, reset, get_info, destroy.
+ */
+#define STARK_B200_MIXER_LATENT 1u     /* attention over a cached latent and a shared rotated key part */
+#define STARK_B200_FF_NONE 0u
+#define STARK_B200_FF_CLAMPED_GATE 1u  /* min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1), with biases */
+#define STARK_B200_ROT_PLAIN 0u
+#define STARK_B200_ROT_YARN 1u         /* frequencies blended with themselves / factor between two pair indices */
+typedef struct stark_b200_layer_desc {
+    uint32_t struct_size;
+    uint32_t mixer;
+    uint32_t feed_forward;
+    uint32_t weights_of;  /* UINT32_MAX: tensors of its own; otherwise the layer whose tensors it uses (cache of its own) */
+    uint32_t heads;
+    uint32_t dim;      /* unrotated query / key entries per head */
+    uint32_t rot_dim;  /* rotated query / key entries per head */
+    uint32_t vdim;     /* value entries per head */
+    uint32_t kv_rank;  /* latent entries */
+    uint32_t ff_width;
+    float scale;       /* on the scores */
+    float ff_limit;
+    uint32_t rot_dims; /* entries of the rotated part that rotate (interleaved pairs); the rest pass unchanged */
+    uint32_t rot_scaling;
+    double rot_base;
+    double rot_factor, rot_original, rot_fast, rot_slow; /* STARK_B200_ROT_YARN */
+} stark_b200_layer_desc;
+typedef struct stark_b200_layered_config {
+    uint32_t struct_size;
+    uint32_t abi_version;
+    uint32_t vocab;
+    uint32_t width;
+    uint32_t layers;
+    uint32_t context_tokens;
+    uint32_t compute;        /* STARK_B200_BF16: bf16 products with f32 accumulation, bf16 cache; STARK_B200_F32: all f32 */
+    uint32_t bigram_buckets; /* 0: no bigram table */
+    uint64_t bigram_mul_prev, bigram_mul_cur;
+    float embed_scale;
+    float eps;
+} stark_b200_layered_config;
+/* Which tensor a set call addresses; all bf16, row-major [rows, columns] (vectors: rows = 1), in the model's own
+ * layout -- the library pads and fuses. */
+#define STARK_B200_LAYERED_EMBED 0u      /* [vocab, width] */
+#define STARK_B200_LAYERED_BIGRAM 1u     /* [buckets + 1, width] */
+#define STARK_B200_LAYERED_EMBED_NORM 2u
+#define STARK_B200_LAYERED_FINAL_NORM 3u
+#define STARK_B200_LAYERED_HEAD 4u       /* [vocab, width] */
+#define STARK_B200_LAYERED_NORM1 5u
+#define STARK_B200_LAYERED_Q 6u          /* [heads * (dim + rot_dim), width] */
+#define STARK_B200_LAYERED_DKV 7u        /* [kv_rank + rot_dim, width] */
+#define STARK_B200_LAYERED_DKV_NORM 8u   /* [kv_rank] */
+#define STARK_B200_LAYERED_UK 9u         /* [heads * dim, kv_rank] */
+#define STARK_B200_LAYERED_UV 10u        /* [heads * vdim, kv_rank] */
+#define STARK_B200_LAYERED_O 11u         /* [width, heads * vdim] */
+#define STARK_B200_LAYERED_NORM2 12u
+#define STARK_B200_LAYERED_GATE 13u      /* [ff_width, width] */
+#define STARK_B200_LAYERED_GATE_BIAS 14u
+#define STARK_B200_LAYERED_UP 15u
+#define STARK_B200_LAYERED_UP_BIAS 16u
+#define STARK_B200_LAYERED_DOWN 17u      /* [width, ff_width] */
+#define STARK_B200_LAYERED_DOWN_BIAS 18u
+stark_b200_status stark_b200_layered_create(const stark_b200_layered_config *config, const stark_b200_layer_desc *layers,
+                                            stark_b200_model **out_model);
+stark_b200_status stark_b200_layered_set_tensor(stark_b200_model *model, uint32_t layer, uint32_t which,
+                                                const void *data_bf16, uint32_t rows, uint32_t columns);
+
 #ifdef __cplusplus
 }
 #endif

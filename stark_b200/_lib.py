@@ -10,6 +10,9 @@ from pathlib import Path
 
 PKG = Path(__file__).resolve().parent
 LIB_PATH = PKG / "libstark_b200.so"
+# The shared token loop and the layered family alone (``build.build("layered")``): what a process that serves only such
+# a model needs compiled.
+LAYERED_LIB_PATH = PKG / "libstark_b200_layered.so"
 
 ABI_VERSION = 1
 HOST, DEVICE = 0, 1
@@ -51,6 +54,27 @@ class MoeConfig(C.Structure):
                                           "experts", "active_experts", "expert_intermediate", "context_tokens")] + [
         ("rms_eps", C.c_float), ("rope_theta", C.c_float)]
 
+
+class LayerDesc(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("struct_size", "mixer", "feed_forward", "weights_of", "heads", "dim", "rot_dim",
+                                          "vdim", "kv_rank", "ff_width")] + [
+        ("scale", C.c_float), ("ff_limit", C.c_float), ("rot_dims", C.c_uint32), ("rot_scaling", C.c_uint32)] + [
+        (n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("struct_size", "abi_version", "vocab", "width", "layers", "context_tokens",
+                                          "compute", "bigram_buckets")] + [
+        ("bigram_mul_prev", C.c_uint64), ("bigram_mul_cur", C.c_uint64), ("embed_scale", C.c_float), ("eps", C.c_float)]
+
+
+MIXER_LATENT = 1
+FF_NONE, FF_CLAMPED_GATE = 0, 1
+ROT_PLAIN, ROT_YARN = 0, 1
+NO_LAYER = 0xFFFFFFFF
+(LAYERED_EMBED, LAYERED_BIGRAM, LAYERED_EMBED_NORM, LAYERED_FINAL_NORM, LAYERED_HEAD, LAYERED_NORM1, LAYERED_Q, LAYERED_DKV,
+ LAYERED_DKV_NORM, LAYERED_UK, LAYERED_UV, LAYERED_O, LAYERED_NORM2, LAYERED_GATE, LAYERED_GATE_BIAS, LAYERED_UP,
+ LAYERED_UP_BIAS, LAYERED_DOWN, LAYERED_DOWN_BIAS) = range(19)
 
 MOE_MAT_QKV, MOE_MAT_O, MOE_MAT_GATE_UP, MOE_MAT_DOWN, MOE_MAT_OUTPUT = range(5)
 (MOE_ATTN_NORM, MOE_FFN_NORM, MOE_Q_NORM, MOE_K_NORM, MOE_FINAL_NORM, MOE_ROUTER, MOE_TOKEN_TABLE) = range(7)
@@ -103,16 +127,17 @@ def sampling(seed=None, temperature=None, top_k=None, top_p=None, min_p=None, or
 _lib = None
 
 
-def load() -> C.CDLL:
-    """Load the shared library; raises if it is missing (build it with ``python -m stark_b200.build``)."""
+def load(path: Path = LIB_PATH) -> C.CDLL:
+    """Load the shared library; raises if it is missing (build it with ``python -m stark_b200.build``).  A process loads
+    one library: the first call's."""
     global _lib
     if _lib is not None:
         return _lib
-    if not LIB_PATH.exists():
+    if not path.exists():
         raise RuntimeError(
-            f"{LIB_PATH} is missing: the CUDA library has not been built "
+            f"{path} is missing: the CUDA library has not been built "
             "(run `python -m stark_b200.build`); there is no fallback path")
-    lib = C.CDLL(str(LIB_PATH))
+    lib = C.CDLL(str(path))
     vp, u32, u64, sz = C.c_void_p, C.c_uint32, C.c_uint64, C.c_size_t
     sig = {
         "stark_b200_abi_version": (u32, []),
@@ -201,13 +226,20 @@ def load() -> C.CDLL:
         "stark_b200_moe_model_launches_per_token": (u32, [vp, C.POINTER(u32)]),
         "stark_b200_moe_model_stream": (u32, [vp, C.POINTER(vp)]),
         "stark_b200_moe_model_destroy": (u32, [C.POINTER(vp)]),
+        "stark_b200_layered_create": (u32, [C.POINTER(LayeredConfig), C.POINTER(LayerDesc), C.POINTER(vp)]),
+        "stark_b200_layered_set_tensor": (u32, [vp, u32, u32, vp, u32, u32]),
         "stark_b200_graph_begin": (u32, [vp]),
         "stark_b200_graph_end": (u32, [vp, C.POINTER(vp)]),
         "stark_b200_graph_launch": (u32, [vp, vp]),
         "stark_b200_graph_destroy": (u32, [C.POINTER(vp)]),
     }
     for name, (res, args) in sig.items():
-        fn = getattr(lib, name)
+        try:
+            fn = getattr(lib, name)
+        except AttributeError:
+            if path == LIB_PATH:
+                raise
+            continue  # the part of the library that was built does not have this family
         fn.restype = res
         fn.argtypes = args
     if lib.stark_b200_abi_version() != ABI_VERSION:

@@ -173,6 +173,107 @@ def read_artifact(directory) -> tuple[dict, dict]:
     return cfg, out
 
 
+# ----------------------------------------------------------------------------- layered decoders
+
+LAYERED_ARCHITECTURES = ("Guvulorn",)
+
+
+def layered_config(root: dict) -> dict:
+    """The engine's description of a layered decoder from its ``config.json``: model-wide sizes and constants, and per
+    layer the latent attention's sizes, its rotation, the feed-forward and whose tensors it uses."""
+    if root.get("architecture") not in LAYERED_ARCHITECTURES:
+        raise ArtifactError(f"architecture {root.get('architecture')} is not a layered decoder this engine knows")
+    layers = []
+    for i, entry in enumerate(root["layers"]):
+        if not str(entry["type"]).startswith("latent_attention"):
+            raise ArtifactError(f"layer {i}: mixer {entry['type']} is not implemented")
+        m, mlp, rot = entry["mixer"], entry.get("mlp"), entry["mixer"].get("rot")
+        ff = None
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise ArtifactError(f"layer {i}: feed-forward {mlp['kind']} is not implemented")
+            ff = dict(width=int(mlp["ff"]), limit=float(mlp["limit"]))
+        scaling = rot.get("scaling")
+        layers.append(dict(
+            heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+            kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), ff=ff,
+            rot=dict(base=float(rot["base"]), dims=int(rot.get("dims", m["rot_dim"])),
+                     scaling=None if scaling is None else {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}),
+            weights_of=None if entry.get("weights_of") is None else int(entry["weights_of"])))
+    for i, layer in enumerate(layers):  # a layer that points to one without tensors of its own means that one's source
+        seen = {i}
+        while layer["weights_of"] is not None and layers[layer["weights_of"]]["weights_of"] is not None:
+            layer["weights_of"] = layers[layer["weights_of"]]["weights_of"]
+            if layer["weights_of"] in seen:
+                raise ArtifactError(f"layer {i}: circular weights_of")
+            seen.add(layer["weights_of"])
+    emb = root["embedding"]
+    bigram = emb.get("bigram")
+    return dict(architecture=root["architecture"], vocab=int(root["vocab"]), width=int(root["width"]),
+                eps=float(root["norm"]["eps"]), embed_scale=float(emb.get("scale", 1.0)),
+                bigram=None if bigram is None else {k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")},
+                layers=layers)
+
+
+def layered_tensors(cfg: dict) -> list[tuple]:
+    """Every tensor of a layered decoder: (name in the file, layer, id of the set call, shape)."""
+    from . import _lib as L
+    D, V = cfg["width"], cfg["vocab"]
+    out = [("embed", 0, L.LAYERED_EMBED, (V, D)), ("embed.norm", 0, L.LAYERED_EMBED_NORM, (D,)),
+           ("final.norm", 0, L.LAYERED_FINAL_NORM, (D,)), ("head", 0, L.LAYERED_HEAD, (V, D))]
+    if cfg["bigram"] is not None:
+        out.append(("bigram", 0, L.LAYERED_BIGRAM, (cfg["bigram"]["buckets"] + 1, D)))
+    for i, l in enumerate(cfg["layers"]):
+        if l["weights_of"] is not None:
+            continue
+        p, H, dim, rd, vd, rank = f"l{i}", l["heads"], l["dim"], l["rot_dim"], l["vdim"], l["kv_rank"]
+        out += [(p + ".norm1", i, L.LAYERED_NORM1, (D,)), (p + ".mix.q", i, L.LAYERED_Q, (H * (dim + rd), D)),
+                (p + ".mix.dkv", i, L.LAYERED_DKV, (rank + rd, D)), (p + ".mix.dkv.norm", i, L.LAYERED_DKV_NORM, (rank,)),
+                (p + ".mix.uk", i, L.LAYERED_UK, (H * dim, rank)), (p + ".mix.uv", i, L.LAYERED_UV, (H * vd, rank)),
+                (p + ".mix.o", i, L.LAYERED_O, (D, H * vd))]
+        if l["ff"] is not None:
+            F = l["ff"]["width"]
+            out += [(p + ".norm2", i, L.LAYERED_NORM2, (D,)),
+                    (p + ".mlp.gate", i, L.LAYERED_GATE, (F, D)), (p + ".mlp.gate.b", i, L.LAYERED_GATE_BIAS, (F,)),
+                    (p + ".mlp.up", i, L.LAYERED_UP, (F, D)), (p + ".mlp.up.b", i, L.LAYERED_UP_BIAS, (F,)),
+                    (p + ".mlp.down", i, L.LAYERED_DOWN, (D, F)), (p + ".mlp.down.b", i, L.LAYERED_DOWN_BIAS, (D,))]
+    return out
+
+
+def read_layered(directory) -> tuple[dict, dict]:
+    """Returns ``(cfg, weights)`` in the form ``LayeredModel.load`` takes.  Strict: every tensor must have the shape the
+    configuration gives it, and every tensor of the file must be used."""
+    directory = Path(directory)
+    try:
+        cfg = layered_config(json.loads((directory / "config.json").read_text()))
+    except (KeyError, TypeError, AttributeError) as e:
+        raise ArtifactError(f"config.json lacks or mistypes {e}") from None
+    header, _, data = _read_safetensors(directory / "model.safetensors")
+    used: set = set()
+    weights = {name: _tensor(header, data, name, "BF16", shape, used) for name, _, _, shape in layered_tensors(cfg)}
+    extra = set(header) - used
+    if extra:
+        raise ArtifactError(f"artifact has {len(extra)} tensors the decoder does not use, e.g. {sorted(extra)[0]}")
+    return cfg, weights
+
+
+def write_layered(directory, root: dict, weights: dict) -> None:
+    """Writes a layered decoder's ``config.json`` (``root``) and ``model.safetensors`` (name -> bf16 bit patterns)."""
+    directory = Path(directory)
+    directory.mkdir(parents=True, exist_ok=True)
+    (directory / "config.json").write_text(json.dumps(root, indent=1))
+    header, offset = {}, 0
+    for name, a in weights.items():
+        header[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [offset, offset + a.nbytes]}
+        offset += a.nbytes
+    encoded = json.dumps(header).encode("utf-8")
+    encoded += b" " * (-len(encoded) % 8)
+    with (directory / "model.safetensors").open("wb") as f:
+        f.write(struct.pack("<Q", len(encoded)) + encoded)
+        for a in weights.values():
+            f.write(np.ascontiguousarray(a, np.uint16).tobytes())
+
+
 # ----------------------------------------------------------------------------- writer (tests, synthetic models)
 
 def write_artifact(directory, cfg: dict, weights: dict) -> None:

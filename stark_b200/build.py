@@ -17,6 +17,12 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 OBJ = PKG / "csrc" / "build"
 LIB = PKG / "libstark_b200.so"
+# Parts of the library a process may need alone: (library, sources).
+PARTS = {
+    "layered": (PKG / "libstark_b200_layered.so",
+                ("abi_core", "abi_session", "token_loop", "layered_model", "layered_rows", "dense_b16", "gemm_b16",
+                 "latent_attention", "latent_attention_tc", "ops", "sampling", "tunables")),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -41,11 +47,24 @@ def _stale(target: Path, deps: list[Path]) -> bool:
     return any(d.stat().st_mtime > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def _headers() -> list[Path]:
+    return sorted(CSRC.glob("*.cuh")) + [PKG.parent / "include" / "stark_b200.h"]
+
+
+def ensure(part: str) -> Path:
+    """The library a process that needs only ``part`` should load: the whole one where it is built and current,
+    otherwise the part's own, compiled if need be."""
+    if not _stale(LIB, sorted(CSRC.glob("*.cu")) + _headers()):
+        return LIB
+    return build(part=part)
+
+
+def build(force: bool = False, verbose: bool = False, part: str | None = None) -> Path:
     nvcc = _nvcc()
     OBJ.mkdir(exist_ok=True)
-    sources = sorted(CSRC.glob("*.cu"))
-    headers = sorted(CSRC.glob("*.cuh")) + [PKG.parent / "include" / "stark_b200.h"]
+    lib = LIB if part is None else PARTS[part][0]
+    sources = sorted(CSRC.glob("*.cu")) if part is None else [CSRC / (n + ".cu") for n in PARTS[part][1]]
+    headers = _headers()
     env = dict(os.environ)
     env.pop("CC", None)
     env.pop("CXX", None)
@@ -63,14 +82,14 @@ def build(force: bool = False, verbose: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(sources))) as pool:
         objs = list(pool.map(compile_one, sources))
-    if force or _stale(LIB, objs):
-        cmd = [nvcc, "-shared", "-ccbin", "/usr/bin/g++", "-o", str(LIB), *map(str, objs), "-lcudart"]
+    if force or _stale(lib, objs):
+        cmd = [nvcc, "-shared", "-ccbin", "/usr/bin/g++", "-Xlinker", "-z,defs", "-o", str(lib), *map(str, objs), "-lcudart"]
         res = subprocess.run(cmd, capture_output=True, text=True, env=env)
         if res.returncode:
             sys.stderr.write(res.stdout + res.stderr)
-            raise RuntimeError("link of libstark_b200.so failed")
-    return LIB
+            raise RuntimeError(f"link of {lib.name} failed")
+    return lib
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose=True))
+    print(build(force="--force" in sys.argv, verbose=True, part=next((p for p in PARTS if p in sys.argv), None)))

@@ -1,6 +1,6 @@
 """Host-side mirror of the reference's engine-level operator surface for the token loop.
 
-``DenseModel`` follows ``hybrid::Model`` (crates/stark-engine/src/engine/hybrid/mod.rs:347-1428):
+``SessionModel`` (with its families ``DenseModel`` and ``LayeredModel``) follows ``hybrid::Model`` (crates/stark-engine/src/engine/hybrid/mod.rs:347-1428):
 ``load`` -> ``reset`` -> ``ingest_prefix`` / ``prefill`` -> ``step(token) -> logits`` with the same
 argument meaning and error behaviour (invalid token or context overflow raise and leave the model
 reset).  All arithmetic happens in ``libstark_b200.so``; this class only marshals.
@@ -100,9 +100,158 @@ class TensorParallel:
         self.wait_ns, self.unanswered = wait_ns, bool(unanswered)
 
 
-class DenseModel:
-    PREFIX_CHUNK_TOKENS = 1024  # crates/stark-generate/src/prefix_cache.rs:14
+class SessionModel:
+    """One sequence on one handle: what every model family shares (prompt, step, read-outs, sampling, greedy chaining on
+    the device, prefix rewind).  A family's class builds the handle and loads its tensors."""
 
+    PREFIX_CHUNK_TOKENS = 1024  # crates/stark-generate/src/prefix_cache.rs:14
+    tp = None
+
+    def _gather_vocab(self, local: np.ndarray) -> np.ndarray:
+        """Whole-vocabulary vector from the ranks' read-out shards (identity on one GPU)."""
+        if self.tp is None:
+            return local
+        parts = self.tp.all_gather(local.tobytes())
+        return np.concatenate([np.frombuffer(p, local.dtype) for p in parts])
+
+    # ------------------------------------------------------------------ token loop
+    def reset(self):
+        check(_lib.load().stark_b200_reset(self._h), "reset")
+
+    def _guard(self, status: int, where: str):
+        if status != 0:
+            # hybrid::Model resets itself after any error (mod.rs:876-885)
+            if status not in (_lib.STATUS_NAMES.index("reload_required"),):
+                _lib.load().stark_b200_reset(self._h)
+            raise StarkB200Error(status, where)
+
+    def prefill(self, token_ids) -> None:
+        ids = np.ascontiguousarray(token_ids, np.uint32)
+        if self.tp is not None:
+            # Ranks wait for one another on the device with a time limit: line the hosts up where a
+            # request starts, so that host-side skew (tokenising, scoring) is not charged to that limit.
+            self.tp.all_gather(b"")
+        self._guard(_lib.load().stark_b200_prefill(self._h, ids.ctypes.data, ids.size), "prefill")
+
+    def prefill_rows(self, token_ids, wanted) -> np.ndarray:
+        """A portion of a prompt with the logits of chosen rows: ``wanted`` are ascending indices into ``token_ids``;
+        returns f32 ``[len(wanted), vocab]``."""
+        ids = np.ascontiguousarray(token_ids, np.uint32)
+        rows = np.ascontiguousarray(wanted, np.uint32)
+        out = np.empty((rows.size, self.cfg["vocab"]), np.float32)
+        self._guard(_lib.load().stark_b200_prefill_rows(self._h, ids.ctypes.data, ids.size, rows.ctypes.data, rows.size,
+                                                        out.ctypes.data), "prefill_rows")
+        return out
+
+    def ingest_prefix(self, token_ids) -> None:
+        self.prefill(token_ids)
+
+    def step(self, token: int) -> np.ndarray:
+        """Feed one token, return the full-vocabulary logits (f32) of its row."""
+        self._guard(_lib.load().stark_b200_step(self._h, int(token)), "step")
+        return self.logits()
+
+    def step_async(self, token: int) -> None:
+        self._guard(_lib.load().stark_b200_step(self._h, int(token)), "step")
+
+    def logits(self) -> np.ndarray:
+        out = np.empty(self.cfg["vocab"], np.float32)
+        self._guard(_lib.load().stark_b200_readout_f32(self._h, out.ctypes.data, out.size), "readout_f32")
+        return self._gather_vocab(out)
+
+    def logits_bf16(self) -> np.ndarray:
+        out = np.empty(self.cfg["vocab"], np.uint16)
+        self._guard(_lib.load().stark_b200_readout_bf16(self._h, out.ctypes.data, out.size), "readout_bf16")
+        return self._gather_vocab(out)
+
+    def log_probabilities(self) -> np.ndarray:
+        if self.tp is not None:  # normalise over the gathered vocabulary with the same f64 kernel
+            from . import ops
+            return ops.log_softmax(self.logits()).astype(np.float32)
+        out = np.empty(self.cfg["vocab"], np.float32)
+        self._guard(_lib.load().stark_b200_readout_logprobs_f32(self._h, out.ctypes.data, out.size),
+                    "readout_logprobs_f32")
+        return out
+
+    def argmax(self) -> int:
+        t = C.c_uint32(0)
+        self._guard(_lib.load().stark_b200_argmax(self._h, C.byref(t)), "argmax")
+        return t.value
+
+    def sample(self, seed=None, temperature=None, top_k=None, top_p=None, min_p=None, ordered: bool = False) -> int:
+        """One token from the last row's logits through the device sampler (the reference's unified
+        sampler; ``seed`` is the per-position seed, see ``position_seed``).  ``ordered`` selects the
+        generation worker's host-sampler semantics instead (crates/stark-generate/src/hybrid.rs:1122-1212);
+        ``seed`` is then the SplitMix64 state before the draw."""
+        params = _lib.sampling(seed, temperature, top_k, top_p, min_p, ordered)
+        t = C.c_uint32(0)
+        self._guard(_lib.load().stark_b200_sample(self._h, C.byref(params), C.byref(t)), "sample")
+        return t.value
+
+    def generate_greedy(self, steps: int) -> np.ndarray:
+        out = np.empty(steps + 1, np.uint32)
+        self._guard(_lib.load().stark_b200_generate_greedy(self._h, steps, out.ctypes.data), "generate_greedy")
+        return out
+
+    def rewind(self, position: int) -> None:
+        check(_lib.load().stark_b200_rewind(self._h, position), "rewind")
+
+    def drain(self) -> None:
+        check(_lib.load().stark_b200_drain(self._h), "drain")
+
+    def cancel(self) -> None:
+        check(_lib.load().stark_b200_cancel(self._h), "cancel")
+
+    def info(self) -> _lib.Info:
+        i = _lib.Info()
+        i.struct_size = C.sizeof(_lib.Info)
+        i.abi_version = _lib.ABI_VERSION
+        check(_lib.load().stark_b200_get_info(self._h, C.byref(i)), "get_info")
+        return i
+
+    def read_trace(self) -> np.ndarray:
+        """Timeline of the launches since the last call, ``uint64[launches_per_step, 6]`` (ns): first CTA
+        entered, first wait returned, last prologue done, last CTA left, last CTA entered, last wait returned."""
+        n = self.info().trace_slots
+        out = np.empty((n, 6), np.uint64)
+        check(_lib.load().stark_b200_read_trace(self._h, out.ctypes.data, out.size), "read_trace")
+        return out
+
+    def recapture(self, **tunables: int) -> None:
+        """Sets launch-shape settings (``stark_b200_set_tunable`` names) and records the token sequences again."""
+        for name, value in tunables.items():
+            check(_lib.load().stark_b200_set_tunable(name.encode(), int(value)), f"set_tunable {name}")
+        check(_lib.load().stark_b200_model_recapture(self._h), "model_recapture")
+
+    def stream(self) -> int:
+        """The cudaStream_t the model issues its work on (an integer handle)."""
+        p = C.c_void_p()
+        check(_lib.load().stark_b200_model_stream(self._h, C.byref(p)), "model_stream")
+        return p.value or 0
+
+    @property
+    def position(self) -> int:
+        return int(self.info().position)
+
+    def close(self, collective: bool = True):
+        if self._h and self._h.value and self.tp is not None and collective:
+            # peers read this rank's exchange buffers: nobody unmaps before everybody is idle
+            try:
+                _lib.load().stark_b200_drain(self._h)
+                self.tp.all_gather(b"")
+            except Exception:
+                pass
+        if self._h and self._h.value:
+            _lib.load().stark_b200_destroy(C.byref(self._h))
+
+    def __del__(self):
+        try:
+            self.close(collective=False)
+        except Exception:
+            pass
+
+
+class DenseModel(SessionModel):
     def __init__(self, cfg: dict, context_tokens: int):
         self.cfg = dict(cfg)
         self.context_tokens = int(context_tokens)
@@ -220,106 +369,6 @@ class DenseModel:
         m.cfg = dict(vocab=int(info.vocab_size))
         return m
 
-    def _gather_vocab(self, local: np.ndarray) -> np.ndarray:
-        """Whole-vocabulary vector from the ranks' read-out shards (identity on one GPU)."""
-        if self.tp is None:
-            return local
-        parts = self.tp.all_gather(local.tobytes())
-        return np.concatenate([np.frombuffer(p, local.dtype) for p in parts])
-
-    # ------------------------------------------------------------------ token loop
-    def reset(self):
-        check(_lib.load().stark_b200_reset(self._h), "reset")
-
-    def _guard(self, status: int, where: str):
-        if status != 0:
-            # hybrid::Model resets itself after any error (mod.rs:876-885)
-            if status not in (_lib.STATUS_NAMES.index("reload_required"),):
-                _lib.load().stark_b200_reset(self._h)
-            raise StarkB200Error(status, where)
-
-    def prefill(self, token_ids) -> None:
-        ids = np.ascontiguousarray(token_ids, np.uint32)
-        if self.tp is not None:
-            # Ranks wait for one another on the device with a time limit: line the hosts up where a
-            # request starts, so that host-side skew (tokenising, scoring) is not charged to that limit.
-            self.tp.all_gather(b"")
-        self._guard(_lib.load().stark_b200_prefill(self._h, ids.ctypes.data, ids.size), "prefill")
-
-    def ingest_prefix(self, token_ids) -> None:
-        self.prefill(token_ids)
-
-    def step(self, token: int) -> np.ndarray:
-        """Feed one token, return the full-vocabulary logits (f32) of its row."""
-        self._guard(_lib.load().stark_b200_step(self._h, int(token)), "step")
-        return self.logits()
-
-    def step_async(self, token: int) -> None:
-        self._guard(_lib.load().stark_b200_step(self._h, int(token)), "step")
-
-    def logits(self) -> np.ndarray:
-        out = np.empty(self.cfg["vocab"], np.float32)
-        self._guard(_lib.load().stark_b200_readout_f32(self._h, out.ctypes.data, out.size), "readout_f32")
-        return self._gather_vocab(out)
-
-    def logits_bf16(self) -> np.ndarray:
-        out = np.empty(self.cfg["vocab"], np.uint16)
-        self._guard(_lib.load().stark_b200_readout_bf16(self._h, out.ctypes.data, out.size), "readout_bf16")
-        return self._gather_vocab(out)
-
-    def log_probabilities(self) -> np.ndarray:
-        if self.tp is not None:  # normalise over the gathered vocabulary with the same f64 kernel
-            from . import ops
-            return ops.log_softmax(self.logits()).astype(np.float32)
-        out = np.empty(self.cfg["vocab"], np.float32)
-        self._guard(_lib.load().stark_b200_readout_logprobs_f32(self._h, out.ctypes.data, out.size),
-                    "readout_logprobs_f32")
-        return out
-
-    def argmax(self) -> int:
-        t = C.c_uint32(0)
-        self._guard(_lib.load().stark_b200_argmax(self._h, C.byref(t)), "argmax")
-        return t.value
-
-    def sample(self, seed=None, temperature=None, top_k=None, top_p=None, min_p=None, ordered: bool = False) -> int:
-        """One token from the last row's logits through the device sampler (the reference's unified
-        sampler; ``seed`` is the per-position seed, see ``position_seed``).  ``ordered`` selects the
-        generation worker's host-sampler semantics instead (crates/stark-generate/src/hybrid.rs:1122-1212);
-        ``seed`` is then the SplitMix64 state before the draw."""
-        params = _lib.sampling(seed, temperature, top_k, top_p, min_p, ordered)
-        t = C.c_uint32(0)
-        self._guard(_lib.load().stark_b200_sample(self._h, C.byref(params), C.byref(t)), "sample")
-        return t.value
-
-    def generate_greedy(self, steps: int) -> np.ndarray:
-        out = np.empty(steps + 1, np.uint32)
-        self._guard(_lib.load().stark_b200_generate_greedy(self._h, steps, out.ctypes.data), "generate_greedy")
-        return out
-
-    def rewind(self, position: int) -> None:
-        check(_lib.load().stark_b200_rewind(self._h, position), "rewind")
-
-    def drain(self) -> None:
-        check(_lib.load().stark_b200_drain(self._h), "drain")
-
-    def cancel(self) -> None:
-        check(_lib.load().stark_b200_cancel(self._h), "cancel")
-
-    def info(self) -> _lib.Info:
-        i = _lib.Info()
-        i.struct_size = C.sizeof(_lib.Info)
-        i.abi_version = _lib.ABI_VERSION
-        check(_lib.load().stark_b200_get_info(self._h, C.byref(i)), "get_info")
-        return i
-
-    def read_trace(self) -> np.ndarray:
-        """Timeline of the launches since the last call, ``uint64[launches_per_step, 6]`` (ns): first CTA
-        entered, first wait returned, last prologue done, last CTA left, last CTA entered, last wait returned."""
-        n = self.info().trace_slots
-        out = np.empty((n, 6), np.uint64)
-        check(_lib.load().stark_b200_read_trace(self._h, out.ctypes.data, out.size), "read_trace")
-        return out
-
     # ------------------------------------------------------------------ multi-token prediction
     def mtp_initial(self) -> int:
         """After ``prefill``: the pending token (greedy pick of the prompt's last row), not yet committed."""
@@ -371,38 +420,52 @@ class DenseModel:
                     "mtp_readout_row_f32")
         return out
 
-    def recapture(self, **tunables: int) -> None:
-        """Sets launch-shape settings (``stark_b200_set_tunable`` names) and records the token sequences again."""
-        for name, value in tunables.items():
-            check(_lib.load().stark_b200_set_tunable(name.encode(), int(value)), f"set_tunable {name}")
-        check(_lib.load().stark_b200_model_recapture(self._h), "model_recapture")
 
-    def stream(self) -> int:
-        """The cudaStream_t the model issues its work on (an integer handle)."""
-        p = C.c_void_p()
-        check(_lib.load().stark_b200_model_stream(self._h, C.byref(p)), "model_stream")
-        return p.value or 0
+class LayeredModel(SessionModel):
+    """A layered decoder (``artifact.read_layered``): every layer's mixer and feed-forward as its configuration lists
+    them, over bf16 weights; ``dtype`` "bfloat16" or "float32" is the precision of products, activations and cache."""
 
-    @property
-    def position(self) -> int:
-        return int(self.info().position)
+    def __init__(self, cfg: dict, context_tokens: int, dtype: str = "bfloat16"):
+        self.cfg = dict(cfg)
+        self.context_tokens = int(context_tokens)
+        self.dtype = dtype
+        self._h = C.c_void_p()
+        bigram = cfg.get("bigram") or dict(buckets=0, mul_prev=0, mul_cur=0)
+        c = _lib.LayeredConfig(C.sizeof(_lib.LayeredConfig), _lib.ABI_VERSION, cfg["vocab"], cfg["width"],
+                               len(cfg["layers"]), self.context_tokens, {"bfloat16": _lib.BF16, "float32": _lib.F32}[dtype],
+                               bigram["buckets"], bigram["mul_prev"], bigram["mul_cur"], cfg["embed_scale"], cfg["eps"])
+        descs = (_lib.LayerDesc * len(cfg["layers"]))(*[self._desc(layer) for layer in cfg["layers"]])
+        check(_lib.load().stark_b200_layered_create(C.byref(c), descs, C.byref(self._h)), "layered_create")
 
-    def close(self, collective: bool = True):
-        if self._h and self._h.value and self.tp is not None and collective:
-            # peers read this rank's exchange buffers: nobody unmaps before everybody is idle
-            try:
-                _lib.load().stark_b200_drain(self._h)
-                self.tp.all_gather(b"")
-            except Exception:
-                pass
-        if self._h and self._h.value:
-            _lib.load().stark_b200_destroy(C.byref(self._h))
+    @staticmethod
+    def _desc(layer: dict) -> "_lib.LayerDesc":
+        rot, ff = layer["rot"], layer["ff"]
+        yarn = rot.get("scaling")
+        own = layer["weights_of"] is None
+        return _lib.LayerDesc(C.sizeof(_lib.LayerDesc), _lib.MIXER_LATENT, _lib.FF_NONE if ff is None else _lib.FF_CLAMPED_GATE,
+                              _lib.NO_LAYER if own else layer["weights_of"], layer["heads"], layer["dim"], layer["rot_dim"],
+                              layer["vdim"], layer["kv_rank"], 0 if ff is None else ff["width"], layer["scale"],
+                              0.0 if ff is None else ff["limit"], rot["dims"], _lib.ROT_YARN if yarn else _lib.ROT_PLAIN,
+                              rot["base"], *([yarn[k] for k in ("factor", "original", "fast", "slow")] if yarn else [0.0] * 4))
 
-    def __del__(self):
-        try:
-            self.close(collective=False)
-        except Exception:
-            pass
+    @classmethod
+    def load(cls, cfg: dict, weights: dict, context_tokens: int, dtype: str = "bfloat16") -> "LayeredModel":
+        """``weights``: tensor name -> bf16 bit patterns (uint16), vectors or [rows, columns], named as in the file."""
+        from .artifact import layered_tensors
+        m = cls(cfg, context_tokens, dtype)
+        for name, layer, which, shape in layered_tensors(cfg):
+            a = np.ascontiguousarray(weights[name], np.uint16)
+            rows, columns = (1, shape[0]) if len(shape) == 1 else shape
+            check(_lib.load().stark_b200_layered_set_tensor(m._h, layer, which, a.ctypes.data, rows, columns),
+                  f"layered_set_tensor {name}")
+        check(_lib.load().stark_b200_model_finalize(m._h), "model_finalize")
+        return m
+
+    @classmethod
+    def from_artifact(cls, directory, context_tokens: int, dtype: str = "bfloat16") -> "LayeredModel":
+        from .artifact import read_layered
+        cfg, weights = read_layered(directory)
+        return cls.load(cfg, weights, context_tokens, dtype)
 
 
 def position_seed(seed: int, position: int) -> int:

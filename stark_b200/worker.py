@@ -351,8 +351,8 @@ def read_frame(stream, wire_bytes: int):
 # ----------------------------------------------------------------------------------------------- backend
 
 class B200Backend:
-    """The engine behind both workers: a converted-model directory (``config.json`` + ``model.safetensors`` in the
-    reference's layout, optional ``tokenizer.json``) on one B200."""
+    """The engine behind both workers: a model directory (``config.json`` + ``model.safetensors``, optional
+    ``tokenizer.json``) of a family the registry knows, on one B200."""
 
     def __init__(self, path: Path, context_tokens: int | None = None):
         config = path / "config.json"
@@ -362,19 +362,15 @@ class B200Backend:
             root = json.loads(config.read_text())
         except (OSError, ValueError):
             raise Refusal("invalid_model_config") from None
-        from .artifact import ArtifactError, read_artifact
-        from .engine import DenseModel
+        from .artifact import ArtifactError
+        from .registry import open_model
         try:
-            cfg, weights = read_artifact(path)
+            self.opened = open_model(path)
         except (ArtifactError, KeyError, TypeError, OSError, ValueError):
             raise Refusal("invalid_model_config") from None
-        try:
-            layer0 = root["decoder_config"]["transformer_config"]["layer_configs"][0]
-            model_max = int(layer0["rope_config"].get("max_sequence_length") or 32768)
-        except (KeyError, IndexError, TypeError, ValueError):
-            model_max = 32768
+        cfg = self.opened.cfg
         want = context_tokens or int(os.environ.get("STARK_B200_WORKER_CONTEXT", "8192"))
-        self.capacity = max(2, min(model_max, want))
+        self.capacity = max(2, min(self.opened.max_context, want))
         generation = root.get("generation_config") or {}
         self.eos = [int(t) for t in generation.get("stop_token_ids", []) if 0 <= int(t) < cfg["vocab"]]
         self.cfg = cfg
@@ -386,7 +382,7 @@ class B200Backend:
             except Exception:  # noqa: BLE001 - a tokenizer that does not load is a model that does not load
                 raise Refusal("tokenizer_unavailable") from None
         try:
-            self.model = DenseModel.load(cfg, weights, context_tokens=self.capacity)
+            self.model = self.opened.load(self.capacity, os.environ.get("STARK_B200_WORKER_DTYPE"))
         except Exception:  # noqa: BLE001
             raise Refusal("model_load_failed") from None
         self.has_head = bool(cfg.get("mtp"))
@@ -418,17 +414,12 @@ class B200Backend:
 
     def plan_context_length(self, input_tokens: int, maximum: int, drafts: int):
         """The largest context up to `maximum` this engine can serve now.  The paged cache is allocated when the model
-        loads (`capacity` rows: 147 KB each for the 8B shape), so a context costs nothing further; what a request may
+        loads (`capacity` rows: 147 KB each for the 8B dense shape), so a context costs nothing further; what a request may
         still allocate are the working buffers of a prompt pass (4 096 rows of every intermediate) and, with
         proposals, the rows of the verify pass.  They have to fit the device memory that is free, with a reserve."""
         import ctypes as C
         from . import _lib
-        c = self.cfg
-        rows = 4096
-        qkv = (c["q_heads"] + 2 * c["kv_heads"]) * c["head_dim"]
-        scratch = rows * 2 * (2 * c["hidden"] + qkv + c["q_heads"] * c["head_dim"] + c["inter"])
-        if drafts:
-            scratch += 16 * 2 * (c["vocab"] + 4 * c["hidden"])
+        scratch = self.opened.prompt_scratch_bytes(drafts)
         free, total = C.c_uint64(0), C.c_uint64(0)
         try:
             _lib.check(_lib.load().stark_b200_device_memory(C.byref(free), C.byref(total)), "device_memory")
