@@ -40,6 +40,10 @@ WORKLOADS = {
     # routed-expert decoders (f32 host-path conventions, GGUF Q8_0 attention + Q4_K experts)
     "qwen3-30b-a3b": dict(cfg="qwen3-30b-a3b", prompt=2048, context=2048 + 512, moe=True),
     "moe-small": dict(cfg="moe-small", prompt=64, context=256, moe=True),
+    # layered decoders (bf16 weights, latent attention), with the dense family's model of equal size timed beside them
+    "guvulorn-8b": dict(layered="guvulorn-8b", cfg="qwen3-8b", prompt=4096, context=4096 + 1024),
+    "guvulorn-0.6b": dict(layered="guvulorn-0.6b", cfg="qwen3-0.6b", prompt=2048, context=2048 + 1024),
+    "guvulorn-8b-layers": dict(layered="guvulorn-8b-layers", cfg="qwen3-8b-layers", prompt=4096, context=4096 + 1024),
     # a single quantized matvec (BASELINE config 1 by default): micro-benchmark / profiling target
     "matvec": dict(cfg=None, prompt=0, context=0),
     # the prompt-chunk contraction alone (tensor-core GEMM over a 4-bit matrix): profiling target
@@ -416,6 +420,100 @@ def run_moe(args, wl) -> None:
         dist.destroy_process_group()
 
 
+def layered_work(root: dict, context: float) -> dict:
+    """Algorithmic work of a layered decoder: weights a token reads, bytes of a decode step over `context` cached rows,
+    and multiply-adds (x2) of a prompt of `context` rows in the expanded form."""
+    D, V = root["width"], root["vocab"]
+    w = kv = flops = 0.0
+    for l in root["layers"]:
+        m, F = l["mixer"], l["mlp"]["ff"] if l["mlp"] else 0
+        H, dim, rd, vd, r = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+        proj = (H * (dim + rd) + r + rd) * D + D * H * vd + 3 * F * D
+        up = H * (dim + vd) * r
+        w += proj + up
+        kv += (r + rd) * 2 * context
+        flops += 2.0 * context * (proj + up) + 2.0 * context * context / 2.0 * H * (dim + rd + vd)
+    return {"weights": w + V * D, "bytes": 2.0 * (w + V * D) + kv, "flops": flops}
+
+
+def run_layered(args, wl) -> None:
+    """Prompt and greedy decode of a layered decoder with random weights; the dense family's model of equal size (4-bit
+    weights) is timed the same way in the same process and printed beside it."""
+    import torch
+    from stark_b200.artifact import layered_config
+    from stark_b200.engine import DenseModel, LayeredModel
+    from stark_b200.ops import take_device_error
+    assert int(os.environ.get("WORLD_SIZE", "1")) == 1, "the layered workloads run on one GPU"
+    root = S.LAYERED_CONFIGS[wl["layered"]]
+    steps, warmup = args.steps, max(args.warmup, 3)
+    repeats = args.repeats if args.repeats > 0 else max(3, min(16, -(-160 // max(steps, 1))))
+    context = max(wl["context"], wl["prompt"] + warmup + repeats * steps + 8)
+    prompt = np.random.default_rng(args.seed + 1).integers(0, root["vocab"], wl["prompt"]).astype(np.uint32)
+
+    def timed(model, ids):
+        stream = torch.cuda.ExternalStream(model.stream())
+        marks = [torch.cuda.Event(enable_timing=True) for _ in range(repeats + 1)]
+        prefills = []
+        for i in range(4):   # the first allocates the row buffers
+            model.reset()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(stream)
+            model.prefill(ids)
+            b.record(stream)
+            model.drain()
+            if i:
+                prefills.append(a.elapsed_time(b))
+        model.generate_greedy(warmup)
+        torch.cuda.synchronize()
+        with ClockSampler(0) as clocks:
+            marks[0].record(stream)
+            for r in range(repeats):
+                model.generate_greedy(steps)
+                marks[r + 1].record(stream)
+            torch.cuda.synchronize()
+        regions = [marks[r].elapsed_time(marks[r + 1]) for r in range(repeats)]
+        # end to end: token in from the host, logits row out to the host, every step
+        model.reset()
+        model.prefill(ids)
+        token, n = model.argmax(), min(steps, 64)
+        t0 = time.perf_counter()
+        for _ in range(n):
+            token = int(model.step(token).argmax())
+        e2e = (time.perf_counter() - t0) / n
+        assert take_device_error() == 0, "a kernel reported a timed-out wait"
+        return float(np.median(regions)) / steps, float(np.median(prefills)), clocks.summary(), e2e
+
+    model = LayeredModel.load(layered_config(root), S.layered_weights(root, args.seed), context)
+    info = model.info()
+    ms, prefill_ms, clocks, e2e = timed(model, prompt)
+    model.close()
+    cfg = S.CONFIGS[wl["cfg"]]
+    dense = DenseModel.load(cfg, S.dense_weights(cfg, seed=args.seed), context_tokens=context)
+    dms, dprefill_ms, _, _ = timed(dense, prompt % cfg["vocab"])
+    dense.close()
+    peak, kind = peaks()
+    tpeak, tkind = tensor_peak()
+    rows = wl["prompt"] + warmup + repeats * steps / 2.0
+    step, ingest = layered_work(root, rows), layered_work(root, wl["prompt"] - 1)
+    gbs, tflops = step["bytes"] / ms / 1e6, ingest["flops"] / prefill_ms / 1e9
+    dbytes, dflops = step_bytes(cfg, rows), prefill_flops(cfg, wl["prompt"])
+    print(json.dumps({
+        "metric": "batch-1 decode tok/s", "value": 1e3 / ms, "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
+        "ms_per_step": ms, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic",
+        "config": {"workload": f"{wl['layered']} bf16 layered decoder, batch 1, {wl['prompt']}-token prompt, greedy decode",
+                   "l2": "per-step inputs (%.2f GB) exceed the 126 MB L2" % (step["bytes"] / 1e9),
+                   "timed_regions": {"repeats": repeats, "steps_each": steps, "value_from": "median region"}},
+        "e2e": {"value": 1.0 / e2e, "unit": "tok/s", "h2d_bytes_per_step": 4, "d2h_bytes_per_step": 4 * root["vocab"]},
+        "gpu_launches": int(repeats * steps * info.launches_per_step), "clocks": clocks,
+        "roofline": {"bound": "hbm", "achieved": gbs, "peak": peak, "unit": "GB/s", "frac": gbs / peak, "peak_kind": kind},
+        "prefill": {"ms": prefill_ms, "prefill_tok_s": wl["prompt"] / prefill_ms * 1e3, "achieved_tflops": tflops,
+                    "peak_tflops": tpeak, "frac": tflops / tpeak, "peak_kind": tkind},
+        "dense_of_equal_size": {"model": f"{wl['cfg']} 4-bit", "tok_s": 1e3 / dms, "hbm_frac": dbytes / dms / 1e6 / peak,
+                                "prefill_ms": dprefill_ms, "prefill_tok_s": wl["prompt"] / dprefill_ms * 1e3,
+                                "prefill_frac": dflops / dprefill_ms / 1e9 / tpeak}}))
+
+
 def mtp_round_bytes(cfg: dict, drafts: int, context_rows: float) -> float:
     """Algorithmic bytes of one speculative round: the target's matrices once (the verify pass reads each record
     once for all rows), its KV rows once, and per proposal the head's fusion matrix, its one layer, the read-out
@@ -589,6 +687,12 @@ def main() -> None:
     wl = WORKLOADS[args.workload]
     if wl.get("moe"):
         run_moe(args, wl)
+        return
+    if wl.get("layered"):
+        if args.impl == "reference":
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no layered decoder"}))
+            return
+        run_layered(args, wl)
         return
     if args.workload == "matvec":
         run_matvec(args)

@@ -316,7 +316,7 @@ stark_b200_status rows_attention(Model *m, const Layer &layer, uint32_t mrows, u
     a.qd_b16 = !L->f32;
     a.out_b16 = !L->f32;
     const size_t element = L->f32 ? 4u : 2u;
-    if (!L->f32 && mrows > kPrefillSmallRows && latent_prefill_tc_supports(layer.s)) {
+    if (!L->f32 && mrows > kPrefillSmallRows && layer.d.scale > 0.0f && latent_prefill_tc_supports(layer.s)) {
         const size_t visible = ((size_t)first_pos + mrows + kPageTokens - 1u) / kPageTokens * kPageTokens;
         if (L->expanded_rows < visible) {
             SB_CUDA(cudaStreamSynchronize(m->stream));

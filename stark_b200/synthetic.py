@@ -196,3 +196,47 @@ def moe_weights(cfg: dict, seed: int = 0) -> dict:
                 output=q8_0_rows(rng, cfg["vocab"], cfg["hidden"], scale=3e-4),
                 final_norm=(1.0 + 0.1 * rng.standard_normal(cfg["hidden"])).astype(np.float32),
                 layers=[moe_layer_weights(cfg, rng) for _ in range(cfg["layers"])])
+
+
+# ----------------------------------------------------------------------------- layered decoders
+
+def _layered(width, heads, rank, ff, layers, distinct, vocab=151936, dim=128, rot_dim=64, vdim=128) -> dict:
+    """A layered decoder's ``config.json`` at the sizes of a real model's layers; layers beyond the first ``distinct`` use
+    the tensors of those in turn (every layer's tensors are far larger than L2 together, so each is read from memory)."""
+    entries = []
+    for i in range(layers):
+        rot = {"base": 1e6, "dims": rot_dim}
+        if i % 2:
+            rot["scaling"] = {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+        e = {"type": "latent_attention" if i % 2 else "latent_attention_2",
+             "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank,
+                       "scale": (dim + rot_dim) ** -0.5, "rot": rot},
+             "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+        if i >= distinct:
+            e["weights_of"] = i % distinct
+        entries.append(e)
+    return {"architecture": "Guvulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 40503, "mul_cur": 9973}}, "layers": entries}
+
+
+LAYERED_CONFIGS = {
+    "guvulorn-8b": _layered(4096, 32, 512, 12288, 36, 4),
+    "guvulorn-0.6b": _layered(1024, 16, 256, 3072, 28, 28),
+    # two layers at the 8b dimensions: the same kernels on a gigabyte of weights
+    "guvulorn-8b-layers": _layered(4096, 32, 512, 12288, 2, 2, vocab=32768),
+}
+
+
+def layered_weights(root: dict, seed: int = 0) -> dict:
+    """bf16 bit patterns by tensor name: matrices uniform in sign and mantissa around 2^-6, norms and biases small."""
+    from .artifact import layered_config, layered_tensors
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, _, _, shape in layered_tensors(layered_config(root)):
+        if len(shape) == 1:
+            plain = name.endswith("dkv.norm")  # weight around one
+            out[name] = (np.full(shape, 1.0 if plain else 0.0, np.float32).view(np.uint32) >> 16).astype(np.uint16)
+        else:
+            bits = rng.integers(0, 1 << 16, shape, np.uint16, endpoint=False)
+            out[name] = (bits & np.uint16(0x807F)) | np.uint16(0x3C80 if name not in ("embed", "bigram") else 0x3F00)
+    return out
