@@ -214,10 +214,11 @@ stark_b200_status gemm_b16_launch(const GemmB16Args &a, cudaStream_t stream) {
     if (!make(&x_map, a.x, a.x_rows, a.ld_x, 128u) || !make(&w_map, a.w.data, a.w.rows, a.w.cols, kBN))
         return STARK_B200_DEVICE_FAILURE;
     const GemmB16Params p{a.w.cols / kBK, a.m, a.out_cols, a.ld_out, a.out, a.bias, a.limit, ctx->error_word};
-    // 256-row tiles unless they leave more SMs idle than 128-row tiles would
+    // 256-row tiles unless 128-row tiles fill the SMs so much better that it pays for their loading the weight tile
+    // once per 128 rows (a fifth slower per row)
     const uint32_t wide = (a.out_cols + kBN - 1u) / kBN, tall = (a.m + 255u) / 256u, flat = (a.m + 127u) / 128u;
     const uint32_t waves2 = (wide * tall + 147u) / 148u * 2u, waves1 = (wide * flat + 147u) / 148u;
-    return waves1 < waves2 ? launch<1>(a, x_map, w_map, p, stream) : launch<2>(a, x_map, w_map, p, stream);
+    return waves1 * 5u < waves2 * 4u ? launch<1>(a, x_map, w_map, p, stream) : launch<2>(a, x_map, w_map, p, stream);
 }
 
 }  // namespace sb

@@ -194,7 +194,7 @@ __global__ void __launch_bounds__(kAttendThreads) latent_attend_kernel(const Lat
 // blockIdx.x: (head, 64 output values), blockIdx.y: row
 template <typename O>
 __global__ void __launch_bounds__(256) latent_value_kernel(const LatentArgs a) {
-    extern __shared__ __align__(16) float o[];  // [rank_p]
+    extern __shared__ __align__(16) float o[];  // [rank_p], then the pieces of the merge
     __shared__ float weight[kLatentMaxSplits];
     const LatentShape &s = a.s;
     const uint32_t blocks = s.vdim_p / 64u, head = blockIdx.x / blocks, piece = blockIdx.x % blocks, row = blockIdx.y;
@@ -207,22 +207,50 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentArgs a) {
         w[j] = lane * 8u < s.rank_p ? ldg_nc_v4(uv + (size_t)j * s.rank_p + lane * 8u) : make_uint4(0u, 0u, 0u, 0u);
     pdl_launch_dependents();
     pdl_wait();
-    if (threadIdx.x < a.splits) weight[threadIdx.x] = partial_of(a, row, head, threadIdx.x)[0];
+    const float *part = partial_of(a, row, head, 0);
+    const uint32_t pitch = s.rank_p + 4u;
+    // every warp forms the spans' weights exp2(m - max) / sum for itself; the first one leaves them for the columns
+    {
+        float m[2], l[2], top = -INFINITY, sum = 0.0f;
+#pragma unroll
+        for (uint32_t j = 0; j < 2u; ++j) {
+            const uint32_t k = lane + 32u * j;
+            const float2 v = k < a.splits ? *reinterpret_cast<const float2 *>(part + (size_t)k * pitch) : make_float2(-INFINITY, 0.0f);
+            m[j] = v.x, l[j] = v.y;
+            top = fmaxf(top, v.x);
+        }
+        top = warp_max(top);
+#pragma unroll
+        for (uint32_t j = 0; j < 2u; ++j) {
+            m[j] = exp2f(m[j] - top);  // 0 for an empty span
+            sum = fmaf(m[j], l[j], sum);
+        }
+        const float inv = 1.0f / warp_sum(sum);
+        if (warp == 0u) weight[lane] = m[0] * inv, weight[lane + 32u] = m[1] * inv;
+    }
     __syncthreads();
-    float top = -INFINITY;
-    for (uint32_t k = 0; k < a.splits; ++k) top = fmaxf(top, weight[k]);
+    // four columns a thread; where the latent is narrow several threads share the spans of the same four
+    const uint32_t quads = s.rank_p / 4u, shares = quads >= 256u ? 1u : 256u / quads;
+    float4 *pieces = reinterpret_cast<float4 *>(o + s.rank_p);  // [shares][quads]
+    for (uint32_t t = threadIdx.x; t < quads * shares; t += 256u) {
+        const uint32_t quad = t % quads, share = t / quads;
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+        for (uint32_t k = share; k < a.splits; k += shares) {
+            const float4 x = *reinterpret_cast<const float4 *>(part + (size_t)k * pitch + 4u + quad * 4u);
+            const float c = weight[k];
+            v.x = fmaf(c, x.x, v.x), v.y = fmaf(c, x.y, v.y), v.z = fmaf(c, x.z, v.z), v.w = fmaf(c, x.w, v.w);
+        }
+        pieces[t] = v;
+    }
     __syncthreads();
-    if (threadIdx.x < a.splits) weight[threadIdx.x] = weight[threadIdx.x] == -INFINITY ? 0.0f : exp2f(weight[threadIdx.x] - top);
-    __syncthreads();
-    float l = 0.0f;
-    for (uint32_t k = 0; k < a.splits; ++k)
-        if (weight[k] != 0.0f) l += weight[k] * partial_of(a, row, head, k)[1];
-    const float inv = 1.0f / l;
-    for (uint32_t i = threadIdx.x; i < s.rank_p; i += 256u) {
-        float v = 0.0f;
-        for (uint32_t k = 0; k < a.splits; ++k)
-            if (weight[k] != 0.0f) v += weight[k] * partial_of(a, row, head, k)[4u + i];  // an empty span wrote nothing
-        o[i] = v * inv;
+    for (uint32_t quad = threadIdx.x; quad < quads; quad += 256u) {
+        float4 v = pieces[quad];
+        for (uint32_t k = 1; k < shares; ++k) {
+            const float4 x = pieces[k * quads + quad];
+            v.x += x.x, v.y += x.y, v.z += x.z, v.w += x.w;
+        }
+        reinterpret_cast<float4 *>(o)[quad] = v;
     }
     __syncthreads();
     float acc[8] = {};
@@ -298,6 +326,7 @@ stark_b200_status latent_query_launch(const LatentArgs &a, cudaStream_t stream) 
 stark_b200_status latent_attend_launch(const LatentArgs &a, cudaStream_t stream) {
     if (stark_b200_status st = check_args(a)) return st;
     if (!a.queries || !a.partials) return STARK_B200_INVALID_ARGUMENT;
+    if (!a.cache_f32 && latent_attend_mma_supports(a.s)) return latent_attend_mma_launch(a, stream);
     auto kernel = a.cache_f32 ? latent_attend_kernel<float> : latent_attend_kernel<uint16_t>;
     return launch_chained(kernel, dim3(a.splits, a.s.heads, a.m), dim3(kAttendThreads), a.s.row() * 4u, a.pdl, stream, a);
 }
@@ -306,7 +335,8 @@ stark_b200_status latent_value_launch(const LatentArgs &a, cudaStream_t stream) 
     if (stark_b200_status st = check_args(a)) return st;
     if (!a.partials || !a.out) return STARK_B200_INVALID_ARGUMENT;
     auto kernel = a.out_b16 ? latent_value_kernel<uint16_t> : latent_value_kernel<float>;
-    return launch_chained(kernel, dim3(a.s.heads * (a.s.vdim_p / 64u), a.m), dim3(256), a.s.rank_p * 4u, a.pdl, stream, a);
+    return launch_chained(kernel, dim3(a.s.heads * (a.s.vdim_p / 64u), a.m), dim3(256),
+                          a.s.rank_p * 4u + std::max(a.s.rank_p * 4u, 4096u), a.pdl, stream, a);
 }
 
 stark_b200_status latent_rotate_append_launch(const LatentArgs &a, cudaStream_t stream) {

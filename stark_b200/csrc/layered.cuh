@@ -105,7 +105,7 @@ stark_b200_status norm_gather_rows_launch(const float *x, const uint32_t *rows, 
 stark_b200_status clamped_gate_rows_launch(const float *gu, float *act, uint32_t m, uint32_t ff_padded, float limit,
                                            cudaStream_t stream);
 
-// ---- latent attention (latent_attention.cu, latent_attention_tc.cu) -----------------------------------------------
+// ---- latent attention (latent_attention.cu, latent_attend_mma.cu, latent_attention_tc.cu) -----------------------
 // Cache of one layer: pages of kPageTokens rows of [latent, padded | rotated key part, padded], bf16 or f32.
 struct LatentShape {
     uint32_t heads, dim, rot_dim, vdim, rank;       // true sizes
@@ -155,6 +155,10 @@ bool latent_shape_supported(const LatentShape &s);
 stark_b200_status latent_query_launch(const LatentArgs &a, cudaStream_t stream);
 stark_b200_status latent_attend_launch(const LatentArgs &a, cudaStream_t stream);
 stark_b200_status latent_value_launch(const LatentArgs &a, cudaStream_t stream);
+// latent_attend on the tensor cores over a bf16 cache (latent_attend_mma.cu): what latent_attend_launch calls when the
+// shape allows it.
+bool latent_attend_mma_supports(const LatentShape &s);
+stark_b200_status latent_attend_mma_launch(const LatentArgs &a, cudaStream_t stream);
 // The expanded form for prompt passes: new rows into the cache and the queries' rotation in place (bf16 rows), keys and
 // values of every visible row by one contraction, causal attention on the tensor cores.
 bool latent_prefill_tc_supports(const LatentShape &s);
