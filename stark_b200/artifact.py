@@ -211,7 +211,10 @@ def layered_config(root: dict) -> dict:
     bigram = emb.get("bigram")
     return dict(architecture=root["architecture"], vocab=int(root["vocab"]), width=int(root["width"]),
                 eps=float(root["norm"]["eps"]), embed_scale=float(emb.get("scale", 1.0)),
-                bigram=None if bigram is None else {k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")},
+                # the hash is taken modulo the bucket count, so its factors may be
+                bigram=None if bigram is None else dict(buckets=int(bigram["buckets"]),
+                                                        mul_prev=int(bigram["mul_prev"]) % int(bigram["buckets"]),
+                                                        mul_cur=int(bigram["mul_cur"]) % int(bigram["buckets"])),
                 layers=layers)
 
 

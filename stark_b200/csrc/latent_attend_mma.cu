@@ -9,8 +9,9 @@
 //               fragments in registers as bf16 hi + lo, the partial score tiles are added in shared memory
 //   softmax     f32, running maximum and sum per head across the span's pages; weights as bf16 hi + lo
 //   latents     the columns of the weighted sum are divided among the warps, accumulators stay in registers
-// so scores and weights keep f32 accuracy against the bf16 cache.  The span's (maximum, sum, weighted latents) go to the
-// partials the value kernel merges.  Every wait is bounded; a wait that runs out sets the error word.
+// so scores and weights keep f32 accuracy against the bf16 cache.  Up to eight spans' CTAs form a cluster and merge their
+// (maximum, sum, weighted latents) through distributed shared memory, each taking a share of the columns; what is left for
+// the value kernel to merge is one partial per cluster.  Every wait is bounded; a wait that runs out sets the error word.
 #include <cuda.h>
 
 #include "layered.cuh"
@@ -25,6 +26,7 @@ constexpr uint32_t kWarps = 8, kThreads = kWarps * 32u, kHeads = 16;
 constexpr uint32_t kBox = kPageTokens * 128u;      // 64 keys x 64 columns bf16
 constexpr uint32_t kMaxSteps = 6;                  // 16-wide score steps per warp: rows up to 768 values
 constexpr uint32_t kMaxBlocks = 2;                 // 64-wide latent blocks per warp
+constexpr uint32_t kMaxCluster = 8;
 constexpr uint32_t kScorePitch = 68, kWeightPitch = 72;
 constexpr uint32_t kScoreBytes = kWarps * kHeads * kScorePitch * 4u, kWeightBytes = 2u * kHeads * kWeightPitch * 2u;
 
@@ -51,17 +53,39 @@ __device__ inline void split(float x, float y, uint32_t &hi, uint32_t &lo) {
     lo = f32x2_to_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 
+__device__ inline void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// The address of a shared-memory word of this CTA in another CTA of the cluster.
+__device__ inline uint32_t peer_smem(const void *p, uint32_t rank) {
+    uint32_t a;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(smem_u32(p)), "r"(rank));
+    return a;
+}
+__device__ inline float peer_load(uint32_t addr) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+    return v;
+}
+__device__ inline float4 peer_load4(uint32_t addr) {
+    float4 v;
+    asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
+    return v;
+}
+
 struct AttendParams {
     const float *queries;
     float *partials;
     const int32_t *block_table;
     const StepState *state;
-    uint32_t first_pos, heads, splits, latent_blocks, blocks;  // blocks of 64 columns: of the latent, of the whole row
+    uint32_t first_pos, heads, latent_blocks, blocks;  // blocks of 64 columns: of the latent, of the whole row
+    uint32_t splits, cluster;                          // partials a head leaves; CTAs (spans) merged into each
     uint32_t tiles;                                            // page tiles in flight: 1 or 2
     uint32_t *error_word;
 };
 
-// blockIdx: (span, group of 16 heads, row)
+// blockIdx: (span, group of 16 heads, row); BLOCKS: 64-wide latent blocks per warp
+template <uint32_t BLOCKS>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_attend_mma_kernel(const __grid_constant__ CUtensorMap map, const AttendParams p) {
     extern __shared__ uint8_t attend_tiles[];
@@ -76,7 +100,7 @@ latent_attend_mma_kernel(const __grid_constant__ CUtensorMap map, const AttendPa
     const uint32_t span_i = blockIdx.x, head0 = blockIdx.y * kHeads, row = blockIdx.z;
     // the step state does not change while a token's kernels run, except by its last one
     const uint32_t pos = p.state ? p.state->position : p.first_pos + row;
-    const uint32_t pages = pos / kPageTokens + 1u, span = (pages + p.splits - 1u) / p.splits;
+    const uint32_t pages = pos / kPageTokens + 1u, spans = p.splits * p.cluster, span = (pages + spans - 1u) / spans;
     const uint32_t lo = min(pages, span_i * span), hi = min(pages, lo + span);
 
     if (tid == 0) {
@@ -118,9 +142,9 @@ latent_attend_mma_kernel(const __grid_constant__ CUtensorMap map, const AttendPa
             split(v.x, v.y, q_hi[i][e], q_lo[i][e]);
         }
     }
-    float out[kMaxBlocks][8][4];
+    float out[BLOCKS][8][4];
 #pragma unroll
-    for (uint32_t b = 0; b < kMaxBlocks; ++b)
+    for (uint32_t b = 0; b < BLOCKS; ++b)
 #pragma unroll
         for (uint32_t n = 0; n < 8u; ++n)
 #pragma unroll
@@ -206,7 +230,7 @@ latent_attend_mma_kernel(const __grid_constant__ CUtensorMap map, const AttendPa
         const float k0 = keep[lane >> 2], k1 = keep[(lane >> 2) + 8u];
         if (page != lo) {
 #pragma unroll
-            for (uint32_t b = 0; b < kMaxBlocks; ++b)
+            for (uint32_t b = 0; b < BLOCKS; ++b)
 #pragma unroll
                 for (uint32_t n = 0; n < 8u; ++n) out[b][n][0] *= k0, out[b][n][1] *= k0, out[b][n][2] *= k1, out[b][n][3] *= k1;
         }
@@ -221,7 +245,7 @@ latent_attend_mma_kernel(const __grid_constant__ CUtensorMap map, const AttendPa
             }
             const uint32_t key = ks * 16u + (mi & 1u) * 8u + mr;
 #pragma unroll
-            for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+            for (uint32_t b = 0; b < BLOCKS; ++b) {
                 const uint32_t block = warp + kWarps * b;
                 if (block >= p.latent_blocks) break;
                 const uint32_t line = base + block * kBox + key * 128u;
@@ -243,26 +267,55 @@ latent_attend_mma_kernel(const __grid_constant__ CUtensorMap map, const AttendPa
         abort_flag = 1;
         atomicOr(p.error_word, kErrMbarTimeout);
     }
-    // ---- the span's state; an empty span says so with its maximum and leaves zeros
-    auto partial = [&](uint32_t head) { return p.partials + (((size_t)row * p.heads + head) * p.splits + span_i) * (rank + 4u); };
-    if (tid < kHeads && head0 + tid < p.heads) {
-        float *dst = partial(head0 + tid);
-        dst[0] = run_m[tid];
-        dst[1] = run_l[tid];
-    }
+    // ---- merge within the cluster: this span's weighted latents and statistics into shared memory (the page tiles are
+    // free), then every CTA forms its share of the columns over the cluster's spans
+    float *state = reinterpret_cast<float *>(tile);  // [head][rank]
 #pragma unroll
-    for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+    for (uint32_t b = 0; b < BLOCKS; ++b) {
         const uint32_t block = warp + kWarps * b;
         if (block >= p.latent_blocks) break;
 #pragma unroll
         for (uint32_t e = 0; e < 2u; ++e) {
-            const uint32_t head = head0 + (lane >> 2) + 8u * e;
-            if (head >= p.heads) continue;
-            float *dst = partial(head) + 4u + block * 64u + (lane & 3u) * 2u;
+            float *dst = state + ((lane >> 2) + 8u * e) * rank + block * 64u + (lane & 3u) * 2u;
 #pragma unroll
             for (uint32_t n = 0; n < 8u; ++n) *reinterpret_cast<float2 *>(dst + n * 8u) = make_float2(out[b][n][2u * e], out[b][n][2u * e + 1u]);
         }
     }
+    if (p.cluster > 1u) cluster_sync();
+    else __syncthreads();
+    const uint32_t me = span_i % p.cluster, split_i = span_i / p.cluster;
+    // thread = (head, quads of this CTA's columns); an empty span's weight is 0 and its latents are zeros
+    const uint32_t h = tid >> 4, head = head0 + h, quads = rank / 4u;
+    float weight[kMaxCluster], top = -INFINITY, sum = 0.0f;
+#pragma unroll
+    for (uint32_t c = 0; c < kMaxCluster; ++c) {
+        weight[c] = c < p.cluster ? peer_load(peer_smem(&run_m[h], c)) : -INFINITY;
+        top = fmaxf(top, weight[c]);
+    }
+#pragma unroll
+    for (uint32_t c = 0; c < kMaxCluster; ++c) {
+        weight[c] = weight[c] == -INFINITY ? 0.0f : exp2f(weight[c] - top);
+        if (c < p.cluster) sum = fmaf(weight[c], peer_load(peer_smem(&run_l[h], c)), sum);
+    }
+    if (head < p.heads) {
+        float *dst = p.partials + (((size_t)row * p.heads + head) * p.splits + split_i) * (rank + 4u);
+        if (me == 0u && (tid & 15u) == 0) {
+            dst[0] = top;  // -infinity: no span of the cluster had a page
+            dst[1] = sum;
+        }
+        for (uint32_t q = me + p.cluster * (tid & 15u); q < quads; q += 16u * p.cluster) {
+            float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+            for (uint32_t c = 0; c < kMaxCluster; ++c) {
+                if (c >= p.cluster) break;
+                const float4 x = peer_load4(peer_smem(state + h * rank + q * 4u, c));
+                v.x = fmaf(weight[c], x.x, v.x), v.y = fmaf(weight[c], x.y, v.y);
+                v.z = fmaf(weight[c], x.z, v.z), v.w = fmaf(weight[c], x.w, v.w);
+            }
+            *reinterpret_cast<float4 *>(dst + 4u + q * 4u) = v;
+        }
+    }
+    if (p.cluster > 1u) cluster_sync();  // nobody leaves while another CTA may read its shared memory
 }
 
 uint32_t attend_smem(const LatentShape &s, uint32_t tiles) {
@@ -277,7 +330,8 @@ bool latent_attend_mma_supports(const LatentShape &s) {
 }
 
 stark_b200_status latent_attend_mma_launch(const LatentArgs &a, cudaStream_t stream) {
-    if (!a.queries || !a.partials || a.cache_f32 || !a.cache || a.m == 0) return STARK_B200_INVALID_ARGUMENT;
+    if (!a.queries || !a.partials || a.cache_f32 || !a.cache || a.m == 0 || a.cluster == 0 || a.cluster > kMaxCluster)
+        return STARK_B200_INVALID_ARGUMENT;
     const LatentShape &s = a.s;
     if (!latent_attend_mma_supports(s)) return STARK_B200_UNSUPPORTED;
     CUtensorMap map;
@@ -287,12 +341,26 @@ stark_b200_status latent_attend_mma_launch(const LatentArgs &a, cudaStream_t str
                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
         return STARK_B200_DEVICE_FAILURE;
-    AttendParams p{a.queries, a.partials, a.block_table, a.state, a.first_pos, s.heads, a.splits, s.rank_p / 64u, s.row() / 64u,
-                   attend_smem(s, 2) <= 220u * 1024u ? 2u : 1u, a.error_word};
-    static SmemOptIn once;
-    if (stark_b200_status st = ensure_dynamic_smem(latent_attend_mma_kernel, 220 * 1024, once)) return st;
-    return launch_chained(latent_attend_mma_kernel, dim3(a.splits, (s.heads + kHeads - 1u) / kHeads, a.m), dim3(kThreads),
-                          attend_smem(s, p.tiles), a.pdl, stream, map, p);
+    AttendParams p{a.queries, a.partials, a.block_table, a.state, a.first_pos, s.heads, s.rank_p / 64u, s.row() / 64u,
+                   a.splits, a.cluster, attend_smem(s, 2) <= 220u * 1024u ? 2u : 1u, a.error_word};
+    auto kernel = s.rank_p <= kWarps * 64u ? latent_attend_mma_kernel<1> : latent_attend_mma_kernel<2>;
+    static SmemOptIn once[2];
+    if (stark_b200_status st = ensure_dynamic_smem(kernel, 220 * 1024, once[s.rank_p <= kWarps * 64u ? 0 : 1])) return st;
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(a.splits * a.cluster, (s.heads + kHeads - 1u) / kHeads, a.m);
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = attend_smem(s, p.tiles);
+    cfg.stream = stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = a.cluster;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = a.pdl ? 2 : 1;
+    SB_CUDA(cudaLaunchKernelEx(&cfg, kernel, map, p));
+    return STARK_B200_OK;
 }
 
 }  // namespace sb

@@ -327,6 +327,7 @@ stark_b200_status latent_attend_launch(const LatentArgs &a, cudaStream_t stream)
     if (stark_b200_status st = check_args(a)) return st;
     if (!a.queries || !a.partials) return STARK_B200_INVALID_ARGUMENT;
     if (!a.cache_f32 && latent_attend_mma_supports(a.s)) return latent_attend_mma_launch(a, stream);
+    if (a.cluster != 1u) return STARK_B200_INVALID_ARGUMENT;
     auto kernel = a.cache_f32 ? latent_attend_kernel<float> : latent_attend_kernel<uint16_t>;
     return launch_chained(kernel, dim3(a.splits, a.s.heads, a.m), dim3(kAttendThreads), a.s.row() * 4u, a.pdl, stream, a);
 }

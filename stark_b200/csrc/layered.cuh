@@ -137,7 +137,7 @@ struct LatentArgs {
     // absorbed form
     float *queries;            // [m, heads, row()] scaled by scale * log2(e)
     float *partials;           // [m, heads, splits, rank_p + 4]
-    uint32_t splits;
+    uint32_t splits, cluster;  // partials per head; spans of the cache merged into each before it is written (1..8)
     // expanded form (prompt passes)
     uint16_t *expanded;        // [pages * 64, heads * (dim_p + vdim_p)]
     void *out;                 // [m, heads * vdim_p] f32, or bf16 (out_b16)

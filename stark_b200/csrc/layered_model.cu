@@ -147,11 +147,18 @@ LayerTensors &tensors_of(LayeredState *L, const Layer &layer) { return L->layers
 // ---- one token ------------------------------------------------------------------------------------------------------
 
 // Spans the cached rows are divided into: about one CTA per SM, a CTA being 16 heads of a row where the tensor cores
-// serve it, else one.
-uint32_t attend_splits(const LatentShape &s, bool f32, uint32_t rows) {
-    const bool grouped = !f32 && latent_attend_mma_supports(s);
-    const uint32_t ctas = (grouped ? (s.heads + 15u) / 16u : s.heads) * rows;
-    return std::max(1u, std::min(kLatentMaxSplits, (grouped ? 148u : 296u) / ctas));
+// serve it (a power of two of spans, eight to a cluster), else one head.
+void divide_cache(LatentArgs &a, uint32_t rows) {
+    a.cluster = 1;
+    if (!a.cache_f32 && latent_attend_mma_supports(a.s)) {
+        const uint32_t ctas = (a.s.heads + 15u) / 16u * rows, most = std::max(1u, std::min(64u, 148u / ctas));
+        uint32_t spans = 1;
+        while (spans * 2u <= most) spans *= 2u;
+        a.cluster = std::min(8u, spans);
+        a.splits = spans / a.cluster;
+    } else {
+        a.splits = std::max(1u, std::min(kLatentMaxSplits, 296u / (a.s.heads * rows)));
+    }
 }
 
 LatentArgs latent_args(Model *m, const Layer &layer) {
@@ -230,7 +237,7 @@ stark_b200_status layered_issue_token(Model *m, bool full, uint32_t *launches) {
         la.qd = L->qd;
         la.state = m->state;
         la.m = 1;
-        la.splits = attend_splits(layer.s, L->f32, 1);
+        divide_cache(la, 1);
         la.out = L->attn;
         la.pdl = pdl;
         SB_TRY(latent_query_launch(la, s));
@@ -357,7 +364,7 @@ stark_b200_status rows_attention(Model *m, const Layer &layer, uint32_t mrows, u
         a.first_pos = first_pos + r;
         a.qd = static_cast<const uint8_t *>(L->rqd) + (size_t)r * a.ld_qd * element;
         a.out = static_cast<uint8_t *>(L->rattn) + (size_t)r * layer.s.heads * layer.s.vdim_p * element;
-        a.splits = attend_splits(layer.s, L->f32, a.m);
+        divide_cache(a, a.m);
         SB_TRY(latent_query_launch(a, m->stream));
         SB_TRY(latent_attend_launch(a, m->stream));
         SB_TRY(latent_value_launch(a, m->stream));
@@ -575,8 +582,13 @@ stark_b200_status build_layers(Model *m, const stark_b200_layer_desc *descs) {
         L->max_ff = std::max(L->max_ff, l.ff_p);
         L->max_expand = std::max(L->max_expand, s.heads * (s.dim_p + s.vdim_p));
         L->query_floats = std::max(L->query_floats, (size_t)kAttendRows * s.heads * s.row());
-        for (uint32_t r = 1; r <= kAttendRows; ++r)
-            L->partial_floats = std::max(L->partial_floats, latent_partial_floats(s, r, attend_splits(s, L->f32, r)));
+        for (uint32_t r = 1; r <= kAttendRows; ++r) {
+            LatentArgs probe{};
+            probe.s = s;
+            probe.cache_f32 = L->f32;
+            divide_cache(probe, r);
+            L->partial_floats = std::max(L->partial_floats, latent_partial_floats(s, r, probe.splits));
+        }
     }
     for (const MatrixB16 probe : {MatrixB16{nullptr, 1, L->width_p}, MatrixB16{nullptr, 1, L->max_attn},
                                   MatrixB16{nullptr, 1, std::max(64u, L->max_ff)}})

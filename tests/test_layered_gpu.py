@@ -244,6 +244,19 @@ def test_read_outs_and_sampling():
     m.close()
 
 
+def test_library_loader_serves_the_same_model(tmp_path):
+    from stark_b200.artifact import write_layered
+    from stark_b200.engine import LayeredModel
+    root = deep()
+    w = L.weights(root, seed=21)
+    write_layered(tmp_path, root, w)
+    ids = L.tokens(root, 90)
+    a, b = LayeredModel.from_artifact(tmp_path, 128), LayeredModel.load_path(tmp_path, 128)
+    assert np.array_equal(feed(a, ids, [40, 50]), feed(b, ids, [40, 50]))
+    a.close()
+    b.close()
+
+
 def greedy_reference(root, w, ids, n):
     o = L.oracle(root, w)
     row = o.feed(ids)[-1]

@@ -71,6 +71,42 @@ def test_weights_of_chain_resolves():
     assert [l["weights_of"] for l in layered_config(root)["layers"]] == [None, 0, 0]
 
 
+def c_load(path) -> int:
+    import ctypes as C
+    from stark_b200 import _lib
+    opts = _lib.LoadOptions(C.sizeof(_lib.LoadOptions), _lib.ABI_VERSION, 64, 0)
+    handle = C.c_void_p()
+    raw = str(path).encode()
+    status = _lib.load().stark_b200_load(raw, len(raw), C.byref(opts), C.byref(handle))
+    if handle.value:
+        _lib.load().stark_b200_destroy(C.byref(handle))
+    return status
+
+
+@pytest.mark.parametrize("spoil,status", [("missing", 1), ("extra", 1), ("shape", 1), ("mixer", 5), ("kind", 5), ("circle", 1),
+                                          ("size", 1), (None, None)])
+def test_library_loader_checks_before_it_touches_a_device(tmp_path, spoil, status):
+    from stark_b200.artifact import write_layered
+    root = small()
+    w = L.weights(root)
+    if spoil == "missing":
+        del w["l1.mix.uk"]
+    elif spoil == "extra":
+        w["l1.norm2"] = w["l1.norm1"]
+    elif spoil == "shape":
+        w["head"] = w["head"][:, :-1].copy()
+    elif spoil == "mixer":
+        root["layers"][0]["type"] = "something_else"
+    elif spoil == "kind":
+        root["layers"][0]["mlp"]["kind"] = "routed"
+    elif spoil == "circle":
+        root["layers"][2]["weights_of"] = 2
+    elif spoil == "size":
+        root["width"] = 80
+    write_layered(tmp_path, root, w)
+    assert c_load(tmp_path) == status if status is not None else c_load(tmp_path) in (0, 8)  # 8: no device here
+
+
 class FakeModel:
     def __init__(self):
         self.calls = []
