@@ -53,7 +53,9 @@ gemm_b16_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
     uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(acc_full + 1);
     volatile uint32_t *abort_flag = tmem_slot + 1;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    const uint32_t n0 = blockIdx.x * kBN, m0 = blockIdx.y * (128u * HALVES);
+    // row tiles are the fast index: a wave of CTAs then shares few weight tiles, so the weights stream from memory once
+    // while the activations of a pass stay in L2
+    const uint32_t n0 = blockIdx.y * kBN, m0 = blockIdx.x * (128u * HALVES);
 
     if (tid == 0) {
         for (uint32_t s = 0; s < T::kDepth; ++s) {
@@ -185,7 +187,7 @@ stark_b200_status launch(const GemmB16Args &a, const CUtensorMap &x_map, const C
                                       : (a.kind == kGemmF32 ? gemm_b16_kernel<HALVES, kGemmF32> : gemm_b16_kernel<HALVES, kGemmGate>);
     static SmemOptIn once[3];
     if (stark_b200_status st = ensure_dynamic_smem(kernel, (int)T::kSmem, once[a.kind])) return st;
-    kernel<<<dim3((a.out_cols + kBN - 1u) / kBN, (a.m + 128u * HALVES - 1u) / (128u * HALVES)), kGemmThreads, T::kSmem, stream>>>(
+    kernel<<<dim3((a.m + 128u * HALVES - 1u) / (128u * HALVES), (a.out_cols + kBN - 1u) / kBN), kGemmThreads, T::kSmem, stream>>>(
         x_map, w_map, p);
     SB_CUDA(cudaGetLastError());
     return STARK_B200_OK;

@@ -9,7 +9,7 @@
 //               fragments in registers as bf16 hi + lo, the partial score tiles are added in shared memory
 //   softmax     f32, running maximum and sum per head across the span's pages; weights as bf16 hi + lo
 //   latents     the columns of the weighted sum are divided among the warps, accumulators stay in registers
-// so scores and weights keep f32 accuracy against the bf16 cache.  Up to eight spans' CTAs form a cluster and merge their
+// so scores and weights keep f32 accuracy against the bf16 cache.  A few spans' CTAs (four unless set otherwise) form a cluster and merge their
 // (maximum, sum, weighted latents) through distributed shared memory, each taking a share of the columns; what is left for
 // the value kernel to merge is one partial per cluster.  Every wait is bounded; a wait that runs out sets the error word.
 #include <cuda.h>

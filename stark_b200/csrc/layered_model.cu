@@ -147,14 +147,15 @@ LayerTensors &tensors_of(LayeredState *L, const Layer &layer) { return L->layers
 // ---- one token ------------------------------------------------------------------------------------------------------
 
 // Spans the cached rows are divided into: about one CTA per SM, a CTA being 16 heads of a row where the tensor cores
-// serve it (a power of two of spans, eight to a cluster), else one head.
+// serve it (a power of two of spans, a few to a cluster), else one head.
 void divide_cache(LatentArgs &a, uint32_t rows) {
     a.cluster = 1;
     if (!a.cache_f32 && latent_attend_mma_supports(a.s)) {
         const uint32_t ctas = (a.s.heads + 15u) / 16u * rows, most = std::max(1u, std::min(64u, 148u / ctas));
         uint32_t spans = 1;
         while (spans * 2u <= most) spans *= 2u;
-        a.cluster = std::min(8u, spans);
+        if (tunables().latent_spans) spans = std::min(spans, tunables().latent_spans);
+        a.cluster = std::min(tunables().latent_cluster, spans);
         a.splits = spans / a.cluster;
     } else {
         a.splits = std::max(1u, std::min(kLatentMaxSplits, 296u / (a.s.heads * rows)));
@@ -587,7 +588,7 @@ stark_b200_status build_layers(Model *m, const stark_b200_layer_desc *descs) {
             probe.s = s;
             probe.cache_f32 = L->f32;
             divide_cache(probe, r);
-            L->partial_floats = std::max(L->partial_floats, latent_partial_floats(s, r, probe.splits));
+            L->partial_floats = std::max(L->partial_floats, latent_partial_floats(s, r, probe.splits * probe.cluster));
         }
     }
     for (const MatrixB16 probe : {MatrixB16{nullptr, 1, L->width_p}, MatrixB16{nullptr, 1, L->max_attn},

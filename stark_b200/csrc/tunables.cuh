@@ -27,6 +27,8 @@ struct Tunables {
     uint32_t tp_rows_push;        // STARK_B200_TP_ROWS_PUSH     a prompt pass's contractions store their tiles to the other ranks themselves: 1 always, 2 between two ranks only, 0 never (a copy kernel after each)
     uint32_t rows_attention;      // STARK_B200_ROWS_ATTENTION   1: a handful of rows attend in the keys-as-rows form, 0: in 16-row tiles
     uint32_t rows_matvec;         // STARK_B200_ROWS_MATVEC      1: up to 8 rows go through the several-rows matvec, 0: through the tensor-core tile kernels
+    uint32_t latent_spans;        // STARK_B200_LATENT_SPANS     spans of the latent cache a decode step attends to in parallel (0 = chosen from the head count, at most 64)
+    uint32_t latent_cluster;      // STARK_B200_LATENT_CLUSTER   spans merged through distributed shared memory (1, 2, 4 or 8)
 };
 
 Tunables &tunables();
