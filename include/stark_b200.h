@@ -646,13 +646,15 @@ stark_b200_status stark_b200_moe_model_destroy(stark_b200_moe_model **model);
 
 /* ------------------------------------------------------------------------------------------
  * Layered decoders: a model whose configuration lists every layer's mixer and feed-forward with sizes of their own
- * (Guvulorn), over bf16 weights.  Nothing in the reference corresponds to it.  Built empty from its description,
+ * (Guvulorn, Pomelix), over bf16 weights.  Nothing in the reference corresponds to it.  Built empty from its description,
  * filled tensor by tensor, finalized; from then on the handle is an ordinary stark_b200_model: prefill, prefill_rows,
  * step, read-outs, sample, generate_greedy, rewind, reset, get_info, destroy.
  */
 #define STARK_B200_MIXER_LATENT 1u     /* attention over a cached latent and a shared rotated key part */
+#define STARK_B200_MIXER_GROUPED 2u    /* grouped-query attention: short convolutions, unit queries and keys, query temperature, value mixing */
 #define STARK_B200_FF_NONE 0u
 #define STARK_B200_FF_CLAMPED_GATE 1u  /* min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1), with biases */
+#define STARK_B200_FF_SILU_GATE 2u     /* silu(g) * u, no biases */
 #define STARK_B200_ROT_PLAIN 0u
 #define STARK_B200_ROT_YARN 1u         /* frequencies blended with themselves / factor between two pair indices */
 typedef struct stark_b200_layer_desc {
@@ -662,9 +664,9 @@ typedef struct stark_b200_layer_desc {
     uint32_t weights_of;  /* UINT32_MAX: tensors of its own; otherwise the layer whose tensors it uses (cache of its own) */
     uint32_t heads;
     uint32_t dim;      /* unrotated query / key entries per head */
-    uint32_t rot_dim;  /* rotated query / key entries per head */
+    uint32_t rot_dim;  /* rotated query / key entries per head (STARK_B200_MIXER_LATENT; 0 otherwise) */
     uint32_t vdim;     /* value entries per head */
-    uint32_t kv_rank;  /* latent entries */
+    uint32_t kv_rank;  /* latent entries (STARK_B200_MIXER_LATENT; 0 otherwise) */
     uint32_t ff_width;
     float scale;       /* on the scores */
     float ff_limit;
@@ -672,7 +674,20 @@ typedef struct stark_b200_layer_desc {
     uint32_t rot_scaling;
     double rot_base;
     double rot_factor, rot_original, rot_fast, rot_slow; /* STARK_B200_ROT_YARN */
+    /* STARK_B200_MIXER_GROUPED */
+    uint32_t kv_heads;     /* key / value heads; query head h uses h / (heads / kv_heads) */
+    uint32_t conv_taps;    /* taps of the causal convolution over time on queries, keys and values (0: none) */
+    uint32_t q_temp_every; /* queries times 1 + q_temp_coef * ln((position + 1) / q_temp_every + 1), whole division */
+    float q_temp_coef;
+    uint32_t v_mix;        /* values mixed with the values of the first layer that has this set */
+    uint32_t reserved;
 } stark_b200_layer_desc;
+/* How a layer's sublayers meet the residual stream x. */
+#define STARK_B200_ARRANGE_POST_NORM 0u /* x += norm1(mixer(x)), then x += norm2(ff(x)) */
+#define STARK_B200_ARRANGE_PARALLEL 1u  /* h = norm1(x); x += residual_mult * (scale1 * mixer(h) + scale2 * ff(h)) */
+#define STARK_B200_LAYERED_NORM_AROUND_ZERO 1u /* residual-stream norms multiply by 1 + w instead of w */
+#define STARK_B200_LAYERED_HAS_EMBED_NORM 2u   /* a norm behind the embedding */
+#define STARK_B200_LAYERED_TIED_HEAD 4u        /* logits from the embedding table; no head tensor */
 typedef struct stark_b200_layered_config {
     uint32_t struct_size;
     uint32_t abi_version;
@@ -685,6 +700,10 @@ typedef struct stark_b200_layered_config {
     uint64_t bigram_mul_prev, bigram_mul_cur;
     float embed_scale;
     float eps;
+    uint32_t arrangement;    /* STARK_B200_ARRANGE_* */
+    uint32_t flags;          /* STARK_B200_LAYERED_NORM_AROUND_ZERO | ... */
+    float residual_mult;     /* STARK_B200_ARRANGE_PARALLEL */
+    uint32_t reserved;
 } stark_b200_layered_config;
 /* Which tensor a set call addresses; all bf16, row-major [rows, columns] (vectors: rows = 1), in the model's own
  * layout -- the library pads and fuses. */
@@ -707,6 +726,14 @@ typedef struct stark_b200_layered_config {
 #define STARK_B200_LAYERED_UP_BIAS 16u
 #define STARK_B200_LAYERED_DOWN 17u      /* [width, ff_width] */
 #define STARK_B200_LAYERED_DOWN_BIAS 18u
+#define STARK_B200_LAYERED_K 19u         /* [kv_heads * dim, width] */
+#define STARK_B200_LAYERED_V 20u         /* [kv_heads * vdim, width] */
+#define STARK_B200_LAYERED_Q_CONV 21u    /* [heads * dim, conv_taps]; the last column weighs the current row */
+#define STARK_B200_LAYERED_K_CONV 22u    /* [kv_heads * dim, conv_taps] */
+#define STARK_B200_LAYERED_V_CONV 23u    /* [kv_heads * vdim, conv_taps] */
+#define STARK_B200_LAYERED_V_SHARE 24u   /* [1]: share of the first mixing layer's values */
+#define STARK_B200_LAYERED_SCALE1 25u    /* [width]: on the mixer's output */
+#define STARK_B200_LAYERED_SCALE2 26u    /* [width]: on the feed-forward's output */
 stark_b200_status stark_b200_layered_create(const stark_b200_layered_config *config, const stark_b200_layer_desc *layers,
                                             stark_b200_model **out_model);
 stark_b200_status stark_b200_layered_set_tensor(stark_b200_model *model, uint32_t layer, uint32_t which,

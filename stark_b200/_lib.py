@@ -59,22 +59,28 @@ class LayerDesc(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("struct_size", "mixer", "feed_forward", "weights_of", "heads", "dim", "rot_dim",
                                           "vdim", "kv_rank", "ff_width")] + [
         ("scale", C.c_float), ("ff_limit", C.c_float), ("rot_dims", C.c_uint32), ("rot_scaling", C.c_uint32)] + [
-        (n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
+        (n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")] + [
+        ("kv_heads", C.c_uint32), ("conv_taps", C.c_uint32), ("q_temp_every", C.c_uint32), ("q_temp_coef", C.c_float),
+        ("v_mix", C.c_uint32), ("reserved", C.c_uint32)]
 
 
 class LayeredConfig(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("struct_size", "abi_version", "vocab", "width", "layers", "context_tokens",
                                           "compute", "bigram_buckets")] + [
-        ("bigram_mul_prev", C.c_uint64), ("bigram_mul_cur", C.c_uint64), ("embed_scale", C.c_float), ("eps", C.c_float)]
+        ("bigram_mul_prev", C.c_uint64), ("bigram_mul_cur", C.c_uint64), ("embed_scale", C.c_float), ("eps", C.c_float),
+        ("arrangement", C.c_uint32), ("flags", C.c_uint32), ("residual_mult", C.c_float), ("reserved", C.c_uint32)]
 
 
-MIXER_LATENT = 1
-FF_NONE, FF_CLAMPED_GATE = 0, 1
+MIXER_LATENT, MIXER_GROUPED = 1, 2
+FF_NONE, FF_CLAMPED_GATE, FF_SILU_GATE = 0, 1, 2
+ARRANGE_POST_NORM, ARRANGE_PARALLEL = 0, 1
+LAYERED_NORM_AROUND_ZERO, LAYERED_HAS_EMBED_NORM, LAYERED_TIED_HEAD = 1, 2, 4
 ROT_PLAIN, ROT_YARN = 0, 1
 NO_LAYER = 0xFFFFFFFF
 (LAYERED_EMBED, LAYERED_BIGRAM, LAYERED_EMBED_NORM, LAYERED_FINAL_NORM, LAYERED_HEAD, LAYERED_NORM1, LAYERED_Q, LAYERED_DKV,
  LAYERED_DKV_NORM, LAYERED_UK, LAYERED_UV, LAYERED_O, LAYERED_NORM2, LAYERED_GATE, LAYERED_GATE_BIAS, LAYERED_UP,
- LAYERED_UP_BIAS, LAYERED_DOWN, LAYERED_DOWN_BIAS) = range(19)
+ LAYERED_UP_BIAS, LAYERED_DOWN, LAYERED_DOWN_BIAS, LAYERED_K, LAYERED_V, LAYERED_Q_CONV, LAYERED_K_CONV, LAYERED_V_CONV,
+ LAYERED_V_SHARE, LAYERED_SCALE1, LAYERED_SCALE2) = range(27)
 
 MOE_MAT_QKV, MOE_MAT_O, MOE_MAT_GATE_UP, MOE_MAT_DOWN, MOE_MAT_OUTPUT = range(5)
 (MOE_ATTN_NORM, MOE_FFN_NORM, MOE_Q_NORM, MOE_K_NORM, MOE_FINAL_NORM, MOE_ROUTER, MOE_TOKEN_TABLE) = range(7)

@@ -175,31 +175,57 @@ def read_artifact(directory) -> tuple[dict, dict]:
 
 # ----------------------------------------------------------------------------- layered decoders
 
-LAYERED_ARCHITECTURES = ("Guvulorn",)
+# What a layered architecture fixes for all of its models; sizes, constants and the order of layers are config.json's.
+#   arrangement   how a layer's sublayers meet the residual stream: "post_norm" (each sublayer's output is normed and added in
+#                 turn), "parallel" (both sublayers read one normed row, their scaled outputs are added together)
+#   mixer         prefix or name of a layer entry's type -> the mixer that serves it
+LAYERED_ARCHITECTURES = {
+    "Guvulorn": dict(arrangement="post_norm", mixer="latent", mixer_type="latent_attention", any_suffix=True,
+                     feed_forward="clamped_gate", norm_around_zero=True, embed_norm=True, tied=False),
+    "Pomelix": dict(arrangement="parallel", mixer="grouped", mixer_type="attention", any_suffix=False,
+                    feed_forward="silu_gate", norm_around_zero=False, embed_norm=False, tied=True),
+}
+
+
+def _latent_mixer(m: dict) -> dict:
+    rot = m.get("rot")
+    scaling = rot.get("scaling")
+    return dict(mixer="latent", heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+                rot=dict(base=float(rot["base"]), dims=int(rot.get("dims", m["rot_dim"])),
+                         scaling=None if scaling is None else {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}))
+
+
+def _grouped_mixer(m: dict) -> dict:
+    temp = m.get("q_temp")
+    out = dict(mixer="grouped", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+               scale=float(m["scale"]), conv=int(m.get("conv") or 0), v_mix=bool(m.get("v_mix")),
+               q_temp=None if temp is None else dict(coef=float(temp["coef"]), every=int(temp["every"])))
+    if out["kv_heads"] < 1 or out["heads"] % out["kv_heads"] or (out["q_temp"] and out["q_temp"]["every"] < 1):
+        raise ArtifactError("heads must be a multiple of kv_heads, and q_temp.every at least 1")
+    return out
 
 
 def layered_config(root: dict) -> dict:
     """The engine's description of a layered decoder from its ``config.json``: model-wide sizes and constants, and per
-    layer the latent attention's sizes, its rotation, the feed-forward and whose tensors it uses."""
-    if root.get("architecture") not in LAYERED_ARCHITECTURES:
+    layer the mixer's sizes and constants, the feed-forward and whose tensors it uses."""
+    fixed = LAYERED_ARCHITECTURES.get(root.get("architecture"))
+    if fixed is None:
         raise ArtifactError(f"architecture {root.get('architecture')} is not a layered decoder this engine knows")
     layers = []
     for i, entry in enumerate(root["layers"]):
-        if not str(entry["type"]).startswith("latent_attention"):
-            raise ArtifactError(f"layer {i}: mixer {entry['type']} is not implemented")
-        m, mlp, rot = entry["mixer"], entry.get("mlp"), entry["mixer"].get("rot")
-        ff = None
+        kind = str(entry["type"])
+        if not (kind.startswith(fixed["mixer_type"]) if fixed["any_suffix"] else kind == fixed["mixer_type"]):
+            raise ArtifactError(f"layer {i}: mixer {kind} is not implemented")
+        mlp, ff = entry.get("mlp"), None
         if mlp is not None:
             if mlp["kind"] != "dense":
                 raise ArtifactError(f"layer {i}: feed-forward {mlp['kind']} is not implemented")
-            ff = dict(width=int(mlp["ff"]), limit=float(mlp["limit"]))
-        scaling = rot.get("scaling")
-        layers.append(dict(
-            heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
-            kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), ff=ff,
-            rot=dict(base=float(rot["base"]), dims=int(rot.get("dims", m["rot_dim"])),
-                     scaling=None if scaling is None else {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}),
-            weights_of=None if entry.get("weights_of") is None else int(entry["weights_of"])))
+            ff = dict(kind=fixed["feed_forward"], width=int(mlp["ff"]))
+            if ff["kind"] == "clamped_gate":
+                ff["limit"] = float(mlp["limit"])
+        mixer = (_latent_mixer if fixed["mixer"] == "latent" else _grouped_mixer)(entry["mixer"])
+        layers.append(dict(mixer, ff=ff, weights_of=None if entry.get("weights_of") is None else int(entry["weights_of"])))
     for i, layer in enumerate(layers):  # a layer that points to one without tensors of its own means that one's source
         seen = {i}
         while layer["weights_of"] is not None and layers[layer["weights_of"]]["weights_of"] is not None:
@@ -207,10 +233,12 @@ def layered_config(root: dict) -> dict:
             if layer["weights_of"] in seen:
                 raise ArtifactError(f"layer {i}: circular weights_of")
             seen.add(layer["weights_of"])
-    emb = root["embedding"]
+    emb = root.get("embedding") or {}
     bigram = emb.get("bigram")
     return dict(architecture=root["architecture"], vocab=int(root["vocab"]), width=int(root["width"]),
                 eps=float(root["norm"]["eps"]), embed_scale=float(emb.get("scale", 1.0)),
+                residual_mult=float(root["residual_mult"]) if fixed["arrangement"] == "parallel" else 1.0,
+                **{k: fixed[k] for k in ("arrangement", "norm_around_zero", "embed_norm", "tied")},
                 # the hash is taken modulo the bucket count, so its factors may be
                 bigram=None if bigram is None else dict(buckets=int(bigram["buckets"]),
                                                         mul_prev=int(bigram["mul_prev"]) % int(bigram["buckets"]),
@@ -218,28 +246,53 @@ def layered_config(root: dict) -> dict:
                 layers=layers)
 
 
+def _mixer_tensors(p: str, i: int, l: dict, D: int) -> list[tuple]:
+    from . import _lib as L
+    H, dim, vd = l["heads"], l["dim"], l["vdim"]
+    if l["mixer"] == "latent":
+        rd, rank = l["rot_dim"], l["kv_rank"]
+        return [(p + ".mix.q", i, L.LAYERED_Q, (H * (dim + rd), D)), (p + ".mix.dkv", i, L.LAYERED_DKV, (rank + rd, D)),
+                (p + ".mix.dkv.norm", i, L.LAYERED_DKV_NORM, (rank,)), (p + ".mix.uk", i, L.LAYERED_UK, (H * dim, rank)),
+                (p + ".mix.uv", i, L.LAYERED_UV, (H * vd, rank)), (p + ".mix.o", i, L.LAYERED_O, (D, H * vd))]
+    G, taps = l["kv_heads"], l["conv"]
+    out = [(p + ".mix.q", i, L.LAYERED_Q, (H * dim, D)), (p + ".mix.k", i, L.LAYERED_K, (G * dim, D)),
+           (p + ".mix.v", i, L.LAYERED_V, (G * vd, D)), (p + ".mix.o", i, L.LAYERED_O, (D, H * vd))]
+    if taps:
+        out += [(p + ".mix.q.conv", i, L.LAYERED_Q_CONV, (H * dim, taps)), (p + ".mix.k.conv", i, L.LAYERED_K_CONV, (G * dim, taps)),
+                (p + ".mix.v.conv", i, L.LAYERED_V_CONV, (G * vd, taps))]
+    if l["v_mix"]:
+        out.append((p + ".mix.vmix", i, L.LAYERED_V_SHARE, ()))
+    return out
+
+
 def layered_tensors(cfg: dict) -> list[tuple]:
     """Every tensor of a layered decoder: (name in the file, layer, id of the set call, shape)."""
     from . import _lib as L
     D, V = cfg["width"], cfg["vocab"]
-    out = [("embed", 0, L.LAYERED_EMBED, (V, D)), ("embed.norm", 0, L.LAYERED_EMBED_NORM, (D,)),
-           ("final.norm", 0, L.LAYERED_FINAL_NORM, (D,)), ("head", 0, L.LAYERED_HEAD, (V, D))]
+    out = [("embed", 0, L.LAYERED_EMBED, (V, D)), ("final.norm", 0, L.LAYERED_FINAL_NORM, (D,))]
+    if cfg["embed_norm"]:
+        out.append(("embed.norm", 0, L.LAYERED_EMBED_NORM, (D,)))
+    if not cfg["tied"]:
+        out.append(("head", 0, L.LAYERED_HEAD, (V, D)))
     if cfg["bigram"] is not None:
         out.append(("bigram", 0, L.LAYERED_BIGRAM, (cfg["bigram"]["buckets"] + 1, D)))
+    parallel = cfg["arrangement"] == "parallel"
     for i, l in enumerate(cfg["layers"]):
         if l["weights_of"] is not None:
             continue
-        p, H, dim, rd, vd, rank = f"l{i}", l["heads"], l["dim"], l["rot_dim"], l["vdim"], l["kv_rank"]
-        out += [(p + ".norm1", i, L.LAYERED_NORM1, (D,)), (p + ".mix.q", i, L.LAYERED_Q, (H * (dim + rd), D)),
-                (p + ".mix.dkv", i, L.LAYERED_DKV, (rank + rd, D)), (p + ".mix.dkv.norm", i, L.LAYERED_DKV_NORM, (rank,)),
-                (p + ".mix.uk", i, L.LAYERED_UK, (H * dim, rank)), (p + ".mix.uv", i, L.LAYERED_UV, (H * vd, rank)),
-                (p + ".mix.o", i, L.LAYERED_O, (D, H * vd))]
-        if l["ff"] is not None:
-            F = l["ff"]["width"]
-            out += [(p + ".norm2", i, L.LAYERED_NORM2, (D,)),
-                    (p + ".mlp.gate", i, L.LAYERED_GATE, (F, D)), (p + ".mlp.gate.b", i, L.LAYERED_GATE_BIAS, (F,)),
-                    (p + ".mlp.up", i, L.LAYERED_UP, (F, D)), (p + ".mlp.up.b", i, L.LAYERED_UP_BIAS, (F,)),
-                    (p + ".mlp.down", i, L.LAYERED_DOWN, (D, F)), (p + ".mlp.down.b", i, L.LAYERED_DOWN_BIAS, (D,))]
+        p = f"l{i}"
+        out += [(p + ".norm1", i, L.LAYERED_NORM1, (D,))] + _mixer_tensors(p, i, l, D)
+        if parallel:
+            out.append((p + ".ls1", i, L.LAYERED_SCALE1, (D,)))
+        if l["ff"] is None:
+            continue
+        F = l["ff"]["width"]
+        out.append((p + ".ls2", i, L.LAYERED_SCALE2, (D,)) if parallel else (p + ".norm2", i, L.LAYERED_NORM2, (D,)))
+        out += [(p + ".mlp.gate", i, L.LAYERED_GATE, (F, D)), (p + ".mlp.up", i, L.LAYERED_UP, (F, D)),
+                (p + ".mlp.down", i, L.LAYERED_DOWN, (D, F))]
+        if l["ff"]["kind"] == "clamped_gate":
+            out += [(p + ".mlp.gate.b", i, L.LAYERED_GATE_BIAS, (F,)), (p + ".mlp.up.b", i, L.LAYERED_UP_BIAS, (F,)),
+                    (p + ".mlp.down.b", i, L.LAYERED_DOWN_BIAS, (D,))]
     return out
 
 
@@ -254,7 +307,8 @@ def read_layered(directory) -> tuple[dict, dict]:
     header, _, data = _read_safetensors(directory / "model.safetensors")
     used: set = set()
     weights = {name: _tensor(header, data, name, "BF16", shape, used) for name, _, _, shape in layered_tensors(cfg)}
-    extra = set(header) - used
+    # a mixing share in a layer that does not mix is as unused as the first mixing layer's
+    extra = set(header) - used - {f"l{i}.mix.vmix" for i, l in enumerate(cfg["layers"]) if l["mixer"] == "grouped" and not l["v_mix"]}
     if extra:
         raise ArtifactError(f"artifact has {len(extra)} tensors the decoder does not use, e.g. {sorted(extra)[0]}")
     return cfg, weights

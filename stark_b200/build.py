@@ -21,8 +21,9 @@ LIB = PKG / "libstark_b200.so"
 PARTS = {
     "layered": (PKG / "libstark_b200_layered.so",
                 ("abi_core", "abi_session", "token_loop", "layered_model", "layered_rows", "dense_b16", "gemm_b16",
-                 "latent_attention", "latent_attend_mma",
-                 "latent_attention_tc", "ops", "sampling", "tunables")),
+                 "span_attend",
+                 "latent_attention", "latent_attend_mma", "grouped_attention", "grouped_attend_mma",
+                 "layered_attention_tc", "ops", "sampling", "tunables")),
 }
 
 NVCC_FLAGS = [

@@ -5,8 +5,10 @@
 // in flight.  The first batch of loads is issued before the wait on the previous kernel: weights depend on nothing.
 // The input row stays f32 throughout (a bf16 weight times an f32 activation, f32 accumulation), so the one-row path has
 // no rounding of activations at all and serves the 32-bit mode unchanged.
-// The input row is formed by every CTA in its prologue: plain, or the residual add of a normed sublayer output, or that
-// followed by the model's last norm.
+// The input row is formed by every CTA in its prologue: plain, its norm, or the residual add of a normed sublayer output,
+// or that followed by the model's last norm.  Rows in front of gated ones may be stored plainly (one pass over the row for
+// a mixer's projections and a feed-forward's gate and up halves), and two contractions that end in the same residual add
+// may share a launch, their inputs and weights side by side (kRowResidual).
 #include "layered.cuh"
 #include "layered_math.cuh"
 
@@ -38,18 +40,22 @@ __device__ inline void fma8(float &acc, const uint4 &w, const float4 &a, const f
 
 struct MatvecParams {
     const uint16_t *w;
-    uint32_t rows, cols;
+    uint32_t rows, cols;  // rows of w are cols apart
     const float *x, *y, *norm_w, *last_w;
     float *x_out;
     uint32_t width;
     float eps;
     const float *bias;
-    float limit;
+    Gate gate;
     float *out;
     uint32_t out_rows;
     float *partial_max;
     uint32_t *partial_index;
-    uint32_t pairs;  // row pairs
+    uint32_t pairs;         // row pairs
+    uint32_t stored_pairs;  // kRowGate: pairs of neighbours in front of the gated pairs
+    float *stored_out;
+    const float *residual, *scale_a, *scale_b;
+    uint32_t split_col;
 };
 
 template <uint32_t PRO, uint32_t EPI>
@@ -64,18 +70,23 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
     uint32_t pair = blockIdx.x * kWarps + warp;
 
     // rows of a pair: gate and up 16 apart, or neighbours
-    auto row0 = [&](uint32_t pr) { return EPI == kRowGate ? (pr >> 4) * 32u + (pr & 15u) : 2u * pr; };
-    constexpr uint32_t kApart = EPI == kRowGate ? 16u : 1u;
+    auto is_gate = [&](uint32_t pr) { return EPI == kRowGate && pr >= p.stored_pairs; };
+    auto row0 = [&](uint32_t pr) {
+        if (!is_gate(pr)) return 2u * pr;
+        const uint32_t unit = pr - p.stored_pairs;
+        return 2u * p.stored_pairs + (unit >> 4) * 32u + (unit & 15u);
+    };
+    auto apart = [&](uint32_t pr) { return is_gate(pr) ? 16u : 1u; };
     uint4 buf[2][kUnroll][2];
     auto fetch = [&](uint4 (&b)[kUnroll][2], uint32_t pr, uint32_t chunk) {
-        const uint32_t r = row0(pr);
+        const uint32_t r = row0(pr), step = apart(pr);
 #pragma unroll
         for (uint32_t u = 0; u < kUnroll; ++u) {
             const uint32_t col = (chunk + u) * kChunk + lane * 8u;
             const bool in = pr < p.pairs && col < p.cols;
 #pragma unroll
             for (uint32_t j = 0; j < 2u; ++j) {
-                const uint32_t rr = r + j * kApart;
+                const uint32_t rr = r + j * step;
                 b[u][j] = in && rr < p.rows ? ldg_nc_v4(p.w + (size_t)rr * p.cols + col) : make_uint4(0u, 0u, 0u, 0u);
             }
         }
@@ -91,6 +102,20 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
             const float4 v = i < p.cols ? *reinterpret_cast<const float4 *>(p.x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
             *reinterpret_cast<float4 *>(xs + spread(i)) = v;
         }
+    } else if (PRO == kRowNorm) {
+        float s = 0.0f;
+        for (uint32_t i = threadIdx.x * 4u; i < padded; i += kThreads * 4u) {
+            const float4 v = i < p.cols ? *reinterpret_cast<const float4 *>(p.x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+            *reinterpret_cast<float4 *>(xs + spread(i)) = v;
+        }
+        const float inv = inverse_rms(block_sum(s, scratch), p.width, p.eps);
+        for (uint32_t i = threadIdx.x * 4u; i < p.cols; i += kThreads * 4u) {  // each thread its own elements
+            float4 v = *reinterpret_cast<float4 *>(xs + spread(i));
+            const float4 g = *reinterpret_cast<const float4 *>(p.norm_w + i);
+            v.x *= inv * g.x, v.y *= inv * g.y, v.z *= inv * g.z, v.w *= inv * g.w;
+            *reinterpret_cast<float4 *>(xs + spread(i)) = v;
+        }
     } else {
         float s = 0.0f;
         for (uint32_t i = threadIdx.x * 4u; i < padded; i += kThreads * 4u) {
@@ -103,10 +128,10 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
         for (uint32_t i = threadIdx.x * 4u; i < p.cols; i += kThreads * 4u) {  // each thread its own elements
             float4 v = *reinterpret_cast<float4 *>(xs + spread(i));
             const float4 x = *reinterpret_cast<const float4 *>(p.x + i), g = *reinterpret_cast<const float4 *>(p.norm_w + i);
-            v.x = x.x + v.x * inv * (1.0f + g.x);
-            v.y = x.y + v.y * inv * (1.0f + g.y);
-            v.z = x.z + v.z * inv * (1.0f + g.z);
-            v.w = x.w + v.w * inv * (1.0f + g.w);
+            v.x = x.x + v.x * inv * g.x;
+            v.y = x.y + v.y * inv * g.y;
+            v.z = x.z + v.z * inv * g.z;
+            v.w = x.w + v.w * inv * g.w;
             *reinterpret_cast<float4 *>(xs + spread(i)) = v;
             if (blockIdx.x == 0 && p.x_out) *reinterpret_cast<float4 *>(p.x_out + i) = v;
             s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -116,7 +141,7 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
             for (uint32_t i = threadIdx.x * 4u; i < p.cols; i += kThreads * 4u) {
                 float4 v = *reinterpret_cast<float4 *>(xs + spread(i));
                 const float4 g = *reinterpret_cast<const float4 *>(p.last_w + i);
-                v.x *= inv * (1.0f + g.x), v.y *= inv * (1.0f + g.y), v.z *= inv * (1.0f + g.z), v.w *= inv * (1.0f + g.w);
+                v.x *= inv * g.x, v.y *= inv * g.y, v.z *= inv * g.z, v.w *= inv * g.w;
                 *reinterpret_cast<float4 *>(xs + spread(i)) = v;
             }
         }
@@ -127,7 +152,21 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
     uint32_t top_i = 0xffffffffu;
     bool bad = false;
     uint32_t chunk = 0, cur = 0;
-    float acc[2] = {0.0f, 0.0f};
+    float acc[2] = {0.0f, 0.0f}, behind[2] = {0.0f, 0.0f};  // behind: columns from split_col on
+    float res[2], sa[2], sb[2];
+    auto fetch_residual = [&](uint32_t pr) {  // asked for when a pair begins, used when it ends
+        if constexpr (EPI == kRowResidual) {
+#pragma unroll
+            for (uint32_t j = 0; j < 2u; ++j) {
+                const uint32_t r = 2u * pr + j;
+                const bool in = pr < p.pairs && r < p.out_rows;
+                res[j] = in ? p.residual[r] : 0.0f;
+                sa[j] = in ? p.scale_a[r] : 0.0f;
+                sb[j] = in && p.scale_b ? p.scale_b[r] : 0.0f;
+            }
+        }
+    };
+    fetch_residual(pair);
     while (pair < p.pairs) {
         uint32_t next_pair = pair, next_chunk = chunk + kUnroll;
         if (next_chunk >= chunks) next_chunk = 0, next_pair = pair + stride;
@@ -138,8 +177,19 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
                 if (chunk + u >= chunks) break;
                 const float *xc = xs + (chunk + u) * kChunk + lane * 4u;
                 const float4 a = *reinterpret_cast<const float4 *>(xc), b = *reinterpret_cast<const float4 *>(xc + 128);
-                fma8(acc[0], now[u][0], a, b);
-                fma8(acc[1], now[u][1], a, b);
+                if (EPI == kRowResidual) {
+                    const bool first = (chunk + u) * kChunk + lane * 8u < p.split_col;
+#pragma unroll
+                    for (uint32_t j = 0; j < 2u; ++j) {
+                        float dot = 0.0f;
+                        fma8(dot, now[u][j], a, b);
+                        acc[j] += first ? dot : 0.0f;
+                        behind[j] += first ? 0.0f : dot;
+                    }
+                } else {
+                    fma8(acc[0], now[u][0], a, b);
+                    fma8(acc[1], now[u][1], a, b);
+                }
             }
         };
         if (cur == 0u) consume(buf[0], buf[1]);
@@ -148,11 +198,21 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
         if (next_pair != pair) {
             float v0 = warp_sum(acc[0]), v1 = warp_sum(acc[1]);
             acc[0] = acc[1] = 0.0f;
+            if constexpr (EPI == kRowResidual) {
+                const float w0 = warp_sum(behind[0]), w1 = warp_sum(behind[1]);
+                behind[0] = behind[1] = 0.0f;
+                v0 = fmaf(sb[0], w0, fmaf(sa[0], v0, res[0]));
+                v1 = fmaf(sb[1], w1, fmaf(sa[1], v1, res[1]));
+                fetch_residual(next_pair);
+            }
             if (lane == 0) {
-                const uint32_t r = row0(pair);
-                if (p.bias) v0 += p.bias[r], v1 += r + kApart < p.rows ? p.bias[r + kApart] : 0.0f;
-                if (EPI == kRowGate) {
-                    p.out[pair] = clamped_gate(v0, v1, p.limit);
+                const uint32_t r = row0(pair), step = apart(pair);
+                if (p.bias) v0 += p.bias[r], v1 += r + step < p.rows ? p.bias[r + step] : 0.0f;
+                if (is_gate(pair)) {
+                    p.out[pair - p.stored_pairs] = gated(p.gate, v0, v1);
+                } else if (EPI == kRowGate) {
+                    p.stored_out[r] = v0;
+                    p.stored_out[r + 1u] = v1;
                 } else {
                     if (r < p.out_rows) p.out[r] = v0;
                     if (r + 1u < p.out_rows) p.out[r + 1u] = v1;
@@ -184,8 +244,9 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
 
 // 64 x 64 tile, 256 threads of 4 x 4 outputs, K in steps of 32
 constexpr uint32_t kTile = 64, kStepK = 32;
-__global__ void __launch_bounds__(256) rows_gemm_f32_kernel(const uint16_t *w, uint32_t n, uint32_t k, const float *x, uint32_t m,
-                                                            const float *bias, float *out, uint32_t ld_out, uint32_t out_cols) {
+__global__ void __launch_bounds__(256) rows_gemm_f32_kernel(const uint16_t *w, uint32_t n, uint32_t k, uint32_t ld_w, const float *x,
+                                                            uint32_t m, const float *bias, float *out, uint32_t ld_out,
+                                                            uint32_t out_cols, const float *add_scale) {
     __shared__ float xt[kStepK][kTile + 4], wt[kStepK][kTile + 4];
     const uint32_t n0 = blockIdx.x * kTile, m0 = blockIdx.y * kTile, t = threadIdx.x;
     const uint32_t tm = (t >> 4) * 4u, tn = (t & 15u) * 4u;
@@ -194,7 +255,7 @@ __global__ void __launch_bounds__(256) rows_gemm_f32_kernel(const uint16_t *w, u
         for (uint32_t i = t; i < kTile * kStepK; i += 256u) {
             const uint32_t r = i / kStepK, c = i % kStepK;
             xt[c][r] = m0 + r < m ? x[(size_t)(m0 + r) * k + k0 + c] : 0.0f;
-            wt[c][r] = n0 + r < n ? bf16_bits_to_f32(w[(size_t)(n0 + r) * k + k0 + c]) : 0.0f;
+            wt[c][r] = n0 + r < n ? bf16_bits_to_f32(w[(size_t)(n0 + r) * ld_w + k0 + c]) : 0.0f;
         }
         __syncthreads();
 #pragma unroll 8
@@ -211,15 +272,22 @@ __global__ void __launch_bounds__(256) rows_gemm_f32_kernel(const uint16_t *w, u
     for (uint32_t i = 0; i < 4u; ++i)
         for (uint32_t j = 0; j < 4u; ++j) {
             const uint32_t r = m0 + tm + i, c = n0 + tn + j;
-            if (r < m && c < out_cols) out[(size_t)r * ld_out + c] = acc[i][j] + (bias ? bias[c] : 0.0f);
+            if (r >= m || c >= out_cols) continue;
+            float *dst = out + (size_t)r * ld_out + c;
+            const float v = acc[i][j] + (bias ? bias[c] : 0.0f);
+            *dst = add_scale ? fmaf(add_scale[c], v, *dst) : v;
         }
 }
 
 using MatvecKernel = void (*)(MatvecParams);
 template <uint32_t PRO>
 MatvecKernel pick(RowEpilogue e) {
-    return e == kRowStore ? matvec_b16_kernel<PRO, kRowStore>
-                          : (e == kRowGate ? matvec_b16_kernel<PRO, kRowGate> : matvec_b16_kernel<PRO, kRowLogits>);
+    switch (e) {
+        case kRowStore: return matvec_b16_kernel<PRO, kRowStore>;
+        case kRowGate: return matvec_b16_kernel<PRO, kRowGate>;
+        case kRowLogits: return matvec_b16_kernel<PRO, kRowLogits>;
+        default: return PRO == kRowPlain ? matvec_b16_kernel<kRowPlain, kRowResidual> : nullptr;
+    }
 }
 
 uint32_t matvec_smem(const MatrixB16 &w) { return (w.cols + kChunk - 1u) / kChunk * kChunk * 4u; }
@@ -229,29 +297,44 @@ uint32_t matvec_smem(const MatrixB16 &w) { return (w.cols + kChunk - 1u) / kChun
 bool matvec_b16_supports(const MatrixB16 &w) { return w.cols != 0 && w.cols % 64u == 0 && matvec_smem(w) <= 200u * 1024u; }
 
 stark_b200_status matvec_b16_launch(const MatvecArgs &a, cudaStream_t stream) {
-    if (!a.w.data || !a.x || !a.out || !matvec_b16_supports(a.w)) return STARK_B200_INVALID_ARGUMENT;
-    if (a.prologue != kRowPlain && (!a.y || !a.norm_w || a.x_out == a.x)) return STARK_B200_INVALID_ARGUMENT;
+    if (!a.w.data || !a.x || !a.out || !matvec_b16_supports(a.w) || a.w.pitch() != a.w.cols) return STARK_B200_INVALID_ARGUMENT;
+    const bool adds = a.prologue == kRowAddNorm || a.prologue == kRowAddNormNorm;
+    if ((adds && (!a.y || a.x_out == a.x)) || (a.prologue != kRowPlain && !a.norm_w)) return STARK_B200_INVALID_ARGUMENT;
     if (a.prologue == kRowAddNormNorm && !a.last_w) return STARK_B200_INVALID_ARGUMENT;
     if (a.epilogue == kRowLogits && (!a.partial_max || !a.partial_index)) return STARK_B200_INVALID_ARGUMENT;
-    if (a.epilogue == kRowGate && a.w.rows % 32u != 0) return STARK_B200_INVALID_ARGUMENT;
-    MatvecParams p{a.w.data, a.w.rows, a.w.cols, a.x, a.y, a.norm_w, a.last_w, a.x_out, a.width, a.eps, a.bias, a.limit,
-                   a.out, a.out_rows, a.partial_max, a.partial_index, (a.w.rows + 1u) / 2u};
+    if (a.epilogue == kRowGate &&
+        (a.w.rows % 32u || a.stored_rows % 32u || a.stored_rows > a.w.rows || (a.stored_rows && !a.stored_out)))
+        return STARK_B200_INVALID_ARGUMENT;
+    if (a.epilogue == kRowResidual &&
+        (a.prologue != kRowPlain || !a.residual || !a.scale_a || a.split_col % 8u || (a.split_col < a.w.cols && !a.scale_b) ||
+         a.out_rows > a.w.rows))
+        return STARK_B200_INVALID_ARGUMENT;
+    MatvecParams p{};
+    p.w = a.w.data, p.rows = a.w.rows, p.cols = a.w.cols;
+    p.x = a.x, p.y = a.y, p.norm_w = a.norm_w, p.last_w = a.last_w, p.x_out = a.x_out;
+    p.width = a.width, p.eps = a.eps, p.bias = a.bias, p.gate = a.gate;
+    p.out = a.out, p.out_rows = a.out_rows, p.partial_max = a.partial_max, p.partial_index = a.partial_index;
+    p.pairs = (a.w.rows + 1u) / 2u;
+    p.stored_pairs = a.epilogue == kRowGate ? a.stored_rows / 2u : 0u, p.stored_out = a.stored_out;
+    p.residual = a.residual, p.scale_a = a.scale_a, p.scale_b = a.scale_b, p.split_col = a.split_col;
     const uint32_t smem = matvec_smem(a.w);
     const uint32_t grid = std::min<uint32_t>((p.pairs + kWarps - 1u) / kWarps, 148u * (smem <= 100u * 1024u ? 2u : 1u));
-    MatvecKernel kernel = a.prologue == kRowPlain ? pick<kRowPlain>(a.epilogue)
-                                                  : (a.prologue == kRowAddNorm ? pick<kRowAddNorm>(a.epilogue)
-                                                                               : pick<kRowAddNormNorm>(a.epilogue));
-    static SmemOptIn once[3][3];
+    MatvecKernel kernel = a.prologue == kRowPlain
+                              ? pick<kRowPlain>(a.epilogue)
+                              : (a.prologue == kRowAddNorm
+                                     ? pick<kRowAddNorm>(a.epilogue)
+                                     : (a.prologue == kRowAddNormNorm ? pick<kRowAddNormNorm>(a.epilogue) : pick<kRowNorm>(a.epilogue)));
+    static SmemOptIn once[4][4];
     if (stark_b200_status st = ensure_dynamic_smem(kernel, 200 * 1024, once[a.prologue][a.epilogue])) return st;
     if (a.out_grid) *a.out_grid = grid;
     return launch_chained(kernel, dim3(grid), dim3(kThreads), smem, a.pdl, stream, p);
 }
 
 stark_b200_status rows_gemm_f32_launch(const MatrixB16 &w, const float *x, uint32_t m, const float *bias, float *out,
-                                       uint32_t ld_out, uint32_t out_cols, cudaStream_t stream) {
+                                       uint32_t ld_out, uint32_t out_cols, cudaStream_t stream, const float *add_scale) {
     if (!w.data || !x || !out || m == 0 || w.cols % 64u != 0) return STARK_B200_INVALID_ARGUMENT;
     rows_gemm_f32_kernel<<<dim3((std::min(w.rows, out_cols) + kTile - 1u) / kTile, (m + kTile - 1u) / kTile), 256, 0, stream>>>(
-        w.data, w.rows, w.cols, x, m, bias, out, ld_out, out_cols);
+        w.data, w.rows, w.cols, w.pitch(), x, m, bias, out, ld_out, out_cols, add_scale);
     SB_CUDA(cudaGetLastError());
     return STARK_B200_OK;
 }

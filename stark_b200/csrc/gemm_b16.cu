@@ -6,7 +6,8 @@
 //   warp 0      one thread: TMA loads of the step's activation boxes and of the weight box, all bf16 in 128-byte
 //               swizzled lines; rows and columns past the ends arrive as zeros
 //   warp 1      owns tensor memory; one thread issues the MMAs and commits them to the barrier that frees the stage
-//   warps 2-9   the epilogue: bias, then f32 or bf16 rows, or the clamped gate of 16 gate / 16 up columns in turn
+//   warps 2-9   the epilogue: bias, then f32 or bf16 rows, or the gate of 16 gate / 16 up columns in turn (columns in front
+//               of the gated ones stored as bf16 rows), or a scaled add to f32 rows (the residual stream)
 // Every wait is bounded; a wait that runs out sets the error word, the CTA drains and frees its tensor memory.
 #include <cuda.h>
 
@@ -38,9 +39,22 @@ struct GemmB16Params {
     uint32_t steps, m, out_cols, ld_out;
     void *out;
     const float *bias;
-    float limit;
+    Gate gate;
+    uint32_t stored_cols, ld_stored;
+    uint16_t *stored_out;
+    const float *scale;
     uint32_t *error_word;
 };
+
+// 32 f32 values as bf16 into a row, 16-byte aligned.
+__device__ inline void store_row32(uint16_t *dst, const uint32_t (&acc)[32]) {
+    uint32_t packed[16];
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) packed[i >> 1] = f32x2_to_bf16x2(__uint_as_float(acc[i]), __uint_as_float(acc[i + 1]));
+#pragma unroll
+    for (int q = 0; q < 4; ++q)
+        reinterpret_cast<uint4 *>(dst)[q] = make_uint4(packed[4 * q], packed[4 * q + 1], packed[4 * q + 2], packed[4 * q + 3]);
+}
 
 template <uint32_t HALVES, uint32_t KIND>
 __global__ void __launch_bounds__(kGemmThreads, 1)
@@ -139,23 +153,35 @@ gemm_b16_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
             }
             if (!row_ok) continue;
             if (KIND == kGemmGate) {
+                if (f0 < p.stored_cols) {
+                    store_row32(p.stored_out + (size_t)row * p.ld_stored + f0, acc);
+                    continue;
+                }
                 uint32_t packed[8];
 #pragma unroll
                 for (int i = 0; i < 16; i += 2)
-                    packed[i >> 1] = f32x2_to_bf16x2(clamped_gate(__uint_as_float(acc[i]), __uint_as_float(acc[16 + i]), p.limit),
-                                                     clamped_gate(__uint_as_float(acc[i + 1]), __uint_as_float(acc[17 + i]), p.limit));
-                uint4 *dst = reinterpret_cast<uint4 *>(static_cast<uint16_t *>(p.out) + (size_t)row * p.ld_out + f0 / 2u);
+                    packed[i >> 1] = f32x2_to_bf16x2(gated(p.gate, __uint_as_float(acc[i]), __uint_as_float(acc[16 + i])),
+                                                     gated(p.gate, __uint_as_float(acc[i + 1]), __uint_as_float(acc[17 + i])));
+                uint4 *dst = reinterpret_cast<uint4 *>(static_cast<uint16_t *>(p.out) + (size_t)row * p.ld_out + (f0 - p.stored_cols) / 2u);
                 dst[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
                 dst[1] = make_uint4(packed[4], packed[5], packed[6], packed[7]);
             } else if (KIND == kGemmBf16) {
-                uint32_t packed[16];
+                store_row32(static_cast<uint16_t *>(p.out) + (size_t)row * p.ld_out + f0, acc);
+            } else if (KIND == kGemmResidual) {
+                float4 *dst = reinterpret_cast<float4 *>(static_cast<float *>(p.out) + (size_t)row * p.ld_out + f0);
+                const float4 *scale = reinterpret_cast<const float4 *>(p.scale + f0);
+                float4 v[8];
 #pragma unroll
-                for (int i = 0; i < 32; i += 2)
-                    packed[i >> 1] = f32x2_to_bf16x2(__uint_as_float(acc[i]), __uint_as_float(acc[i + 1]));
-                uint4 *dst = reinterpret_cast<uint4 *>(static_cast<uint16_t *>(p.out) + (size_t)row * p.ld_out + f0);
+                for (int q = 0; q < 8; ++q) v[q] = dst[q];
 #pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    dst[q] = make_uint4(packed[4 * q], packed[4 * q + 1], packed[4 * q + 2], packed[4 * q + 3]);
+                for (int q = 0; q < 8; ++q) {
+                    const float4 g = __ldg(scale + q);
+                    v[q].x = fmaf(g.x, __uint_as_float(acc[4 * q]), v[q].x);
+                    v[q].y = fmaf(g.y, __uint_as_float(acc[4 * q + 1]), v[q].y);
+                    v[q].z = fmaf(g.z, __uint_as_float(acc[4 * q + 2]), v[q].z);
+                    v[q].w = fmaf(g.w, __uint_as_float(acc[4 * q + 3]), v[q].w);
+                    dst[q] = v[q];
+                }
             } else {
                 float *dst = static_cast<float *>(p.out) + (size_t)row * p.ld_out + f0;
                 if (whole && p.ld_out % 4u == 0) {
@@ -183,9 +209,11 @@ template <uint32_t HALVES>
 stark_b200_status launch(const GemmB16Args &a, const CUtensorMap &x_map, const CUtensorMap &w_map, const GemmB16Params &p,
                          cudaStream_t stream) {
     using T = Tile<HALVES>;
-    auto kernel = a.kind == kGemmBf16 ? gemm_b16_kernel<HALVES, kGemmBf16>
-                                      : (a.kind == kGemmF32 ? gemm_b16_kernel<HALVES, kGemmF32> : gemm_b16_kernel<HALVES, kGemmGate>);
-    static SmemOptIn once[3];
+    auto kernel = a.kind == kGemmBf16
+                      ? gemm_b16_kernel<HALVES, kGemmBf16>
+                      : (a.kind == kGemmF32 ? gemm_b16_kernel<HALVES, kGemmF32>
+                                            : (a.kind == kGemmGate ? gemm_b16_kernel<HALVES, kGemmGate> : gemm_b16_kernel<HALVES, kGemmResidual>));
+    static SmemOptIn once[4];
     if (stark_b200_status st = ensure_dynamic_smem(kernel, (int)T::kSmem, once[a.kind])) return st;
     kernel<<<dim3((a.m + 128u * HALVES - 1u) / (128u * HALVES), (a.out_cols + kBN - 1u) / kBN), kGemmThreads, T::kSmem, stream>>>(
         x_map, w_map, p);
@@ -201,6 +229,8 @@ stark_b200_status gemm_b16_launch(const GemmB16Args &a, cudaStream_t stream) {
         return STARK_B200_INVALID_ARGUMENT;
     // vector stores and bias reads work on whole 32-column blocks; only a bare f32 output may end inside one
     if ((a.kind != kGemmF32 || a.bias) && (a.out_cols % 32u || a.ld_out % 16u)) return STARK_B200_INVALID_ARGUMENT;
+    if (a.kind == kGemmGate && a.stored_cols && (!a.stored_out || a.stored_cols % 32u || a.ld_stored % 16u)) return STARK_B200_INVALID_ARGUMENT;
+    if (a.kind == kGemmResidual && (!a.scale || a.bias)) return STARK_B200_INVALID_ARGUMENT;
     DeviceContext *ctx = device_context();
     EncodeTiledFn encode = encode_tiled();
     if (!ctx || !encode) return STARK_B200_DEVICE_FAILURE;
@@ -213,9 +243,10 @@ stark_b200_status gemm_b16_launch(const GemmB16Args &a, cudaStream_t stream) {
                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                       CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
     };
-    if (!make(&x_map, a.x, a.x_rows, a.ld_x, 128u) || !make(&w_map, a.w.data, a.w.rows, a.w.cols, kBN))
+    if (!make(&x_map, a.x, a.x_rows, a.ld_x, 128u) || !make(&w_map, a.w.data, a.w.rows, a.w.pitch(), kBN))
         return STARK_B200_DEVICE_FAILURE;
-    const GemmB16Params p{a.w.cols / kBK, a.m, a.out_cols, a.ld_out, a.out, a.bias, a.limit, ctx->error_word};
+    const GemmB16Params p{a.w.cols / kBK, a.m, a.out_cols, a.ld_out, a.out, a.bias, a.gate, a.kind == kGemmGate ? a.stored_cols : 0u,
+                          a.ld_stored, a.stored_out, a.scale, ctx->error_word};
     // 256-row tiles unless 128-row tiles fill the SMs so much better that it pays for their loading the weight tile
     // once per 128 rows (a fifth slower per row)
     const uint32_t wide = (a.out_cols + kBN - 1u) / kBN, tall = (a.m + 255u) / 256u, flat = (a.m + 127u) / 128u;

@@ -15,17 +15,6 @@ namespace sb {
 namespace {
 
 constexpr uint32_t kQueryThreads = 256;
-constexpr float kLog2e = 1.4426950408889634f;
-
-template <typename T>
-__device__ inline float load_value(const T *p);
-template <>
-__device__ inline float load_value<float>(const float *p) { return *p; }
-template <>
-__device__ inline float load_value<uint16_t>(const uint16_t *p) { return bf16_bits_to_f32(*p); }
-__device__ inline void store_value(float *p, float v) { *p = v; }
-__device__ inline void store_value(uint16_t *p, float v) { *p = f32_to_bf16_bits(v); }
-
 __device__ inline float *partial_of(const LatentArgs &a, uint32_t row, uint32_t head, uint32_t split) {
     return a.partials + (((size_t)row * a.s.heads + head) * a.splits + split) * (a.s.rank_p + 4u);
 }
@@ -133,69 +122,11 @@ __global__ void __launch_bounds__(kQueryThreads) latent_query_kernel(const Laten
     }
 }
 
-// One head of one row over one span of whole pages, on the CUDA cores.  Serves f32 caches and any rank; the tensor-core
-// form below takes bf16 caches.
-constexpr uint32_t kAttendThreads = 256, kAttendColumns = 8;  // latent columns per thread: rank up to 2048
-template <typename C>
-__global__ void __launch_bounds__(kAttendThreads) latent_attend_kernel(const LatentArgs a) {
-    extern __shared__ float q[];  // [row()]
-    __shared__ float p[kPageTokens];
-    pdl_launch_dependents();
-    pdl_wait();
-    const LatentShape &s = a.s;
-    const uint32_t split = blockIdx.x, head = blockIdx.y, row = blockIdx.z, width = s.row();
-    const uint32_t pos = a.state ? a.state->position : a.first_pos + row;
-    const uint32_t pages = pos / kPageTokens + 1u, span = (pages + a.splits - 1u) / a.splits;
-    const uint32_t lo = min(pages, split * span), hi = min(pages, lo + span);
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
-    const float *src = a.queries + ((size_t)row * s.heads + head) * width;
-    for (uint32_t i = threadIdx.x; i < width; i += kAttendThreads) q[i] = src[i];
-    float m = -INFINITY, l = 0.0f, acc[kAttendColumns] = {};
-    for (uint32_t page = lo; page < hi; ++page) {
-        const C *keys = reinterpret_cast<const C *>(a.cache) + (size_t)a.block_table[page] * kPageTokens * width;
-        __syncthreads();
-        for (uint32_t k = warp; k < kPageTokens; k += kAttendThreads / 32u) {
-            float dot = -INFINITY;
-            if (page * kPageTokens + k <= pos) {
-                dot = 0.0f;
-                for (uint32_t i = lane; i < width; i += 32u) dot = fmaf(q[i], load_value(keys + (size_t)k * width + i), dot);
-                dot = warp_sum(dot);
-            }
-            if (lane == 0) p[k] = dot;
-        }
-        __syncthreads();
-        float top = m;
-        for (uint32_t k = 0; k < kPageTokens; ++k) top = fmaxf(top, p[k]);
-        const float keep = exp2f(m - top);  // 0 on the first page
-        m = top;
-        l *= keep;
-#pragma unroll
-        for (uint32_t c = 0; c < kAttendColumns; ++c) acc[c] *= keep;
-        for (uint32_t k = 0; k < kPageTokens; ++k) {
-            if (page * kPageTokens + k > pos) break;
-            const float w = exp2f(p[k] - top);
-            l += w;
-#pragma unroll
-            for (uint32_t c = 0; c < kAttendColumns; ++c) {
-                const uint32_t i = threadIdx.x + c * kAttendThreads;
-                if (i < s.rank_p) acc[c] = fmaf(w, load_value(keys + (size_t)k * width + i), acc[c]);
-            }
-        }
-    }
-    float *dst = partial_of(a, row, head, split);
-    if (threadIdx.x == 0) dst[0] = m, dst[1] = l;
-#pragma unroll
-    for (uint32_t c = 0; c < kAttendColumns; ++c) {
-        const uint32_t i = threadIdx.x + c * kAttendThreads;
-        if (i < s.rank_p) dst[4u + i] = acc[c];
-    }
-}
-
 // blockIdx.x: (head, 64 output values), blockIdx.y: row
 template <typename O>
 __global__ void __launch_bounds__(256) latent_value_kernel(const LatentArgs a) {
     extern __shared__ __align__(16) float o[];  // [rank_p], then the pieces of the merge
-    __shared__ float weight[kLatentMaxSplits];
+    __shared__ float weight[kMaxSplits];
     const LatentShape &s = a.s;
     const uint32_t blocks = s.vdim_p / 64u, head = blockIdx.x / blocks, piece = blockIdx.x % blocks, row = blockIdx.y;
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
@@ -302,7 +233,7 @@ __global__ void __launch_bounds__(256) latent_rotate_append_kernel(const LatentA
 stark_b200_status check_args(const LatentArgs &a) {
     if (!latent_shape_supported(a.s)) return STARK_B200_UNSUPPORTED;
     if (!a.qd || !a.cache || !a.block_table || !a.uk_uv.data || a.m == 0 || (a.state && a.m != 1u) || !a.rot.freq ||
-        a.splits > kLatentMaxSplits || a.splits == 0)
+        a.splits > kMaxSplits || a.splits == 0)
         return STARK_B200_INVALID_ARGUMENT;
     return STARK_B200_OK;
 }
@@ -311,7 +242,7 @@ stark_b200_status check_args(const LatentArgs &a) {
 
 bool latent_shape_supported(const LatentShape &s) {
     return s.heads != 0 && s.dim != 0 && s.rot_dim % 2u == 0 && s.vdim != 0 && s.rank != 0 &&
-           s.rank_p <= kAttendThreads * kAttendColumns && s.row() <= 4096u && s.dim_p <= 4096u;
+           span_attend_supports(s.row(), s.rank_p) && s.dim_p <= 4096u;
 }
 
 stark_b200_status latent_query_launch(const LatentArgs &a, cudaStream_t stream) {
@@ -328,8 +259,12 @@ stark_b200_status latent_attend_launch(const LatentArgs &a, cudaStream_t stream)
     if (!a.queries || !a.partials) return STARK_B200_INVALID_ARGUMENT;
     if (!a.cache_f32 && latent_attend_mma_supports(a.s)) return latent_attend_mma_launch(a, stream);
     if (a.cluster != 1u) return STARK_B200_INVALID_ARGUMENT;
-    auto kernel = a.cache_f32 ? latent_attend_kernel<float> : latent_attend_kernel<uint16_t>;
-    return launch_chained(kernel, dim3(a.splits, a.s.heads, a.m), dim3(kAttendThreads), a.s.row() * 4u, a.pdl, stream, a);
+    SpanAttendArgs g{};  // all heads share the cached rows; their values are the latent columns of the same rows
+    g.queries = a.queries, g.heads = a.s.heads, g.key_heads = 1, g.width = a.s.row(), g.out_width = a.s.rank_p;
+    g.keys = g.values = a.cache, g.key_pitch = g.value_pitch = a.s.row(), g.cache_f32 = a.cache_f32;
+    g.block_table = a.block_table, g.state = a.state, g.first_pos = a.first_pos, g.m = a.m, g.splits = a.splits;
+    g.partials = a.partials, g.pdl = a.pdl;
+    return span_attend_launch(g, stream);
 }
 
 stark_b200_status latent_value_launch(const LatentArgs &a, cudaStream_t stream) {

@@ -1,12 +1,14 @@
-// Causal latent attention of a prompt pass on the sm_100a tensor cores (tcgen05.mma, accumulators in tensor memory), in
-// the expanded form: keys W_uk c and values W_uv c of every visible row were formed by one contraction over the cache,
-// the rotated key part comes from the cache itself.
+// Causal attention of a prompt pass on the sm_100a tensor cores (tcgen05.mma, accumulators in tensor memory) for the layered
+// decoders' mixers.
 //
 // The scheme is that of prefill_attention_tc.cu -- one CTA owns 128 rows of one head and walks the keys twice, first for
 // every row's maximum, then P = exp2(S - max) and O += P V with P as bf16 hi + lo, so no accumulator is ever rescaled --
-// with two things of its own: query and value widths are arguments (whole blocks of 64, up to 256), and the key tile of a
-// step is put together from two places (per-head blocks of the expanded rows, shared blocks of the cache).  A step is one
-// cache page (64 keys), which leaves room for three key stages at 192-wide queries.
+// with three things of its own: query and value widths are arguments (whole blocks of 64, up to 256); the key tile of a
+// step may be put together from two places (blocks of the head's own, blocks every head shares); and where the scores are
+// bounded beforehand (queries and keys of unit root mean square) the bound stands in for the maximum and the keys are
+// walked once.  A step is one cache page (64 keys), which leaves room for three key stages at 192-wide queries.
+// Latent attention comes in the expanded form: keys W_uk c and values W_uv c of every visible row were formed by one
+// contraction over the cache, the rotated key part comes from the cache itself.  Grouped-query attention reads its pages.
 //   warps 0-7   softmax: thread = row (tensor-memory lane) x half of the step's keys
 //   warp 8      one thread: TMA loads
 //   warp 9      owns tensor memory; one thread issues the MMAs
@@ -17,6 +19,7 @@
 
 #include "device_math.cuh"
 #include "layered.cuh"
+#include "layered_math.cuh"
 #include "tc05.cuh"
 
 namespace sb {
@@ -41,14 +44,17 @@ __device__ inline float ex2_approx(float x) {
     return y;
 }
 
-struct LatentTcParams {
+struct AttendTcParams {
     uint16_t *out;
     const int32_t *block_table;
-    uint32_t m, first_pos, heads;
-    uint32_t nope_blocks, rot_blocks, value_blocks;  // of 64
-    uint32_t rot_column;                             // column of the rotated key part in a cache row
+    uint32_t m, first_pos, heads, key_heads;
+    uint32_t own_blocks, shared_blocks, value_blocks;  // of 64
+    uint32_t key_first, key_stride, value_first, value_stride, shared_first;
     uint32_t key_stages;
     float scale_log2;
+    uint32_t one_pass;                                 // the row's maximum is bound_log2 * |temperature|
+    float bound_log2, temp_coef;
+    uint32_t temp_every;
     uint32_t *error_word;
 };
 
@@ -58,11 +64,11 @@ uint32_t tc_smem_bytes(uint32_t q_blocks, uint32_t v_blocks, uint32_t key_stages
 }
 
 __global__ void __launch_bounds__(kThreads, 1)
-latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap e_map,
-                         const __grid_constant__ CUtensorMap c_map, const LatentTcParams p) {
-    extern __shared__ uint8_t latent_tc_smem[];
-    uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(latent_tc_smem) + 1023u) & ~(uintptr_t)1023u);
-    const uint32_t qb = p.nope_blocks + p.rot_blocks, vb = p.value_blocks;
+attend_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
+                 const __grid_constant__ CUtensorMap v_map, const __grid_constant__ CUtensorMap shared_map, const AttendTcParams p) {
+    extern __shared__ uint8_t attend_tc_smem[];
+    uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(attend_tc_smem) + 1023u) & ~(uintptr_t)1023u);
+    const uint32_t qb = p.own_blocks + p.shared_blocks, vb = p.value_blocks;
     const uint32_t key_bytes = qb * kKeyBlock, value_bytes = vb * kKeyBlock;
     uint8_t *q_smem = smem, *k_smem = q_smem + qb * kRowBlock, *v_smem = k_smem + p.key_stages * key_bytes;
     uint8_t *p_smem = v_smem + kValueStages * value_bytes, *tail = p_smem + 2u * kRowBlock;
@@ -74,7 +80,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
     float *exchange = reinterpret_cast<float *>(tail + 256u);  // [2][128]: what the two warps of a row tell each other
 
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    const uint32_t head = blockIdx.x;
+    const uint32_t head = blockIdx.x, key_head = head / (p.heads / p.key_heads);
     const uint32_t row0 = (gridDim.y - 1u - blockIdx.y) * 128u;  // late row blocks read the most keys: first
     const uint32_t last_row = min(p.m, row0 + 128u) - 1u;
     const uint32_t steps = (p.first_pos + last_row) / kKeys + 1u;
@@ -115,23 +121,23 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
                 tma_load_2d(q_smem + b * kRowBlock, &q_map, (head * qb + b) * 64u, row0, q_full);
             uint32_t ks = 0, kph = 1, vs = 0, vph = 1;  // a fresh barrier passes a wait on parity 1
             bool ok = true;
-            for (uint32_t pass = 0; pass < 2u && ok; ++pass) {
+            for (uint32_t pass = p.one_pass; pass < 2u && ok; ++pass) {
                 for (uint32_t j = 0; j < steps && ok; ++j) {
-                    const uint32_t y = (uint32_t)p.block_table[j] * kKeys;
+                    const uint32_t page = (uint32_t)p.block_table[j], y = (page * p.key_heads + key_head) * kKeys;
                     if (!(ok = mbar_wait_bounded(&k_empty[ks], kph, abort_flag))) break;
                     uint8_t *dst = k_smem + ks * key_bytes;
                     mbar_arrive_expect_tx(&k_full[ks], key_bytes);
-                    for (uint32_t b = 0; b < p.nope_blocks; ++b)
-                        tma_load_2d(dst + b * kKeyBlock, &e_map, (head * p.nope_blocks + b) * 64u, y, &k_full[ks]);
-                    for (uint32_t b = 0; b < p.rot_blocks; ++b)
-                        tma_load_2d(dst + (p.nope_blocks + b) * kKeyBlock, &c_map, p.rot_column + b * 64u, y, &k_full[ks]);
+                    for (uint32_t b = 0; b < p.own_blocks; ++b)
+                        tma_load_2d(dst + b * kKeyBlock, &k_map, p.key_first + head * p.key_stride + b * 64u, y, &k_full[ks]);
+                    for (uint32_t b = 0; b < p.shared_blocks; ++b)
+                        tma_load_2d(dst + (p.own_blocks + b) * kKeyBlock, &shared_map, p.shared_first + b * 64u, page * kKeys, &k_full[ks]);
                     if (++ks == p.key_stages) ks = 0, kph ^= 1u;
                     if (pass == 1u) {
                         if (!(ok = mbar_wait_bounded(&v_empty[vs], vph, abort_flag))) break;
                         mbar_arrive_expect_tx(&v_full[vs], value_bytes);
                         for (uint32_t b = 0; b < vb; ++b)
-                            tma_load_2d(v_smem + vs * value_bytes + b * kKeyBlock, &e_map,
-                                        (p.heads * p.nope_blocks + head * vb + b) * 64u, y, &v_full[vs]);
+                            tma_load_2d(v_smem + vs * value_bytes + b * kKeyBlock, &v_map,
+                                        p.value_first + head * p.value_stride + b * 64u, y, &v_full[vs]);
                         if (++vs == kValueStages) vs = 0, vph ^= 1u;
                     }
                 }
@@ -161,7 +167,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
                 if (++ks == p.key_stages) ks = 0, kph ^= 1u;
                 ++g;
             };
-            for (uint32_t j = 0; j < steps && ok; ++j) scores();
+            for (uint32_t j = 0; j < steps && ok && !p.one_pass; ++j) scores();
             const uint32_t hi_addr = smem_u32(p_smem), lo_addr = hi_addr + kRowBlock;
             for (uint32_t j = 0; j <= steps && ok; ++j) {
                 if (j < steps) scores();  // step j is multiplied while step j - 1 is exponentiated
@@ -193,7 +199,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
         float mrow = -INFINITY;
         uint32_t g = 0;
         bool ok = true;
-        for (uint32_t j = 0; j < steps && ok; ++j, ++g) {
+        for (uint32_t j = 0; j < steps && ok && !p.one_pass; ++j, ++g) {
             const uint32_t b = g & 1u;
             if (!(ok = mbar_wait_bounded(&s_full[b], (g >> 1) & 1u, abort_flag))) break;
             tc_fence_after();
@@ -214,10 +220,14 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
             }
             mrow = fmaxf(mrow, mx * p.scale_log2);  // the scale is positive: it commutes with the maximum
         }
-        exchange[half * 128u + r] = mrow;
-        named_bar_sync(1, kSoftmaxWarps * 32u);
-        mrow = fmaxf(mrow, exchange[(half ^ 1u) * 128u + r]);
-        named_bar_sync(1, kSoftmaxWarps * 32u);  // everybody has read: the words are free for the row sums
+        if (p.one_pass) {
+            mrow = p.bound_log2 * fabsf(query_temperature(pos, p.temp_coef, p.temp_every));
+        } else {
+            exchange[half * 128u + r] = mrow;
+            named_bar_sync(1, kSoftmaxWarps * 32u);
+            mrow = fmaxf(mrow, exchange[(half ^ 1u) * 128u + r]);
+            named_bar_sync(1, kSoftmaxWarps * 32u);  // everybody has read: the words are free for the row sums
+        }
         float l = 0.0f;
         uint8_t *p_hi = p_smem + r * 128u, *p_lo = p_hi + kRowBlock;
         for (uint32_t j = 0; j < steps && ok; ++j, ++g) {
@@ -291,28 +301,32 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid
 
 constexpr uint32_t kSmemLimit = 227u * 1024u;
 
-uint32_t stages_for(const LatentShape &s) {
+uint32_t stages_for(uint32_t key_blocks, uint32_t value_blocks) {
     for (uint32_t k = kMaxKeyStages; k >= 2u; --k)
-        if (tc_smem_bytes(s.q_head() / 64u, s.vdim_p / 64u, k) <= kSmemLimit) return k;
+        if (tc_smem_bytes(key_blocks, value_blocks, k) <= kSmemLimit) return k;
     return 0;
 }
 
+// Twice the bound is how far below it a score can lie; exp2 of that must stay well inside f32 and bf16.
+constexpr float kMostBelowBound = 100.0f;
+
 }  // namespace
 
-bool latent_prefill_tc_supports(const LatentShape &s) {
-    return s.q_head() <= kMaxBlocks * 64u && s.vdim_p <= kMaxBlocks * 64u && stages_for(s) != 0 && encode_tiled() != nullptr;
+bool attend_tc_supports(uint32_t key_blocks, uint32_t value_blocks) {
+    return key_blocks && value_blocks && key_blocks <= kMaxBlocks && value_blocks <= kMaxBlocks &&
+           stages_for(key_blocks, value_blocks) != 0 && encode_tiled() != nullptr;
 }
 
-stark_b200_status latent_prefill_tc_launch(const LatentArgs &a, cudaStream_t stream) {
-    if (!a.qd || !a.qd_b16 || a.cache_f32 || !a.cache || !a.expanded || !a.out || !a.out_b16 || !a.block_table || a.m == 0 ||
-        a.ld_qd % 8u || !(a.scale > 0.0f))
+stark_b200_status attend_tc_launch(const AttendTcArgs &a, cudaStream_t stream) {
+    const uint32_t key_blocks = a.own_blocks + a.shared_blocks;
+    if (!a.queries || !a.keys.base || !a.values.base || (a.shared_blocks && (!a.shared.base || a.key_heads != 1u)) || !a.out ||
+        !a.block_table || a.m == 0 || a.ld_q % 8u || !(a.scale > 0.0f) || !a.key_heads || a.heads % a.key_heads ||
+        (a.dim_bound > 0.0f && !a.temp_every))
         return STARK_B200_INVALID_ARGUMENT;
-    if (!latent_prefill_tc_supports(a.s)) return STARK_B200_UNSUPPORTED;
+    if (!attend_tc_supports(key_blocks, a.value_blocks)) return STARK_B200_UNSUPPORTED;
     EncodeTiledFn encode = encode_tiled();
-    const LatentShape &s = a.s;
-    const uint32_t pages = (a.first_pos + a.m + kPageTokens - 1u) / kPageTokens;
     const cuuint32_t elem[2] = {1u, 1u};
-    CUtensorMap q_map, e_map, c_map;
+    CUtensorMap q_map, k_map, v_map, shared_map;
     auto make = [&](CUtensorMap *map, const void *base, uint64_t columns, uint64_t rows, uint64_t ld, uint32_t box_rows) {
         const cuuint64_t dims[2] = {columns, rows}, strides[1] = {ld * 2u};
         const cuuint32_t box[2] = {64u, box_rows};
@@ -320,30 +334,59 @@ stark_b200_status latent_prefill_tc_launch(const LatentArgs &a, cudaStream_t str
                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                       CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
     };
-    const uint64_t expanded = (uint64_t)s.heads * (s.dim_p + s.vdim_p);
-    if (!make(&q_map, a.qd, s.q_width(), a.m, a.ld_qd, 128u) ||
-        !make(&e_map, a.expanded, expanded, (uint64_t)pages * kPageTokens, expanded, kKeys) ||
-        !make(&c_map, a.cache, s.row(), (uint64_t)a.num_blocks * kPageTokens, s.row(), kKeys))
+    const AttendTile &shared = a.shared_blocks ? a.shared : a.keys;
+    if (!make(&q_map, a.queries, (uint64_t)a.heads * key_blocks * 64u, a.m, a.ld_q, 128u) ||
+        !make(&k_map, a.keys.base, a.keys.columns, a.keys.rows, a.keys.ld, kKeys) ||
+        !make(&v_map, a.values.base, a.values.columns, a.values.rows, a.values.ld, kKeys) ||
+        !make(&shared_map, shared.base, shared.columns, shared.rows, shared.ld, kKeys))
         return STARK_B200_DEVICE_FAILURE;
-    LatentTcParams p{};
-    p.out = static_cast<uint16_t *>(a.out);
+    AttendTcParams p{};
+    p.out = a.out;
     p.block_table = a.block_table;
-    p.m = a.m;
-    p.first_pos = a.first_pos;
-    p.heads = s.heads;
-    p.nope_blocks = s.dim_p / 64u;
-    p.rot_blocks = s.rot_p / 64u;
-    p.value_blocks = s.vdim_p / 64u;
-    p.rot_column = s.rank_p;
-    p.key_stages = stages_for(s);
-    p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.m = a.m, p.first_pos = a.first_pos, p.heads = a.heads, p.key_heads = a.key_heads;
+    p.own_blocks = a.own_blocks, p.shared_blocks = a.shared_blocks, p.value_blocks = a.value_blocks;
+    p.key_first = a.keys.first, p.key_stride = a.keys.stride;
+    p.value_first = a.values.first, p.value_stride = a.values.stride;
+    p.shared_first = a.shared.first;
+    p.key_stages = stages_for(key_blocks, a.value_blocks);
+    p.scale_log2 = a.scale * kLog2e;
+    if (a.dim_bound > 0.0f) {
+        // the temperature moves one way with the position: its largest size is at the first or the last one
+        const float most = std::max(fabsf(query_temperature(0, a.temp_coef, a.temp_every)),
+                                    fabsf(query_temperature(a.first_pos + a.m - 1u, a.temp_coef, a.temp_every)));
+        p.bound_log2 = p.scale_log2 * a.dim_bound;
+        p.one_pass = 2.0f * p.bound_log2 * most <= kMostBelowBound ? 1u : 0u;
+        p.temp_coef = a.temp_coef, p.temp_every = a.temp_every;
+    }
     p.error_word = a.error_word;
     static SmemOptIn once;
-    if (stark_b200_status st = ensure_dynamic_smem(latent_prefill_tc_kernel, (int)kSmemLimit, once)) return st;
-    latent_prefill_tc_kernel<<<dim3(s.heads, (a.m + 127u) / 128u), kThreads,
-                               tc_smem_bytes(s.q_head() / 64u, s.vdim_p / 64u, p.key_stages), stream>>>(q_map, e_map, c_map, p);
+    if (stark_b200_status st = ensure_dynamic_smem(attend_tc_kernel, (int)kSmemLimit, once)) return st;
+    attend_tc_kernel<<<dim3(a.heads, (a.m + 127u) / 128u), kThreads, tc_smem_bytes(key_blocks, a.value_blocks, p.key_stages), stream>>>(
+        q_map, k_map, v_map, shared_map, p);
     SB_CUDA(cudaGetLastError());
     return STARK_B200_OK;
+}
+
+bool latent_prefill_tc_supports(const LatentShape &s) { return attend_tc_supports(s.q_head() / 64u, s.vdim_p / 64u); }
+
+stark_b200_status latent_prefill_tc_launch(const LatentArgs &a, cudaStream_t stream) {
+    if (!a.qd_b16 || a.cache_f32 || !a.cache || !a.expanded || !a.out_b16) return STARK_B200_INVALID_ARGUMENT;
+    const LatentShape &s = a.s;
+    const uint32_t rows = (a.first_pos + a.m + kPageTokens - 1u) / kPageTokens * kPageTokens;
+    const uint32_t expanded = s.heads * (s.dim_p + s.vdim_p);
+    AttendTcArgs t{};
+    t.queries = static_cast<const uint16_t *>(a.qd);
+    t.ld_q = a.ld_qd, t.heads = s.heads, t.key_heads = 1;
+    t.keys = {a.expanded, expanded, rows, expanded, 0u, s.dim_p};
+    t.values = {a.expanded, expanded, rows, expanded, s.heads * s.dim_p, s.vdim_p};
+    t.shared = {static_cast<const uint16_t *>(a.cache), s.row(), a.num_blocks * kPageTokens, s.row(), s.rank_p, 0u};
+    t.own_blocks = s.dim_p / 64u, t.shared_blocks = s.rot_p / 64u, t.value_blocks = s.vdim_p / 64u;
+    t.block_table = a.block_table;
+    t.first_pos = a.first_pos, t.m = a.m;
+    t.scale = a.scale;
+    t.out = static_cast<uint16_t *>(a.out);
+    t.error_word = a.error_word;
+    return attend_tc_launch(t, stream);
 }
 
 }  // namespace sb

@@ -3,7 +3,7 @@
 #include <algorithm>
 #include <cmath>
 
-#include "common.cuh"
+#include "layered.cuh"
 
 namespace sb {
 
@@ -28,6 +28,34 @@ __device__ inline float clamped_gate(float g, float u, float limit) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+__device__ inline float gated(const Gate &gate, float g, float u) {
+    return gate.kind == kGateSilu ? g / (1.0f + expf(-g)) * u : clamped_gate(g, u, gate.limit);
+}
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+template <typename T>
+__device__ inline float load_value(const T *p);
+template <>
+__device__ inline float load_value<float>(const float *p) { return *p; }
+template <>
+__device__ inline float load_value<uint16_t>(const uint16_t *p) { return bf16_bits_to_f32(*p); }
+__device__ inline void store_value(float *p, float v) { *p = v; }
+__device__ inline void store_value(uint16_t *p, float v) { *p = f32_to_bf16_bits(v); }
+// Two neighbours at an even index.
+__device__ inline float2 load_pair(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+__device__ inline float2 load_pair(const uint16_t *p) {
+    const uint32_t w = *reinterpret_cast<const uint32_t *>(p);
+    return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u));
+}
+__device__ inline void store_pair(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
+__device__ inline void store_pair(uint16_t *p, float2 v) { *reinterpret_cast<uint32_t *>(p) = f32x2_to_bf16x2(v.x, v.y); }
+
+// Factor on the queries of a position: 1 + coef * ln((position + 1) / every + 1), whole division.
+__host__ __device__ inline float query_temperature(uint32_t position, float coef, uint32_t every) {
+    return 1.0f + coef * logf((float)((position + 1u) / every + 1u));
 }
 
 template <typename... Params, typename... Args>

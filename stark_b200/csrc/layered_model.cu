@@ -1,16 +1,22 @@
-// The layered family: decoders whose configuration lists every layer's mixer and feed-forward (Guvulorn: latent
-// attention, clamped gated feed-forwards, norms on the sublayers' outputs, a hashed bigram table beside the embedding,
-// layers that use another layer's tensors).  This file holds what such a model owns -- tensors in the padded layout of
-// layered.cuh, one latent cache per layer over the session's page table, the token history -- and what one token and one
-// pass of prompt rows launch; stepping, recording, prompt loop, read-out, sampling and rewind are the shared token loop's.
+// The layered family: decoders whose configuration lists every layer's mixer and feed-forward.  Two mixers (latent
+// attention; grouped-query attention with short convolutions), two gated feed-forwards, two arrangements of a layer, an
+// embedding with or without a hashed bigram table and a norm, a read-out of its own or tied to the embedding, layers that
+// use another layer's tensors: Guvulorn and Pomelix are choices among them.  This file holds what such a model owns --
+// tensors in the padded layout of layered.cuh, a cache per layer over the session's page table, the state of the
+// convolutions, the token history -- and what one token and one pass of prompt rows launch; stepping, recording, prompt
+// loop, read-out, sampling and rewind are the shared token loop's.
 //
-// Per layer a token is seven launches (five without a feed-forward):
-//   [queries | latent, key part] = W x    matvec; the residual add of the sublayer before it in the prologue
-//   query, attend, value                  latent attention (latent_attention.cu)
+// Arrangement "post-norm": x += norm1(mixer(x)), x += norm2(ff(x)).  A token's layer:
+//   u = W x                               matvec; the residual add of the sublayer before it in the prologue
+//   mixer                                 latent: query, attend, value; grouped: one launch
 //   y = W_o attn                          matvec
 //   act = gate(W_gu x)                    matvec, x = x + norm1(y) in the prologue, biases and gate in the epilogue
 //   y = W_down act                        matvec
 // and the read-out matvec forms x + norm2(y) and the last norm in its prologue and the greedy pick in its epilogue.
+// Arrangement "parallel": h = norm1(x), x += mult * (scale1 * mixer(h) + scale2 * ff(h)).  A token's layer:
+//   [u | act] = [W; gate of W_gu] h       one matvec, the norm in its prologue, the gate in its epilogue
+//   mixer
+//   x += scale1 * W_o attn + scale2 * W_down act      one matvec over both inputs, the residual add in its epilogue
 #include "layered.cuh"
 
 #include <algorithm>
@@ -33,19 +39,32 @@ namespace sb {
 namespace {
 
 struct LayerTensors {
-    MatrixB16 qd, uk_uv, o, gate_up, down;
+    // in: the mixer's projections of the layer's input (parallel: gate and up rows behind them); parallel: out = o and
+    // down side by side.  gate_up, o and down are runs of those then, matrices of their own otherwise.
+    MatrixB16 in, out, uk_uv, gate_up, o, down;
     float *latent_norm = nullptr, *norm1 = nullptr, *norm2 = nullptr, *gate_up_b = nullptr, *down_b = nullptr;
+    float *conv_w = nullptr;                            // [taps][width of the projected row]
+    float *scale1 = nullptr, *scale2 = nullptr;         // times residual_mult
+    float share = 0.0f;
     uint32_t seen = 0;  // bit per tensor id
 };
 struct Layer {
     stark_b200_layer_desc d{};
-    LatentShape s{};
+    LatentShape s{};    // STARK_B200_MIXER_LATENT
     Rotation rot{};
     float *freq = nullptr;
+    void *cache = nullptr;
+    GroupedShape g{};   // STARK_B200_MIXER_GROUPED
+    uint32_t taps = 0;  // at least 1: a layer without convolutions has the factor 1 on every channel
+    void *keys = nullptr, *values = nullptr, *recent = nullptr, *tails = nullptr;
+    ValueMix mix = kMixNone;
     uint32_t ff_p = 0;
     uint32_t tensors = 0;  // index of the layer that holds them
     LayerTensors own;
-    void *cache = nullptr;
+    bool latent() const { return d.mixer == STARK_B200_MIXER_LATENT; }
+    uint32_t mixer_width() const { return latent() ? s.q_width() + s.row() : g.width(); }          // projected row
+    uint32_t attn_width() const { return latent() ? s.heads * s.vdim_p : g.heads * g.vdim_p; }     // attention output row
+    Gate gate() const { return {d.feed_forward == STARK_B200_FF_SILU_GATE ? kGateSilu : kGateClamped, d.ff_limit}; }
 };
 
 constexpr uint32_t kAttendRows = 64;    // rows of a pass the absorbed attention takes at a time
@@ -63,17 +82,21 @@ struct LayeredState {
     float *embed_norm = nullptr, *final_norm = nullptr;
     uint32_t seen = 0;
     uint32_t *history = nullptr;  // token ids by position: where a row's previous token comes from
+    bool parallel = false;
     // widest rows over the layers
-    uint32_t max_qd = 0, max_attn = 0, max_ff = 0, max_expand = 0;
+    uint32_t max_in = 0, max_mixer = 0, max_attn = 0, max_ff = 0, max_joint = 0, max_expand = 0, max_q = 0, max_first = 0;
     size_t query_floats = 0, partial_floats = 0;
-    // one token
-    float *x[2] = {nullptr, nullptr}, *y = nullptr, *qd = nullptr, *attn = nullptr, *act = nullptr;
-    float *queries = nullptr, *partials = nullptr;
+    uint32_t max_cluster = 8;  // of the grouped decode attention
+    // one token; attn: attention output with the gated activation behind it
+    float *x[2] = {nullptr, nullptr}, *y = nullptr, *u = nullptr, *attn = nullptr;
+    float *queries = nullptr, *partials = nullptr, *first_values = nullptr;
     // a pass of rows
     uint32_t rows = 0;
     float *rx = nullptr, *ry = nullptr;
-    uint16_t *rx_b16 = nullptr;
-    void *rqd = nullptr, *rattn = nullptr, *ract = nullptr;  // bf16, or f32 in the 32-bit form
+    void *rh = nullptr;                                      // what the contractions read: x or its norm, bf16 or f32
+    void *ru = nullptr, *rattn = nullptr, *ract = nullptr;   // bf16, or f32 in the 32-bit form
+    uint16_t *rq = nullptr;                                  // finished queries of the grouped mixer, bf16 form only
+    float *rfirst = nullptr;
     float *rgu = nullptr;                                    // 32-bit form only
     uint16_t *expanded = nullptr;
     size_t expanded_rows = 0;
@@ -99,7 +122,7 @@ stark_b200_status alloc_matrix(MatrixB16 &m, uint32_t rows, uint32_t cols) {
 // Rows [src_row, src_row + rows) x columns [src_col, src_col + cols) of a host matrix into the padded device matrix.
 stark_b200_status place(MatrixB16 &m, uint32_t row, uint32_t col, const uint16_t *src, uint32_t src_ld, uint32_t src_row,
                         uint32_t src_col, uint32_t rows, uint32_t cols) {
-    SB_CUDA(cudaMemcpy2D(m.data + (size_t)row * m.cols + col, (size_t)m.cols * 2u,
+    SB_CUDA(cudaMemcpy2D(m.data + (size_t)row * m.pitch() + col, (size_t)m.pitch() * 2u,
                          src + (size_t)src_row * src_ld + src_col, (size_t)src_ld * 2u, (size_t)cols * 2u, rows,
                          cudaMemcpyHostToDevice));
     return STARK_B200_OK;
@@ -111,10 +134,10 @@ stark_b200_status alloc_vector(float **dst, uint32_t padded) {
     SB_CUDA(cudaMemset(*dst, 0, (size_t)padded * 4u));
     return STARK_B200_OK;
 }
-stark_b200_status put_vector(float **dst, uint32_t padded, const uint16_t *src, uint32_t n) {
+stark_b200_status put_vector(float **dst, uint32_t padded, const uint16_t *src, uint32_t n, float offset = 0.0f, float factor = 1.0f) {
     SB_TRY(alloc_vector(dst, padded));
     std::vector<float> v(n);
-    for (uint32_t i = 0; i < n; ++i) v[i] = bf16_bits_to_f32(src[i]);
+    for (uint32_t i = 0; i < n; ++i) v[i] = (offset + bf16_bits_to_f32(src[i])) * factor;
     SB_CUDA(cudaMemcpy(*dst, v.data(), (size_t)n * 4u, cudaMemcpyHostToDevice));
     return STARK_B200_OK;
 }
@@ -158,7 +181,7 @@ void divide_cache(LatentArgs &a, uint32_t rows) {
         a.cluster = std::min(tunables().latent_cluster, spans);
         a.splits = spans / a.cluster;
     } else {
-        a.splits = std::max(1u, std::min(kLatentMaxSplits, 296u / (a.s.heads * rows)));
+        a.splits = std::max(1u, std::min(kMaxSplits, 296u / (a.s.heads * rows)));
     }
 }
 
@@ -177,15 +200,65 @@ LatentArgs latent_args(Model *m, const Layer &layer) {
     a.num_blocks = m->num_blocks;
     a.queries = L->queries;
     a.partials = L->partials;
-    a.ld_qd = tensors_of(L, layer).qd.rows;
+    a.ld_qd = layer.mixer_width();
     a.error_word = device_context()->error_word;
     return a;
 }
 
+// Spans of the grouped decode attention: a cluster of CTAs per key / value head (and 16 of its query heads), as large as
+// the SMs allow and the context has pages; more clusters, merged by a launch of their own, where heads are few and the
+// context is long.
+void divide_grouped(const Model *m, GroupedArgs &a) {
+    const uint32_t tiles = a.s.groups * ((a.s.per() + 15u) / 16u), pages = m->num_blocks;
+    uint32_t most = m->layered->max_cluster;
+    if (tunables().grouped_cluster) most = std::min(most, tunables().grouped_cluster);
+    a.cluster = 1;
+    while (a.cluster * 2u <= most && a.cluster * 2u * tiles <= 148u && a.cluster < pages) a.cluster *= 2u;
+    a.splits = std::max(1u, std::min({148u / (a.cluster * tiles), pages / (a.cluster * 16u), kMaxSplits}));
+    if (tunables().grouped_splits) a.splits = tunables().grouped_splits;
+}
+
+GroupedArgs grouped_args(Model *m, const Layer &layer) {
+    LayeredState *L = m->layered;
+    const LayerTensors &t = tensors_of(L, layer);
+    GroupedArgs a{};
+    a.s = layer.g;
+    a.conv = {t.conv_w, layer.taps, layer.recent, layer.tails};
+    a.ld_u = layer.mixer_width();
+    a.eps = L->c.eps, a.scale = layer.d.scale;
+    a.temp_coef = layer.d.q_temp_coef, a.temp_every = layer.d.q_temp_every;
+    a.mix = layer.mix, a.share = t.share;
+    a.keys = layer.keys, a.values = layer.values;
+    a.cache_f32 = L->f32;
+    a.block_table = m->block_table, a.num_blocks = m->num_blocks;
+    a.partials = L->partials;
+    a.splits = a.cluster = 1;
+    a.error_word = device_context()->error_word;
+    return a;
+}
+
+// The span attention over this layer's cache, behind grouped_rows.
+SpanAttendArgs span_args(const GroupedArgs &g, void *out, bool out_b16) {
+    SpanAttendArgs a{};
+    a.queries = g.queries;
+    a.heads = g.s.heads, a.key_heads = g.s.groups, a.width = g.s.dim_p, a.out_width = g.s.vdim_p;
+    a.keys = g.keys, a.values = g.values, a.key_pitch = g.s.dim_p, a.value_pitch = g.s.vdim_p;
+    a.cache_f32 = g.cache_f32;
+    a.block_table = g.block_table, a.state = g.state, a.first_pos = g.first_pos, a.m = g.m;
+    a.splits = g.splits;
+    a.partials = g.partials;
+    a.out = out, a.ld_out = g.s.heads * g.s.vdim_p, a.out_b16 = out_b16;
+    a.pdl = g.pdl;
+    return a;
+}
+uint32_t plain_splits(const GroupedShape &s, uint32_t rows) { return std::max(1u, std::min(kMaxSplits, 296u / (s.heads * rows))); }
+
 EmbedArgs embed_args(Model *m) {
     LayeredState *L = m->layered;
     EmbedArgs e{};
-    e.table = L->embed;
+    const bool tied = (L->c.flags & STARK_B200_LAYERED_TIED_HEAD) != 0u;
+    e.table = tied ? L->head.data : L->embed;
+    e.ld_table = tied ? L->width_p : L->c.width;
     e.bigram = L->bigram;
     e.buckets = L->c.bigram_buckets;
     e.width = L->c.width;
@@ -197,6 +270,85 @@ EmbedArgs embed_args(Model *m) {
     e.norm_w = L->embed_norm;
     e.history = L->history;
     return e;
+}
+
+// A layer's mixer for one token: projected row in `u`, attention output to `attn`.
+stark_b200_status token_mixer(Model *m, const Layer &layer, uint32_t *launches) {
+    LayeredState *L = m->layered;
+    cudaStream_t s = m->stream;
+    const bool pdl = tunables().pdl != 0u;
+    if (layer.latent()) {
+        LatentArgs a = latent_args(m, layer);
+        a.qd = L->u;
+        a.state = m->state;
+        a.m = 1;
+        divide_cache(a, 1);
+        a.out = L->attn;
+        a.pdl = pdl;
+        SB_TRY(latent_query_launch(a, s));
+        SB_TRY(latent_attend_launch(a, s));
+        *launches += 3;
+        return latent_value_launch(a, s);
+    }
+    GroupedArgs a = grouped_args(m, layer);
+    a.u = L->u;
+    a.first_values = L->first_values;
+    a.state = m->state;
+    a.m = 1;
+    a.pdl = pdl;
+    if (!L->f32 && grouped_attend_mma_supports(layer.g)) {
+        divide_grouped(m, a);
+        a.out = L->attn;
+        SB_TRY(grouped_attend_mma_launch(a, s));
+        ++*launches;
+        if (a.splits == 1u) return STARK_B200_OK;
+    } else {
+        a.queries = L->queries;
+        a.splits = plain_splits(layer.g, 1);
+        SB_TRY(grouped_rows_launch(a, s));
+        SB_TRY(span_attend_launch(span_args(a, nullptr, false), s));
+        *launches += 2;
+    }
+    ++*launches;
+    return span_merge_launch(span_args(a, L->attn, false), s);
+}
+
+stark_b200_status token_parallel_layer(Model *m, const Layer &layer, uint32_t *launches) {
+    LayeredState *L = m->layered;
+    const LayerTensors &t = tensors_of(L, layer);
+    const bool pdl = tunables().pdl != 0u, ff = layer.d.feed_forward != STARK_B200_FF_NONE;
+    MatvecArgs a{};
+    a.w = t.in;
+    a.prologue = kRowNorm;
+    a.x = L->x[0];
+    a.norm_w = t.norm1;
+    a.width = L->c.width;
+    a.eps = L->c.eps;
+    a.pdl = pdl;
+    if (ff) {
+        a.epilogue = kRowGate;
+        a.gate = layer.gate();
+        a.stored_rows = layer.mixer_width();
+        a.stored_out = L->u;
+        a.out = L->attn + layer.attn_width();
+    } else {
+        a.out = L->u;
+        a.out_rows = t.in.rows;
+    }
+    SB_TRY(matvec_b16_launch(a, m->stream));
+    SB_TRY(token_mixer(m, layer, launches));
+    MatvecArgs o{};
+    o.w = t.out;
+    o.epilogue = kRowResidual;
+    o.x = L->attn;
+    o.residual = o.out = L->x[0];
+    o.scale_a = t.scale1;
+    o.scale_b = t.scale2;
+    o.split_col = layer.attn_width();
+    o.out_rows = t.out.rows;
+    o.pdl = pdl;
+    *launches += 2;
+    return matvec_b16_launch(o, m->stream);
 }
 
 stark_b200_status layered_issue_token(Model *m, bool full, uint32_t *launches) {
@@ -227,23 +379,18 @@ stark_b200_status layered_issue_token(Model *m, bool full, uint32_t *launches) {
         }
     };
     for (const Layer &layer : L->layers) {
+        if (L->parallel) {
+            SB_TRY(token_parallel_layer(m, layer, &n));
+            continue;
+        }
         const LayerTensors &t = tensors_of(L, layer);
         MatvecArgs a{};
-        a.w = t.qd;
+        a.w = t.in;
         input(a);
-        a.out = L->qd;
-        a.out_rows = t.qd.rows;
+        a.out = L->u;
+        a.out_rows = t.in.rows;
         SB_TRY(matvec_b16_launch(a, s));
-        LatentArgs la = latent_args(m, layer);
-        la.qd = L->qd;
-        la.state = m->state;
-        la.m = 1;
-        divide_cache(la, 1);
-        la.out = L->attn;
-        la.pdl = pdl;
-        SB_TRY(latent_query_launch(la, s));
-        SB_TRY(latent_attend_launch(la, s));
-        SB_TRY(latent_value_launch(la, s));
+        SB_TRY(token_mixer(m, layer, &n));
         MatvecArgs o{};
         o.w = t.o;
         o.x = L->attn;
@@ -252,20 +399,20 @@ stark_b200_status layered_issue_token(Model *m, bool full, uint32_t *launches) {
         o.pdl = pdl;
         SB_TRY(matvec_b16_launch(o, s));
         pending = t.norm1;
-        n += 5;
+        n += 2;
         if (layer.d.feed_forward == STARK_B200_FF_NONE) continue;
+        float *act = L->attn + layer.attn_width();
         MatvecArgs g{};
         g.w = t.gate_up;
         input(g);
         g.epilogue = kRowGate;
         g.bias = t.gate_up_b;
-        g.limit = layer.d.ff_limit;
-        g.out = L->act;
-        g.out_rows = layer.ff_p;
+        g.gate = layer.gate();
+        g.out = act;
         SB_TRY(matvec_b16_launch(g, s));
         MatvecArgs d{};
         d.w = t.down;
-        d.x = L->act;
+        d.x = act;
         d.bias = t.down_b;
         d.out = L->y;
         d.out_rows = t.down.rows;
@@ -278,8 +425,9 @@ stark_b200_status layered_issue_token(Model *m, bool full, uint32_t *launches) {
         MatvecArgs h{};
         h.w = L->head;
         input(h);
-        h.prologue = kRowAddNormNorm;
-        h.last_w = L->final_norm;
+        h.prologue = L->parallel ? kRowNorm : kRowAddNormNorm;
+        if (L->parallel) h.norm_w = L->final_norm;
+        else h.last_w = L->final_norm;
         h.epilogue = kRowLogits;
         h.out = m->logits_f32;
         h.out_rows = L->c.vocab;
@@ -306,13 +454,16 @@ bool layered_rows_ready(Model *m) {
     const uint32_t rows = std::min<uint32_t>(kPrefillBatchRows, m->num_blocks * kPageTokens);
     const size_t element = L->f32 ? 4u : 2u;
     auto bytes = [&](void **p, size_t n) { return dmalloc(reinterpret_cast<uint8_t **>(p), n) == STARK_B200_OK; };
+    // the 32-bit form leaves a fused contraction's gate and up columns beside the projected row; the bf16 form never does
     if (dmalloc(&m->chunk_tokens, kPrefillBatchRows + 8u) != STARK_B200_OK ||
         dmalloc(&L->rx, (size_t)rows * L->width_p) != STARK_B200_OK ||
-        dmalloc(&L->ry, (size_t)rows * L->width_p) != STARK_B200_OK ||
-        dmalloc(&L->rx_b16, (size_t)rows * L->width_p) != STARK_B200_OK ||
-        !bytes(&L->rqd, rows * element * L->max_qd) || !bytes(&L->rattn, rows * element * L->max_attn) ||
+        (!L->parallel && dmalloc(&L->ry, (size_t)rows * L->width_p) != STARK_B200_OK) ||
+        ((L->parallel || !L->f32) && !bytes(&L->rh, rows * element * L->width_p)) ||
+        !bytes(&L->ru, rows * element * (L->f32 ? L->max_in : L->max_mixer)) || !bytes(&L->rattn, rows * element * L->max_attn) ||
         !bytes(&L->ract, rows * element * std::max(64u, L->max_ff)) ||
-        (L->f32 && dmalloc(&L->rgu, (size_t)rows * 2u * std::max(64u, L->max_ff)) != STARK_B200_OK) ||
+        (!L->f32 && L->max_q && dmalloc(&L->rq, (size_t)rows * L->max_q) != STARK_B200_OK) ||
+        (L->max_first && dmalloc(&L->rfirst, (size_t)rows * L->max_first) != STARK_B200_OK) ||
+        (L->f32 && !L->parallel && dmalloc(&L->rgu, (size_t)rows * 2u * std::max(64u, L->max_ff)) != STARK_B200_OK) ||
         dmalloc(&L->picked, kReadoutRows) != STARK_B200_OK ||
         !bytes(&L->picked_x, (size_t)kReadoutRows * L->width_p * 4u) ||
         dmalloc(&L->picked_logits, (size_t)kReadoutRows * L->c.vocab) != STARK_B200_OK)
@@ -321,10 +472,11 @@ bool layered_rows_ready(Model *m) {
     return true;
 }
 
-// Attention of a pass over the cache, query rows in `rqd`, output rows in `rattn`.
-stark_b200_status rows_attention(Model *m, const Layer &layer, uint32_t mrows, uint32_t first_pos, uint32_t *launches) {
+// Attention of a pass over the cache, projected rows in `ru` (ld_u apart), output rows in `rattn`.
+stark_b200_status rows_latent(Model *m, const Layer &layer, uint32_t ld_u, uint32_t mrows, uint32_t first_pos, uint32_t *launches) {
     LayeredState *L = m->layered;
     LatentArgs a = latent_args(m, layer);
+    a.ld_qd = ld_u;
     a.qd_b16 = !L->f32;
     a.out_b16 = !L->f32;
     const size_t element = L->f32 ? 4u : 2u;
@@ -339,7 +491,7 @@ stark_b200_status rows_attention(Model *m, const Layer &layer, uint32_t mrows, u
             SB_TRY(dmalloc(&L->expanded, std::max(want, visible) * L->max_expand));
             L->expanded_rows = std::max(want, visible);
         }
-        a.qd = L->rqd;
+        a.qd = L->ru;
         a.first_pos = first_pos;
         a.m = mrows;
         a.splits = 1;
@@ -363,8 +515,8 @@ stark_b200_status rows_attention(Model *m, const Layer &layer, uint32_t mrows, u
     for (uint32_t r = 0; r < mrows; r += kAttendRows) {
         a.m = std::min(kAttendRows, mrows - r);
         a.first_pos = first_pos + r;
-        a.qd = static_cast<const uint8_t *>(L->rqd) + (size_t)r * a.ld_qd * element;
-        a.out = static_cast<uint8_t *>(L->rattn) + (size_t)r * layer.s.heads * layer.s.vdim_p * element;
+        a.qd = static_cast<const uint8_t *>(L->ru) + (size_t)r * a.ld_qd * element;
+        a.out = static_cast<uint8_t *>(L->rattn) + (size_t)r * layer.attn_width() * element;
         divide_cache(a, a.m);
         SB_TRY(latent_query_launch(a, m->stream));
         SB_TRY(latent_attend_launch(a, m->stream));
@@ -374,9 +526,62 @@ stark_b200_status rows_attention(Model *m, const Layer &layer, uint32_t mrows, u
     return STARK_B200_OK;
 }
 
+stark_b200_status rows_grouped(Model *m, const Layer &layer, uint32_t ld_u, uint32_t mrows, uint32_t first_pos, uint32_t *launches) {
+    LayeredState *L = m->layered;
+    const GroupedShape &s = layer.g;
+    GroupedArgs a = grouped_args(m, layer);
+    a.u_b16 = !L->f32;
+    a.ld_u = ld_u;
+    if (!L->f32 && layer.d.scale > 0.0f && attend_tc_supports(s.dim_p / 64u, s.vdim_p / 64u)) {
+        a.u = L->ru;
+        a.first_values = L->rfirst;
+        a.first_pos = first_pos;
+        a.m = mrows;
+        a.queries_b16 = L->rq;
+        SB_TRY(grouped_rows_launch(a, m->stream));
+        AttendTcArgs t{};
+        const uint32_t cached = m->num_blocks * s.groups * kPageTokens;
+        t.queries = L->rq;
+        t.ld_q = s.heads * s.dim_p, t.heads = s.heads, t.key_heads = s.groups;
+        t.keys = {static_cast<const uint16_t *>(layer.keys), s.dim_p, cached, s.dim_p, 0u, 0u};
+        t.values = {static_cast<const uint16_t *>(layer.values), s.vdim_p, cached, s.vdim_p, 0u, 0u};
+        t.own_blocks = s.dim_p / 64u, t.value_blocks = s.vdim_p / 64u;
+        t.block_table = m->block_table;
+        t.first_pos = first_pos, t.m = mrows;
+        t.scale = layer.d.scale;
+        t.dim_bound = (float)s.dim;  // a query (without its temperature) and a key have norms of sqrt(dim) at most
+        t.temp_coef = a.temp_coef, t.temp_every = a.temp_every;
+        t.out = static_cast<uint16_t *>(L->rattn);
+        t.error_word = a.error_word;
+        *launches += mrows > kConvSpare && layer.taps > 1u ? 3u : 2u;
+        return attend_tc_launch(t, m->stream);
+    }
+    const size_t element = L->f32 ? 4u : 2u;
+    a.queries = L->queries;
+    for (uint32_t r = 0; r < mrows; r += kAttendRows) {
+        a.m = std::min(kAttendRows, mrows - r);
+        a.first_pos = first_pos + r;
+        a.u = static_cast<const uint8_t *>(L->ru) + (size_t)r * ld_u * element;
+        a.first_values = L->rfirst ? L->rfirst + (size_t)r * s.groups * s.vdim_p : nullptr;
+        a.splits = plain_splits(s, a.m);
+        const SpanAttendArgs span =
+            span_args(a, static_cast<uint8_t *>(L->rattn) + (size_t)r * layer.attn_width() * element, !L->f32);
+        SB_TRY(grouped_rows_launch(a, m->stream));
+        SB_TRY(span_attend_launch(span, m->stream));
+        SB_TRY(span_merge_launch(span, m->stream));
+        *launches += a.m > kConvSpare && layer.taps > 1u ? 4u : 3u;
+    }
+    return STARK_B200_OK;
+}
+
+stark_b200_status rows_mixer(Model *m, const Layer &layer, uint32_t ld_u, uint32_t mrows, uint32_t first_pos, uint32_t *launches) {
+    return layer.latent() ? rows_latent(m, layer, ld_u, mrows, first_pos, launches)
+                          : rows_grouped(m, layer, ld_u, mrows, first_pos, launches);
+}
+
 // y = x W^T of a pass; x is the bf16 or f32 form of the rows
 stark_b200_status rows_contract(Model *m, const MatrixB16 &w, const void *x, uint32_t mrows, const float *bias, void *out,
-                                GemmB16Out kind, float limit, uint32_t *launches) {
+                                GemmB16Out kind, Gate gate, uint32_t *launches) {
     LayeredState *L = m->layered;
     ++*launches;
     if (L->f32) {
@@ -384,7 +589,7 @@ stark_b200_status rows_contract(Model *m, const MatrixB16 &w, const void *x, uin
             return rows_gemm_f32_launch(w, static_cast<const float *>(x), mrows, bias, static_cast<float *>(out), w.rows, w.rows, m->stream);
         SB_TRY(rows_gemm_f32_launch(w, static_cast<const float *>(x), mrows, bias, L->rgu, w.rows, w.rows, m->stream));
         ++*launches;
-        return clamped_gate_rows_launch(L->rgu, static_cast<float *>(out), mrows, w.rows / 2u, limit, m->stream);
+        return gate_rows_launch(L->rgu, w.rows, static_cast<float *>(out), mrows, w.rows / 2u, gate, m->stream);
     }
     GemmB16Args g{};
     g.w = w;
@@ -397,8 +602,70 @@ stark_b200_status rows_contract(Model *m, const MatrixB16 &w, const void *x, uin
     g.out_cols = w.rows;
     g.ld_out = kind == kGemmGate ? w.rows / 2u : w.rows;
     g.bias = bias;
-    g.limit = limit;
+    g.gate = gate;
     return gemm_b16_launch(g, m->stream);
+}
+
+// x += scale * (in W^T) of a pass
+stark_b200_status rows_add_contract(Model *m, const MatrixB16 &w, const void *in, uint32_t mrows, const float *scale, uint32_t *launches) {
+    LayeredState *L = m->layered;
+    ++*launches;
+    if (L->f32)
+        return rows_gemm_f32_launch(w, static_cast<const float *>(in), mrows, nullptr, L->rx, L->width_p, w.rows, m->stream, scale);
+    GemmB16Args g{};
+    g.w = w;
+    g.x = static_cast<const uint16_t *>(in);
+    g.x_rows = L->rows;
+    g.m = mrows;
+    g.ld_x = w.cols;
+    g.kind = kGemmResidual;
+    g.out = L->rx;
+    g.ld_out = L->width_p;
+    g.out_cols = w.rows;
+    g.scale = scale;
+    return gemm_b16_launch(g, m->stream);
+}
+
+stark_b200_status rows_parallel_layer(Model *m, const Layer &layer, uint32_t mrows, uint32_t first_pos, uint32_t *launches) {
+    LayeredState *L = m->layered;
+    const LayerTensors &t = tensors_of(L, layer);
+    const bool ff = layer.d.feed_forward != STARK_B200_FF_NONE;
+    const uint32_t mixer = layer.mixer_width();
+    uint32_t ld_u = mixer;
+    SB_TRY(norm_rows_launch(L->rx, nullptr, mrows, t.norm1, L->c.width, L->c.eps, L->f32 ? static_cast<float *>(L->rh) : nullptr,
+                            L->f32 ? nullptr : static_cast<uint16_t *>(L->rh), m->stream));
+    if (L->f32) {
+        float *u = static_cast<float *>(L->ru);
+        ld_u = t.in.rows;
+        SB_TRY(rows_gemm_f32_launch(t.in, static_cast<const float *>(L->rh), mrows, nullptr, u, ld_u, ld_u, m->stream));
+        if (ff) SB_TRY(gate_rows_launch(u + mixer, ld_u, static_cast<float *>(L->ract), mrows, layer.ff_p, layer.gate(), m->stream));
+        *launches += ff ? 3u : 2u;
+    } else {
+        GemmB16Args g{};
+        g.w = t.in;
+        g.x = static_cast<const uint16_t *>(L->rh);
+        g.x_rows = L->rows;
+        g.m = mrows;
+        g.ld_x = t.in.cols;
+        g.out_cols = t.in.rows;
+        if (ff) {
+            g.kind = kGemmGate;
+            g.gate = layer.gate();
+            g.stored_cols = g.ld_stored = mixer;
+            g.stored_out = static_cast<uint16_t *>(L->ru);
+            g.out = L->ract;
+            g.ld_out = layer.ff_p;
+        } else {
+            g.kind = kGemmBf16;
+            g.out = L->ru;
+            g.ld_out = mixer;
+        }
+        SB_TRY(gemm_b16_launch(g, m->stream));
+        *launches += 2;
+    }
+    SB_TRY(rows_mixer(m, layer, ld_u, mrows, first_pos, launches));
+    SB_TRY(rows_add_contract(m, t.o, L->rattn, mrows, t.scale1, launches));
+    return ff ? rows_add_contract(m, t.down, L->ract, mrows, t.scale2, launches) : STARK_B200_OK;
 }
 
 stark_b200_status layered_rows_pass(Model *m, const uint32_t *tokens_device, uint32_t mrows, uint32_t first_pos) {
@@ -411,21 +678,25 @@ stark_b200_status layered_rows_pass(Model *m, const uint32_t *tokens_device, uin
     e.tokens = tokens_device;
     e.first_pos = first_pos;
     e.x = L->rx;
-    e.x_b16 = L->f32 ? nullptr : L->rx_b16;
+    e.x_b16 = L->f32 || L->parallel ? nullptr : static_cast<uint16_t *>(L->rh);
     e.m = mrows;
     SB_TRY(embed_norm_launch(e, s));
-    const void *x = L->f32 ? static_cast<const void *>(L->rx) : static_cast<const void *>(L->rx_b16);
-    uint16_t *rounded = L->f32 ? nullptr : L->rx_b16;
+    const void *x = L->f32 ? static_cast<const void *>(L->rx) : L->rh;
+    uint16_t *rounded = L->f32 ? nullptr : static_cast<uint16_t *>(L->rh);
     for (const Layer &layer : L->layers) {
+        if (L->parallel) {
+            SB_TRY(rows_parallel_layer(m, layer, mrows, first_pos, &n));
+            continue;
+        }
         const LayerTensors &t = tensors_of(L, layer);
-        SB_TRY(rows_contract(m, t.qd, x, mrows, nullptr, L->rqd, L->f32 ? kGemmF32 : kGemmBf16, 0.0f, &n));
-        SB_TRY(rows_attention(m, layer, mrows, first_pos, &n));
-        SB_TRY(rows_contract(m, t.o, L->rattn, mrows, nullptr, L->ry, kGemmF32, 0.0f, &n));
+        SB_TRY(rows_contract(m, t.in, x, mrows, nullptr, L->ru, L->f32 ? kGemmF32 : kGemmBf16, Gate{}, &n));
+        SB_TRY(rows_mixer(m, layer, layer.mixer_width(), mrows, first_pos, &n));
+        SB_TRY(rows_contract(m, t.o, L->rattn, mrows, nullptr, L->ry, kGemmF32, Gate{}, &n));
         SB_TRY(add_norm_rows_launch(L->rx, L->ry, t.norm1, mrows, L->c.width, L->c.eps, rounded, s));
         ++n;
         if (layer.d.feed_forward == STARK_B200_FF_NONE) continue;
-        SB_TRY(rows_contract(m, t.gate_up, x, mrows, t.gate_up_b, L->ract, kGemmGate, layer.d.ff_limit, &n));
-        SB_TRY(rows_contract(m, t.down, L->ract, mrows, t.down_b, L->ry, kGemmF32, 0.0f, &n));
+        SB_TRY(rows_contract(m, t.gate_up, x, mrows, t.gate_up_b, L->ract, kGemmGate, layer.gate(), &n));
+        SB_TRY(rows_contract(m, t.down, L->ract, mrows, t.down_b, L->ry, kGemmF32, Gate{}, &n));
         SB_TRY(add_norm_rows_launch(L->rx, L->ry, t.norm2, mrows, L->c.width, L->c.eps, rounded, s));
         ++n;
     }
@@ -442,9 +713,9 @@ stark_b200_status layered_rows_logits(Model *m, const uint32_t *rows, uint32_t c
         for (uint32_t i = 0; i < n; ++i)
             if (rows[done + i] >= mrows) return STARK_B200_INVALID_ARGUMENT;
         SB_CUDA(cudaMemcpyAsync(L->picked, rows + done, n * 4u, cudaMemcpyHostToDevice, s));
-        SB_TRY(norm_gather_rows_launch(L->rx, L->picked, n, L->final_norm, L->c.width, L->c.eps,
-                                       L->f32 ? static_cast<float *>(L->picked_x) : nullptr,
-                                       L->f32 ? nullptr : static_cast<uint16_t *>(L->picked_x), s));
+        SB_TRY(norm_rows_launch(L->rx, L->picked, n, L->final_norm, L->c.width, L->c.eps,
+                                L->f32 ? static_cast<float *>(L->picked_x) : nullptr,
+                                L->f32 ? nullptr : static_cast<uint16_t *>(L->picked_x), s));
         if (L->f32) {
             SB_TRY(rows_gemm_f32_launch(L->head, static_cast<const float *>(L->picked_x), n, nullptr, L->picked_logits,
                                         (uint32_t)vocab, (uint32_t)vocab, s));
@@ -472,31 +743,71 @@ stark_b200_status layered_rows_logits(Model *m, const uint32_t *rows, uint32_t c
 
 uint32_t layered_vocab(const Model *m) { return m->layered->c.vocab; }
 
+constexpr uint32_t bit(uint32_t id) { return 1u << id; }
+
+uint32_t model_tensors(const stark_b200_layered_config &c) {
+    uint32_t want = bit(STARK_B200_LAYERED_EMBED) | bit(STARK_B200_LAYERED_FINAL_NORM);
+    if (c.flags & STARK_B200_LAYERED_HAS_EMBED_NORM) want |= bit(STARK_B200_LAYERED_EMBED_NORM);
+    if (!(c.flags & STARK_B200_LAYERED_TIED_HEAD)) want |= bit(STARK_B200_LAYERED_HEAD);
+    if (c.bigram_buckets) want |= bit(STARK_B200_LAYERED_BIGRAM);
+    return want;
+}
+
+uint32_t layer_tensors(const LayeredState *L, const Layer &l) {
+    uint32_t want = bit(STARK_B200_LAYERED_NORM1) | bit(STARK_B200_LAYERED_Q) | bit(STARK_B200_LAYERED_O);
+    if (l.latent()) {
+        want |= bit(STARK_B200_LAYERED_DKV) | bit(STARK_B200_LAYERED_DKV_NORM) | bit(STARK_B200_LAYERED_UK) | bit(STARK_B200_LAYERED_UV);
+    } else {
+        want |= bit(STARK_B200_LAYERED_K) | bit(STARK_B200_LAYERED_V);
+        if (l.d.conv_taps) want |= bit(STARK_B200_LAYERED_Q_CONV) | bit(STARK_B200_LAYERED_K_CONV) | bit(STARK_B200_LAYERED_V_CONV);
+        if (l.d.v_mix) want |= bit(STARK_B200_LAYERED_V_SHARE);
+    }
+    if (L->parallel) want |= bit(STARK_B200_LAYERED_SCALE1);
+    if (l.d.feed_forward == STARK_B200_FF_NONE) return want;
+    want |= bit(STARK_B200_LAYERED_GATE) | bit(STARK_B200_LAYERED_UP) | bit(STARK_B200_LAYERED_DOWN);
+    want |= L->parallel ? bit(STARK_B200_LAYERED_SCALE2) : bit(STARK_B200_LAYERED_NORM2);
+    if (l.d.feed_forward == STARK_B200_FF_CLAMPED_GATE)
+        want |= bit(STARK_B200_LAYERED_GATE_BIAS) | bit(STARK_B200_LAYERED_UP_BIAS) | bit(STARK_B200_LAYERED_DOWN_BIAS);
+    return want;
+}
+
 stark_b200_status layered_ready(Model *m) {
     LayeredState *L = m->layered;
-    uint32_t want = 1u << STARK_B200_LAYERED_EMBED | 1u << STARK_B200_LAYERED_EMBED_NORM |
-                    1u << STARK_B200_LAYERED_FINAL_NORM | 1u << STARK_B200_LAYERED_HEAD;
-    if (L->c.bigram_buckets) want |= 1u << STARK_B200_LAYERED_BIGRAM;
-    if (L->seen != want) return STARK_B200_INVALID_STATE;
-    for (uint32_t i = 0; i < L->layers.size(); ++i) {
-        const Layer &layer = L->layers[i];
-        if (layer.tensors != i) continue;
-        uint32_t need = 0;
-        for (uint32_t t = STARK_B200_LAYERED_NORM1; t <= STARK_B200_LAYERED_O; ++t) need |= 1u << t;
-        if (layer.d.feed_forward != STARK_B200_FF_NONE)
-            for (uint32_t t = STARK_B200_LAYERED_NORM2; t <= STARK_B200_LAYERED_DOWN_BIAS; ++t) need |= 1u << t;
-        if (layer.own.seen != need) return STARK_B200_INVALID_STATE;
-    }
+    if (L->seen != model_tensors(L->c)) return STARK_B200_INVALID_STATE;
+    for (uint32_t i = 0; i < L->layers.size(); ++i)
+        if (L->layers[i].tensors == i && L->layers[i].own.seen != layer_tensors(L, L->layers[i])) return STARK_B200_INVALID_STATE;
     return STARK_B200_OK;
+}
+
+// The cache alone does not describe a layer with convolutions: its recent rows are put back as they were at the start of
+// the position's page, and the tokens between are run again.
+stark_b200_status layered_rewind(Model *m, uint64_t position) {
+    LayeredState *L = m->layered;
+    if (position == m->position || position == 0) return STARK_B200_OK;
+    const uint32_t page_start = (uint32_t)(position / kPageTokens * kPageTokens);
+    bool any = false;
+    for (const Layer &layer : L->layers) {
+        if (layer.latent() || layer.taps <= 1u) continue;
+        SB_TRY(short_conv_restore_launch(grouped_args(m, layer), page_start, m->stream));
+        any = true;
+    }
+    if (!any || position == page_start) return STARK_B200_OK;
+    if (!layered_rows_ready(m)) return STARK_B200_OUT_OF_MEMORY;
+    return layered_rows_pass(m, L->history + page_start, (uint32_t)(position - page_start), page_start);
 }
 
 void layered_sizes(const Model *m, uint64_t *weight_bytes, uint64_t *kv_bytes_per_token) {
     const LayeredState *L = m->layered;
-    uint64_t w = L->head.bytes() + (uint64_t)L->c.vocab * L->c.width * 2u +
+    const bool tied = (L->c.flags & STARK_B200_LAYERED_TIED_HEAD) != 0u;
+    uint64_t w = L->head.bytes() + (tied ? 0u : (uint64_t)L->c.vocab * L->c.width * 2u) +
                  (L->c.bigram_buckets ? ((uint64_t)L->c.bigram_buckets + 1u) * L->c.width * 2u : 0u), kv = 0;
     for (const Layer &l : L->layers) {
-        for (const MatrixB16 *t : {&l.own.qd, &l.own.uk_uv, &l.own.o, &l.own.gate_up, &l.own.down}) w += t->bytes();
-        kv += (uint64_t)l.s.row() * (L->f32 ? 4u : 2u);
+        for (const MatrixB16 *t : {&l.own.in, &l.own.out, &l.own.uk_uv}) w += t->bytes();
+        if (!L->parallel)
+            for (const MatrixB16 *t : {&l.own.o, &l.own.gate_up, &l.own.down}) w += t->bytes();
+        const uint64_t row = l.latent() ? l.s.row()
+                                        : l.g.groups * (l.g.dim_p + l.g.vdim_p) + ((l.taps - 1u) * l.g.width() + kPageTokens - 1u) / kPageTokens;
+        kv += row * (L->f32 ? 4u : 2u);
     }
     *weight_bytes = w;
     *kv_bytes_per_token = kv;
@@ -506,15 +817,19 @@ void layered_destroy(Model *m) {
     LayeredState *L = m->layered;
     if (!L) return;
     for (Layer &l : L->layers) {
-        for (MatrixB16 *t : {&l.own.qd, &l.own.uk_uv, &l.own.o, &l.own.gate_up, &l.own.down}) cudaFree(t->data);
-        for (float *p : {l.own.latent_norm, l.own.norm1, l.own.norm2, l.own.gate_up_b, l.own.down_b, l.freq}) cudaFree(p);
-        cudaFree(l.cache);
+        for (MatrixB16 *t : {&l.own.in, &l.own.out, &l.own.uk_uv}) cudaFree(t->data);
+        if (!L->parallel)
+            for (MatrixB16 *t : {&l.own.o, &l.own.gate_up, &l.own.down}) cudaFree(t->data);
+        for (float *p : {l.own.latent_norm, l.own.norm1, l.own.norm2, l.own.gate_up_b, l.own.down_b, l.own.conv_w, l.own.scale1,
+                         l.own.scale2, l.freq})
+            cudaFree(p);
+        for (void *p : {l.cache, l.keys, l.values, l.recent, l.tails}) cudaFree(p);
     }
     for (void *p : {(void *)L->embed, (void *)L->bigram, (void *)L->head.data, (void *)L->embed_norm, (void *)L->final_norm,
-                    (void *)L->history, (void *)L->x[0], (void *)L->x[1], (void *)L->y, (void *)L->qd, (void *)L->attn,
-                    (void *)L->act, (void *)L->queries, (void *)L->partials, (void *)L->rx, (void *)L->ry, (void *)L->rx_b16,
-                    L->rqd, L->rattn, L->ract, (void *)L->rgu, (void *)L->expanded, (void *)L->picked, L->picked_x,
-                    (void *)L->picked_logits})
+                    (void *)L->history, (void *)L->x[0], (void *)L->x[1], (void *)L->y, (void *)L->u, (void *)L->attn,
+                    (void *)L->queries, (void *)L->partials, (void *)L->first_values, (void *)L->rx, (void *)L->ry, L->rh,
+                    L->ru, L->rattn, L->ract, (void *)L->rq, (void *)L->rfirst, (void *)L->rgu, (void *)L->expanded,
+                    (void *)L->picked, L->picked_x, (void *)L->picked_logits})
         cudaFree(p);
     delete L;
     m->layered = nullptr;
@@ -530,21 +845,91 @@ ModelFamily make_layered_family() {
     f.rows_ready = layered_rows_ready;
     f.rows_pass = layered_rows_pass;
     f.rows_logits = layered_rows_logits;
+    f.rewind = layered_rewind;
     f.sizes = layered_sizes;
     f.destroy = layered_destroy;
     return f;
 }
 const ModelFamily kLayeredFamily = make_layered_family();
 
-stark_b200_status check_layer(const stark_b200_layer_desc &d) {
+stark_b200_status check_layer(const stark_b200_layered_config &c, const stark_b200_layer_desc &d) {
     if (d.struct_size != sizeof(d)) return STARK_B200_ABI_MISMATCH;
-    if (d.mixer != STARK_B200_MIXER_LATENT || d.feed_forward > STARK_B200_FF_CLAMPED_GATE || d.rot_scaling > STARK_B200_ROT_YARN)
+    const bool latent = d.mixer == STARK_B200_MIXER_LATENT;
+    if ((!latent && d.mixer != STARK_B200_MIXER_GROUPED) || d.feed_forward > STARK_B200_FF_SILU_GATE ||
+        d.rot_scaling > STARK_B200_ROT_YARN ||
+        (c.arrangement == STARK_B200_ARRANGE_PARALLEL && d.feed_forward == STARK_B200_FF_CLAMPED_GATE))  // has biases
         return STARK_B200_UNSUPPORTED;
-    if (!d.heads || !d.dim || !d.vdim || !d.kv_rank || d.rot_dim % 2u || d.rot_dims % 2u || d.rot_dims > d.rot_dim ||
-        !std::isfinite(d.scale) || !(d.rot_base > 0.0) ||
-        (d.rot_scaling == STARK_B200_ROT_YARN && !(d.rot_factor > 0.0 && d.rot_original > 0.0 && d.rot_fast > 0.0 && d.rot_slow > 0.0)) ||
-        (d.feed_forward == STARK_B200_FF_CLAMPED_GATE && !d.ff_width))
+    if (!d.heads || !d.dim || !d.vdim || !std::isfinite(d.scale) || (d.feed_forward != STARK_B200_FF_NONE && !d.ff_width))
         return STARK_B200_INVALID_ARGUMENT;
+    if (latent &&
+        (!d.kv_rank || d.rot_dim % 2u || d.rot_dims % 2u || d.rot_dims > d.rot_dim || !(d.rot_base > 0.0) ||
+         (d.rot_scaling == STARK_B200_ROT_YARN && !(d.rot_factor > 0.0 && d.rot_original > 0.0 && d.rot_fast > 0.0 && d.rot_slow > 0.0))))
+        return STARK_B200_INVALID_ARGUMENT;
+    if (!latent && (!d.kv_heads || d.heads % d.kv_heads || !d.q_temp_every || !std::isfinite(d.q_temp_coef) || d.rot_dim))
+        return STARK_B200_INVALID_ARGUMENT;
+    return STARK_B200_OK;
+}
+
+stark_b200_status zeroed(void **p, size_t bytes) {
+    SB_TRY(dmalloc(reinterpret_cast<uint8_t **>(p), bytes));
+    SB_CUDA(cudaMemset(*p, 0, bytes ? bytes : 1u));
+    return STARK_B200_OK;
+}
+
+stark_b200_status build_latent(Model *m, Layer &l) {
+    LayeredState *L = m->layered;
+    LatentShape &s = l.s;
+    s.heads = l.d.heads, s.dim = l.d.dim, s.rot_dim = l.d.rot_dim, s.vdim = l.d.vdim, s.rank = l.d.kv_rank;
+    s.dim_p = pad64(s.dim), s.rot_p = pad64(s.rot_dim), s.vdim_p = pad64(s.vdim), s.rank_p = pad64(s.rank);
+    if (!latent_shape_supported(s)) return STARK_B200_UNSUPPORTED;
+    std::vector<float> freq(std::max(1u, s.rot_p / 2u), 0.0f);
+    rotation_table(l.d, freq, &l.rot.factor);
+    SB_TRY(dmalloc(&l.freq, freq.size()));
+    SB_CUDA(cudaMemcpy(l.freq, freq.data(), freq.size() * 4u, cudaMemcpyHostToDevice));
+    l.rot.freq = l.freq;
+    l.rot.pairs = l.d.rot_dims / 2u;
+    SB_TRY(zeroed(&l.cache, (size_t)m->num_blocks * kPageTokens * s.row() * (L->f32 ? 4u : 2u)));
+    L->max_expand = std::max(L->max_expand, s.heads * (s.dim_p + s.vdim_p));
+    L->query_floats = std::max(L->query_floats, (size_t)kAttendRows * s.heads * s.row());
+    for (uint32_t r = 1; r <= kAttendRows; ++r) {
+        LatentArgs probe{};
+        probe.s = s;
+        probe.cache_f32 = L->f32;
+        divide_cache(probe, r);
+        L->partial_floats = std::max(L->partial_floats, latent_partial_floats(s, r, probe.splits * probe.cluster));
+    }
+    return STARK_B200_OK;
+}
+
+stark_b200_status build_grouped(Model *m, Layer &l) {
+    LayeredState *L = m->layered;
+    GroupedShape &s = l.g;
+    s.heads = l.d.heads, s.groups = l.d.kv_heads, s.dim = l.d.dim, s.vdim = l.d.vdim;
+    s.dim_p = pad64(s.dim), s.vdim_p = pad64(s.vdim);
+    l.taps = std::max(1u, l.d.conv_taps);
+    if (!grouped_shape_supported(s, l.taps)) return STARK_B200_UNSUPPORTED;
+    if (!l.d.conv_taps && &tensors_of(L, l) == &l.own) {
+        const std::vector<float> ones(s.width(), 1.0f);
+        SB_TRY(dmalloc(&l.own.conv_w, ones.size()));
+        SB_CUDA(cudaMemcpy(l.own.conv_w, ones.data(), ones.size() * 4u, cudaMemcpyHostToDevice));
+    }
+    const size_t element = L->f32 ? 4u : 2u, positions = (size_t)m->num_blocks * kPageTokens;
+    SB_TRY(zeroed(&l.keys, positions * s.groups * s.dim_p * element));
+    SB_TRY(zeroed(&l.values, positions * s.groups * s.vdim_p * element));
+    SB_TRY(zeroed(&l.recent, (size_t)(l.taps + kConvSpare) * s.width() * element));
+    SB_TRY(zeroed(&l.tails, (size_t)m->num_blocks * (l.taps - 1u) * s.width() * element));
+    L->max_q = std::max(L->max_q, s.heads * s.dim_p);
+    if (l.d.v_mix) {
+        const uint32_t row = s.groups * s.vdim_p;
+        if (L->max_first && row != L->max_first) return STARK_B200_INVALID_ARGUMENT;  // the values mixed must be alike
+        l.mix = L->max_first ? kMixShare : kMixFirst;
+        L->max_first = row;
+    }
+    L->query_floats = std::max(L->query_floats, (size_t)kAttendRows * s.heads * s.dim_p);
+    for (uint32_t r = 1; r <= kAttendRows; ++r)
+        L->partial_floats = std::max(L->partial_floats, span_partial_floats(s.heads, s.vdim_p, r, plain_splits(s, r)));
+    L->partial_floats = std::max(L->partial_floats, span_partial_floats(s.heads, s.vdim_p, 1u, kMaxSplits));
+    if (!L->f32 && grouped_attend_mma_supports(s)) L->max_cluster = std::max(L->max_cluster, grouped_attend_mma_max_cluster(s));
     return STARK_B200_OK;
 }
 
@@ -554,7 +939,7 @@ stark_b200_status build_layers(Model *m, const stark_b200_layer_desc *descs) {
     for (uint32_t i = 0; i < L->c.layers; ++i) {
         Layer &l = L->layers[i];
         l.d = descs[i];
-        SB_TRY(check_layer(l.d));
+        SB_TRY(check_layer(L->c, l.d));
         l.tensors = i;
         if (l.d.weights_of != UINT32_MAX) {
             if (l.d.weights_of >= L->c.layers || descs[l.d.weights_of].weights_of != UINT32_MAX) return STARK_B200_INVALID_ARGUMENT;
@@ -564,41 +949,22 @@ stark_b200_status build_layers(Model *m, const stark_b200_layer_desc *descs) {
             if (memcmp(&a, &b, sizeof a) != 0) return STARK_B200_INVALID_ARGUMENT;
             l.tensors = l.d.weights_of;
         }
-        LatentShape &s = l.s;
-        s.heads = l.d.heads, s.dim = l.d.dim, s.rot_dim = l.d.rot_dim, s.vdim = l.d.vdim, s.rank = l.d.kv_rank;
-        s.dim_p = pad64(s.dim), s.rot_p = pad64(s.rot_dim), s.vdim_p = pad64(s.vdim), s.rank_p = pad64(s.rank);
-        if (!latent_shape_supported(s)) return STARK_B200_UNSUPPORTED;
         l.ff_p = l.d.feed_forward == STARK_B200_FF_NONE ? 0u : pad64(l.d.ff_width);
-        std::vector<float> freq(std::max(1u, s.rot_p / 2u), 0.0f);
-        rotation_table(l.d, freq, &l.rot.factor);
-        SB_TRY(dmalloc(&l.freq, freq.size()));
-        SB_CUDA(cudaMemcpy(l.freq, freq.data(), freq.size() * 4u, cudaMemcpyHostToDevice));
-        l.rot.freq = l.freq;
-        l.rot.pairs = l.d.rot_dims / 2u;
-        const size_t cache = (size_t)m->num_blocks * kPageTokens * s.row() * (L->f32 ? 4u : 2u);
-        SB_CUDA(cudaMalloc(&l.cache, cache));
-        SB_CUDA(cudaMemset(l.cache, 0, cache));
-        L->max_qd = std::max(L->max_qd, s.q_width() + s.row());
-        L->max_attn = std::max(L->max_attn, s.heads * s.vdim_p);
+        SB_TRY(l.latent() ? build_latent(m, l) : build_grouped(m, l));
+        L->max_mixer = std::max(L->max_mixer, l.mixer_width());
+        L->max_in = std::max(L->max_in, l.mixer_width() + (L->parallel ? 2u * l.ff_p : 0u));
+        L->max_attn = std::max(L->max_attn, l.attn_width());
         L->max_ff = std::max(L->max_ff, l.ff_p);
-        L->max_expand = std::max(L->max_expand, s.heads * (s.dim_p + s.vdim_p));
-        L->query_floats = std::max(L->query_floats, (size_t)kAttendRows * s.heads * s.row());
-        for (uint32_t r = 1; r <= kAttendRows; ++r) {
-            LatentArgs probe{};
-            probe.s = s;
-            probe.cache_f32 = L->f32;
-            divide_cache(probe, r);
-            L->partial_floats = std::max(L->partial_floats, latent_partial_floats(s, r, probe.splits * probe.cluster));
-        }
+        L->max_joint = std::max(L->max_joint, l.attn_width() + std::max(64u, l.ff_p));
     }
-    for (const MatrixB16 probe : {MatrixB16{nullptr, 1, L->width_p}, MatrixB16{nullptr, 1, L->max_attn},
-                                  MatrixB16{nullptr, 1, std::max(64u, L->max_ff)}})
+    for (const MatrixB16 &probe : {MatrixB16{nullptr, 1, L->width_p}, MatrixB16{nullptr, 1, L->parallel ? L->max_joint : L->max_attn},
+                                   MatrixB16{nullptr, 1, std::max(64u, L->max_ff)}})
         if (!matvec_b16_supports(probe)) return STARK_B200_UNSUPPORTED;
     SB_TRY(dmalloc(&L->history, (size_t)m->num_blocks * kPageTokens + 1u));
     for (float **p : {&L->x[0], &L->x[1], &L->y}) SB_TRY(dmalloc(p, L->width_p));
-    SB_TRY(dmalloc(&L->qd, L->max_qd));
-    SB_TRY(dmalloc(&L->attn, L->max_attn));
-    SB_TRY(dmalloc(&L->act, std::max(64u, L->max_ff)));
+    SB_TRY(dmalloc(&L->u, L->max_mixer));
+    SB_TRY(dmalloc(&L->attn, L->max_joint));
+    if (L->max_first) SB_TRY(dmalloc(&L->first_values, L->max_first));
     SB_TRY(dmalloc(&L->queries, L->query_floats));
     return dmalloc(&L->partials, L->partial_floats);
 }
@@ -606,7 +972,7 @@ stark_b200_status build_layers(Model *m, const stark_b200_layer_desc *descs) {
 stark_b200_status layered_create(const stark_b200_layered_config &c, const stark_b200_layer_desc *descs, Model **out) {
     *out = nullptr;
     if (!c.vocab || !c.width || !c.layers || !c.context_tokens || c.width > 32768u || !(c.eps >= 0.0f) ||
-        c.compute > STARK_B200_F32 || (uint64_t)c.bigram_buckets + 1u > UINT32_MAX || c.bigram_mul_prev > UINT32_MAX ||
+        c.compute > STARK_B200_F32 || c.arrangement > STARK_B200_ARRANGE_PARALLEL || !std::isfinite(c.residual_mult) || (uint64_t)c.bigram_buckets + 1u > UINT32_MAX || c.bigram_mul_prev > UINT32_MAX ||
         c.bigram_mul_cur > UINT32_MAX)
         return STARK_B200_INVALID_ARGUMENT;
     if (!device_context()) return STARK_B200_DEVICE_FAILURE;
@@ -622,6 +988,7 @@ stark_b200_status layered_create(const stark_b200_layered_config &c, const stark
     L->c = c;
     L->width_p = pad64(c.width);
     L->f32 = c.compute == STARK_B200_F32;
+    L->parallel = c.arrangement == STARK_B200_ARRANGE_PARALLEL;
     m->cfg.layers = c.layers;
     m->cfg.hidden = c.width;
     m->cfg.vocab = c.vocab;
@@ -637,62 +1004,129 @@ stark_b200_status layered_create(const stark_b200_layered_config &c, const stark
     return STARK_B200_OK;
 }
 
+// Storage of the fused matrices, made when the first of their parts arrives.
+stark_b200_status input_matrix(LayeredState *L, Layer &l) {
+    LayerTensors &t = l.own;
+    const uint32_t fused = L->parallel ? 2u * l.ff_p : 0u;
+    SB_TRY(alloc_matrix(t.in, l.mixer_width() + fused, L->width_p));
+    if (!l.ff_p) return STARK_B200_OK;
+    if (fused) t.gate_up = t.in.row_range(l.mixer_width(), fused);
+    else SB_TRY(alloc_matrix(t.gate_up, 2u * l.ff_p, L->width_p));
+    return STARK_B200_OK;
+}
+stark_b200_status output_matrices(LayeredState *L, Layer &l) {
+    LayerTensors &t = l.own;
+    if (!L->parallel) {
+        SB_TRY(alloc_matrix(t.o, L->width_p, l.attn_width()));
+        return l.ff_p ? alloc_matrix(t.down, L->width_p, l.ff_p) : STARK_B200_OK;
+    }
+    SB_TRY(alloc_matrix(t.out, L->width_p, l.attn_width() + l.ff_p));
+    t.o = t.out.column_range(0, l.attn_width());
+    if (l.ff_p) t.down = t.out.column_range(l.attn_width(), l.ff_p);
+    return STARK_B200_OK;
+}
+
+stark_b200_status set_model_tensor(LayeredState *L, uint32_t which, const uint16_t *src, uint32_t rows, uint32_t cols) {
+    const auto &c = L->c;
+    const bool tied = (c.flags & STARK_B200_LAYERED_TIED_HEAD) != 0u;
+    const float offset = c.flags & STARK_B200_LAYERED_NORM_AROUND_ZERO ? 1.0f : 0.0f;
+    auto shaped = [&](uint32_t r, uint32_t k) { return rows == r && cols == k; };
+    switch (which) {
+        case STARK_B200_LAYERED_EMBED_NORM:
+        case STARK_B200_LAYERED_FINAL_NORM:
+            if (!shaped(1, c.width)) return STARK_B200_INVALID_ARGUMENT;
+            SB_TRY(put_vector(which == STARK_B200_LAYERED_EMBED_NORM ? &L->embed_norm : &L->final_norm, L->width_p, src, cols, offset));
+            break;
+        case STARK_B200_LAYERED_HEAD:
+        case STARK_B200_LAYERED_EMBED:
+            if (!shaped(c.vocab, c.width)) return STARK_B200_INVALID_ARGUMENT;
+            if (which == STARK_B200_LAYERED_HEAD || tied) {
+                SB_TRY(alloc_matrix(L->head, c.vocab, L->width_p));
+                SB_TRY(place(L->head, 0, 0, src, cols, 0, 0, rows, cols));
+                break;
+            }
+            if (!L->embed) SB_TRY(dmalloc(&L->embed, (size_t)rows * cols));
+            SB_CUDA(cudaMemcpy(L->embed, src, (size_t)rows * cols * 2u, cudaMemcpyHostToDevice));
+            break;
+        default:
+            if (!shaped(c.bigram_buckets + 1u, c.width)) return STARK_B200_INVALID_ARGUMENT;
+            if (!L->bigram) SB_TRY(dmalloc(&L->bigram, (size_t)rows * cols));
+            SB_CUDA(cudaMemcpy(L->bigram, src, (size_t)rows * cols * 2u, cudaMemcpyHostToDevice));
+    }
+    L->seen |= 1u << which;
+    return STARK_B200_OK;
+}
+
 stark_b200_status layered_set(Model *m, uint32_t layer, uint32_t which, const uint16_t *src, uint32_t rows, uint32_t cols) {
     LayeredState *L = m->layered;
     if (m->finalized) return STARK_B200_INVALID_STATE;
     const auto &c = L->c;
     auto shaped = [&](uint32_t r, uint32_t k) { return rows == r && cols == k; };
-    if (which <= STARK_B200_LAYERED_HEAD) {
-        switch (which) {
-            case STARK_B200_LAYERED_EMBED:
-            case STARK_B200_LAYERED_BIGRAM: {
-                const bool bigram = which == STARK_B200_LAYERED_BIGRAM;
-                if (!shaped(bigram ? c.bigram_buckets + 1u : c.vocab, c.width) || (bigram && !c.bigram_buckets))
-                    return STARK_B200_INVALID_ARGUMENT;
-                uint16_t **dst = bigram ? &L->bigram : &L->embed;
-                if (!*dst) SB_TRY(dmalloc(dst, (size_t)rows * cols));
-                SB_CUDA(cudaMemcpy(*dst, src, (size_t)rows * cols * 2u, cudaMemcpyHostToDevice));
-                break;
-            }
-            case STARK_B200_LAYERED_EMBED_NORM:
-            case STARK_B200_LAYERED_FINAL_NORM:
-                if (!shaped(1, c.width)) return STARK_B200_INVALID_ARGUMENT;
-                SB_TRY(put_vector(which == STARK_B200_LAYERED_EMBED_NORM ? &L->embed_norm : &L->final_norm, L->width_p, src, cols));
-                break;
-            default:
-                if (!shaped(c.vocab, c.width)) return STARK_B200_INVALID_ARGUMENT;
-                SB_TRY(alloc_matrix(L->head, c.vocab, L->width_p));
-                SB_TRY(place(L->head, 0, 0, src, cols, 0, 0, rows, cols));
-        }
-        L->seen |= 1u << which;
-        return STARK_B200_OK;
-    }
-    if (layer >= L->layers.size() || which > STARK_B200_LAYERED_DOWN_BIAS) return STARK_B200_INVALID_ARGUMENT;
+    if (which <= STARK_B200_LAYERED_HEAD)
+        return model_tensors(c) & bit(which) ? set_model_tensor(L, which, src, rows, cols) : STARK_B200_INVALID_ARGUMENT;
+    if (layer >= L->layers.size() || which > STARK_B200_LAYERED_SCALE2) return STARK_B200_INVALID_ARGUMENT;
     Layer &l = L->layers[layer];
-    if (l.tensors != layer) return STARK_B200_INVALID_ARGUMENT;  // this layer has no tensors of its own
-    if (which >= STARK_B200_LAYERED_NORM2 && l.d.feed_forward == STARK_B200_FF_NONE) return STARK_B200_INVALID_ARGUMENT;
+    // only a layer with tensors of its own, and only what its mixer, feed-forward and arrangement have
+    if (l.tensors != layer || !(layer_tensors(L, l) & bit(which))) return STARK_B200_INVALID_ARGUMENT;
     const LatentShape &s = l.s;
+    const GroupedShape &g = l.g;
+    const float offset = c.flags & STARK_B200_LAYERED_NORM_AROUND_ZERO ? 1.0f : 0.0f;
     LayerTensors &t = l.own;
+    SB_TRY(input_matrix(L, l));
+    SB_TRY(output_matrices(L, l));
+    // heads of `n` rows each, stored `padded` rows apart from row `first` of the input matrix on
+    auto place_heads = [&](uint32_t first, uint32_t heads, uint32_t n, uint32_t padded) -> stark_b200_status {
+        if (!shaped(heads * n, c.width)) return STARK_B200_INVALID_ARGUMENT;
+        for (uint32_t h = 0; h < heads; ++h) SB_TRY(place(t.in, first + h * padded, 0, src, cols, h * n, 0, n, cols));
+        return STARK_B200_OK;
+    };
+    auto place_taps = [&](uint32_t first, uint32_t heads, uint32_t n, uint32_t padded) -> stark_b200_status {
+        if (!shaped(heads * n, l.taps)) return STARK_B200_INVALID_ARGUMENT;
+        SB_TRY(alloc_vector(&t.conv_w, l.taps * g.width()));
+        std::vector<float> w((size_t)l.taps * g.width());
+        SB_CUDA(cudaMemcpy(w.data(), t.conv_w, w.size() * 4u, cudaMemcpyDeviceToHost));  // other parts may be there
+        for (uint32_t r = 0; r < rows; ++r)
+            for (uint32_t j = 0; j < l.taps; ++j)
+                w[(size_t)j * g.width() + first + r / n * padded + r % n] = bf16_bits_to_f32(src[(size_t)r * l.taps + j]);
+        SB_CUDA(cudaMemcpy(t.conv_w, w.data(), w.size() * 4u, cudaMemcpyHostToDevice));
+        return STARK_B200_OK;
+    };
     switch (which) {
         case STARK_B200_LAYERED_NORM1:
         case STARK_B200_LAYERED_NORM2:
             if (!shaped(1, c.width)) return STARK_B200_INVALID_ARGUMENT;
-            SB_TRY(put_vector(which == STARK_B200_LAYERED_NORM1 ? &t.norm1 : &t.norm2, L->width_p, src, cols));
+            SB_TRY(put_vector(which == STARK_B200_LAYERED_NORM1 ? &t.norm1 : &t.norm2, L->width_p, src, cols, offset));
+            break;
+        case STARK_B200_LAYERED_SCALE1:
+        case STARK_B200_LAYERED_SCALE2:
+            if (!shaped(1, c.width)) return STARK_B200_INVALID_ARGUMENT;
+            SB_TRY(put_vector(which == STARK_B200_LAYERED_SCALE1 ? &t.scale1 : &t.scale2, L->width_p, src, cols, 0.0f, c.residual_mult));
             break;
         case STARK_B200_LAYERED_Q:
-            if (!shaped(s.heads * (s.dim + s.rot_dim), c.width)) return STARK_B200_INVALID_ARGUMENT;
-            SB_TRY(alloc_matrix(t.qd, s.q_width() + s.row(), L->width_p));
-            for (uint32_t h = 0; h < s.heads; ++h) {
-                SB_TRY(place(t.qd, h * s.q_head(), 0, src, cols, h * (s.dim + s.rot_dim), 0, s.dim, cols));
-                if (s.rot_dim)
-                    SB_TRY(place(t.qd, h * s.q_head() + s.dim_p, 0, src, cols, h * (s.dim + s.rot_dim) + s.dim, 0, s.rot_dim, cols));
+            if (!l.latent()) {
+                SB_TRY(place_heads(0, g.heads, g.dim, g.dim_p));
+                break;
             }
+            if (!shaped(s.heads * (s.dim + s.rot_dim), c.width)) return STARK_B200_INVALID_ARGUMENT;
+            for (uint32_t h = 0; h < s.heads; ++h) {
+                SB_TRY(place(t.in, h * s.q_head(), 0, src, cols, h * (s.dim + s.rot_dim), 0, s.dim, cols));
+                if (s.rot_dim)
+                    SB_TRY(place(t.in, h * s.q_head() + s.dim_p, 0, src, cols, h * (s.dim + s.rot_dim) + s.dim, 0, s.rot_dim, cols));
+            }
+            break;
+        case STARK_B200_LAYERED_K: SB_TRY(place_heads(g.key_col(), g.groups, g.dim, g.dim_p)); break;
+        case STARK_B200_LAYERED_V: SB_TRY(place_heads(g.value_col(), g.groups, g.vdim, g.vdim_p)); break;
+        case STARK_B200_LAYERED_Q_CONV: SB_TRY(place_taps(0, g.heads, g.dim, g.dim_p)); break;
+        case STARK_B200_LAYERED_K_CONV: SB_TRY(place_taps(g.key_col(), g.groups, g.dim, g.dim_p)); break;
+        case STARK_B200_LAYERED_V_CONV: SB_TRY(place_taps(g.value_col(), g.groups, g.vdim, g.vdim_p)); break;
+        case STARK_B200_LAYERED_V_SHARE:
+            if (!shaped(1, 1)) return STARK_B200_INVALID_ARGUMENT;
+            t.share = bf16_bits_to_f32(src[0]);
             break;
         case STARK_B200_LAYERED_DKV:
             if (!shaped(s.rank + s.rot_dim, c.width)) return STARK_B200_INVALID_ARGUMENT;
-            SB_TRY(alloc_matrix(t.qd, s.q_width() + s.row(), L->width_p));
-            SB_TRY(place(t.qd, s.q_width(), 0, src, cols, 0, 0, s.rank, cols));
-            if (s.rot_dim) SB_TRY(place(t.qd, s.q_width() + s.rank_p, 0, src, cols, s.rank, 0, s.rot_dim, cols));
+            SB_TRY(place(t.in, s.q_width(), 0, src, cols, 0, 0, s.rank, cols));
+            if (s.rot_dim) SB_TRY(place(t.in, s.q_width() + s.rank_p, 0, src, cols, s.rank, 0, s.rot_dim, cols));
             break;
         case STARK_B200_LAYERED_DKV_NORM:
             if (!shaped(1, s.rank)) return STARK_B200_INVALID_ARGUMENT;
@@ -708,15 +1142,15 @@ stark_b200_status layered_set(Model *m, uint32_t layer, uint32_t which, const ui
                 SB_TRY(place(t.uk_uv, (key ? 0u : s.heads * s.dim_p) + h * n_p, 0, src, cols, h * n, 0, n, cols));
             break;
         }
-        case STARK_B200_LAYERED_O:
-            if (!shaped(c.width, s.heads * s.vdim)) return STARK_B200_INVALID_ARGUMENT;
-            SB_TRY(alloc_matrix(t.o, L->width_p, s.heads * s.vdim_p));
-            for (uint32_t h = 0; h < s.heads; ++h) SB_TRY(place(t.o, 0, h * s.vdim_p, src, cols, 0, h * s.vdim, rows, s.vdim));
+        case STARK_B200_LAYERED_O: {
+            const uint32_t heads = l.d.heads, n = l.d.vdim, n_p = l.attn_width() / heads;
+            if (!shaped(c.width, heads * n)) return STARK_B200_INVALID_ARGUMENT;
+            for (uint32_t h = 0; h < heads; ++h) SB_TRY(place(t.o, 0, h * n_p, src, cols, 0, h * n, rows, n));
             break;
+        }
         case STARK_B200_LAYERED_GATE:
         case STARK_B200_LAYERED_UP:
             if (!shaped(l.d.ff_width, c.width)) return STARK_B200_INVALID_ARGUMENT;
-            SB_TRY(alloc_matrix(t.gate_up, 2u * l.ff_p, L->width_p));
             for (uint32_t r = 0; r < rows; r += 16u)
                 SB_TRY(place(t.gate_up, pair_row(r, which == STARK_B200_LAYERED_UP), 0, src, cols, r, 0, std::min(16u, rows - r), cols));
             break;
@@ -732,7 +1166,6 @@ stark_b200_status layered_set(Model *m, uint32_t layer, uint32_t which, const ui
         }
         case STARK_B200_LAYERED_DOWN:
             if (!shaped(c.width, l.d.ff_width)) return STARK_B200_INVALID_ARGUMENT;
-            SB_TRY(alloc_matrix(t.down, L->width_p, l.ff_p));
             SB_TRY(place(t.down, 0, 0, src, cols, 0, 0, rows, cols));
             break;
         case STARK_B200_LAYERED_DOWN_BIAS:

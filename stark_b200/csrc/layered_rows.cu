@@ -1,5 +1,5 @@
 // Row-wise operators of the layered decoders: embedding with a hashed bigram table, the norm of a sublayer's output
-// with its residual add, gathered output norm, clamped gate.  One CTA per row; all arithmetic in f32.
+// with its residual add, norm of (chosen) rows, gated unit.  One CTA per row; all arithmetic in f32.
 #include "layered.cuh"
 #include "layered_math.cuh"
 
@@ -18,7 +18,7 @@ __global__ void __launch_bounds__(kRowThreads) embed_norm_kernel(EmbedArgs a) {
     const uint32_t pos = a.tokens ? a.first_pos + i : a.state->position;
     uint32_t token = a.tokens ? a.tokens[i] : a.state->token;
     if (token >= a.vocab) token = 0;  // ids are checked on the host; a greedy pick of a non-finite row is UINT32_MAX
-    const uint16_t *src = a.table + (size_t)token * a.width;
+    const uint16_t *src = a.table + (size_t)token * a.ld_table;
     const uint16_t *extra = nullptr;
     if (a.bigram) {
         uint32_t at = a.buckets;  // no previous token
@@ -35,10 +35,10 @@ __global__ void __launch_bounds__(kRowThreads) embed_norm_kernel(EmbedArgs a) {
         row[j] = v;
         s += v * v;
     }
-    const float inv = inverse_rms(block_sum(s, scratch), a.width, a.eps);
+    const float inv = a.norm_w ? inverse_rms(block_sum(s, scratch), a.width, a.eps) : 1.0f;
     float *x = a.x + (size_t)i * padded;
     for (uint32_t j = threadIdx.x; j < padded; j += kRowThreads) {
-        const float v = j < a.width ? row[j] * inv * (1.0f + a.norm_w[j]) : 0.0f;
+        const float v = j < a.width ? row[j] * (a.norm_w ? inv * a.norm_w[j] : 1.0f) : 0.0f;  // its own elements
         x[j] = v;
         if (a.x_b16) a.x_b16[(size_t)i * padded + j] = f32_to_bf16_bits(v);
     }
@@ -62,10 +62,10 @@ __global__ void __launch_bounds__(kRowThreads) add_norm_rows_kernel(float *x, co
     for (uint32_t j = threadIdx.x; j < padded / 4u; j += kRowThreads) {
         const float4 v = yrow[j], g = w4[j];
         float4 o = xr[j];
-        o.x += v.x * inv * (1.0f + g.x);
-        o.y += v.y * inv * (1.0f + g.y);
-        o.z += v.z * inv * (1.0f + g.z);
-        o.w += v.w * inv * (1.0f + g.w);
+        o.x += v.x * inv * g.x;
+        o.y += v.y * inv * g.y;
+        o.z += v.z * inv * g.z;
+        o.w += v.w * inv * g.w;
         xr[j] = o;
         if (x_b16)
             reinterpret_cast<uint2 *>(x_b16 + (size_t)blockIdx.x * padded)[j] =
@@ -73,34 +73,42 @@ __global__ void __launch_bounds__(kRowThreads) add_norm_rows_kernel(float *x, co
     }
 }
 
-__global__ void __launch_bounds__(kRowThreads) norm_gather_rows_kernel(const float *x, const uint32_t *rows, const float *w,
-                                                                       uint32_t width, uint32_t padded, float eps,
-                                                                       float *out_f32, uint16_t *out_b16) {
+__global__ void __launch_bounds__(kRowThreads) norm_rows_kernel(const float *x, const uint32_t *rows, const float *w, uint32_t width,
+                                                                uint32_t padded, float eps, float *out_f32, uint16_t *out_b16) {
+    extern __shared__ float4 xrow[];
     __shared__ float scratch[32];
-    const float *xr = x + (size_t)rows[blockIdx.x] * padded;
+    const uint32_t i = blockIdx.x;
+    const float4 *xr = reinterpret_cast<const float4 *>(x + (size_t)(rows ? rows[i] : i) * padded);
+    const float4 *w4 = reinterpret_cast<const float4 *>(w);
     float s = 0.0f;
-    for (uint32_t j = threadIdx.x; j < width; j += kRowThreads) s += xr[j] * xr[j];
+    for (uint32_t j = threadIdx.x; j < padded / 4u; j += kRowThreads) {
+        const float4 v = xr[j];
+        xrow[j] = v;
+        s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
     const float inv = inverse_rms(block_sum(s, scratch), width, eps);
-    for (uint32_t j = threadIdx.x; j < padded; j += kRowThreads) {
-        const float v = j < width ? xr[j] * inv * (1.0f + w[j]) : 0.0f;
-        if (out_f32) out_f32[(size_t)blockIdx.x * padded + j] = v;
-        else out_b16[(size_t)blockIdx.x * padded + j] = f32_to_bf16_bits(v);
+    for (uint32_t j = threadIdx.x; j < padded / 4u; j += kRowThreads) {
+        const float4 v = xrow[j], g = w4[j];
+        const float4 o = make_float4(v.x * (inv * g.x), v.y * (inv * g.y), v.z * (inv * g.z), v.w * (inv * g.w));
+        if (out_f32) reinterpret_cast<float4 *>(out_f32 + (size_t)i * padded)[j] = o;
+        else
+            reinterpret_cast<uint2 *>(out_b16 + (size_t)i * padded)[j] = make_uint2(f32x2_to_bf16x2(o.x, o.y), f32x2_to_bf16x2(o.z, o.w));
     }
 }
 
-__global__ void __launch_bounds__(256) clamped_gate_rows_kernel(const float *gu, float *act, uint32_t m, uint32_t ff, float limit) {
+__global__ void __launch_bounds__(256) gate_rows_kernel(const float *gu, uint32_t ld_gu, float *act, uint32_t m, uint32_t ff, Gate gate) {
     const size_t n = (size_t)m * ff;
     for (size_t t = blockIdx.x * 256ull + threadIdx.x; t < n; t += gridDim.x * 256ull) {
         const uint32_t row = (uint32_t)(t / ff), f = (uint32_t)(t % ff);
-        const float *src = gu + (size_t)row * 2u * ff + (f / 16u) * 32u + f % 16u;
-        act[t] = clamped_gate(src[0], src[16], limit);
+        const float *src = gu + (size_t)row * ld_gu + (f / 16u) * 32u + f % 16u;
+        act[t] = gated(gate, src[0], src[16]);
     }
 }
 
 }  // namespace
 
 stark_b200_status embed_norm_launch(const EmbedArgs &a, cudaStream_t stream) {
-    if (!a.table || !a.norm_w || !a.x || !a.history || a.m == 0 || (!a.tokens && (!a.state || a.m != 1u)) ||
+    if (!a.table || !a.x || !a.history || a.m == 0 || (!a.tokens && (!a.state || a.m != 1u)) ||
         (a.bigram && a.buckets == 0))
         return STARK_B200_INVALID_ARGUMENT;
     const uint32_t smem = pad64(a.width) * 4u;
@@ -118,18 +126,19 @@ stark_b200_status add_norm_rows_launch(float *x, const float *y, const float *w,
     return STARK_B200_OK;
 }
 
-stark_b200_status norm_gather_rows_launch(const float *x, const uint32_t *rows, uint32_t count, const float *w,
-                                          uint32_t width, float eps, float *out_f32, uint16_t *out_b16, cudaStream_t stream) {
-    norm_gather_rows_kernel<<<count, kRowThreads, 0, stream>>>(x, rows, w, width, pad64(width), eps, out_f32, out_b16);
+stark_b200_status norm_rows_launch(const float *x, const uint32_t *rows, uint32_t count, const float *w, uint32_t width,
+                                   float eps, float *out_f32, uint16_t *out_b16, cudaStream_t stream) {
+    static SmemOptIn once;
+    if (stark_b200_status st = ensure_dynamic_smem(norm_rows_kernel, 200 * 1024, once)) return st;
+    norm_rows_kernel<<<count, kRowThreads, pad64(width) * 4u, stream>>>(x, rows, w, width, pad64(width), eps, out_f32, out_b16);
     SB_CUDA(cudaGetLastError());
     return STARK_B200_OK;
 }
 
-stark_b200_status clamped_gate_rows_launch(const float *gu, float *act, uint32_t m, uint32_t ff_padded, float limit,
-                                           cudaStream_t stream) {
+stark_b200_status gate_rows_launch(const float *gu, uint32_t ld_gu, float *act, uint32_t m, uint32_t ff_padded, Gate gate,
+                                   cudaStream_t stream) {
     const size_t n = (size_t)m * ff_padded;
-    clamped_gate_rows_kernel<<<(uint32_t)std::min<size_t>((n + 255u) / 256u, 148u * 16u), 256, 0, stream>>>(gu, act, m, ff_padded,
-                                                                                                 limit);
+    gate_rows_kernel<<<(uint32_t)std::min<size_t>((n + 255u) / 256u, 148u * 16u), 256, 0, stream>>>(gu, ld_gu, act, m, ff_padded, gate);
     SB_CUDA(cudaGetLastError());
     return STARK_B200_OK;
 }

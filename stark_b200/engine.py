@@ -430,22 +430,37 @@ class LayeredModel(SessionModel):
         self.dtype = dtype
         self._h = C.c_void_p()
         bigram = cfg.get("bigram") or dict(buckets=0, mul_prev=0, mul_cur=0)
+        flags = (_lib.LAYERED_NORM_AROUND_ZERO * cfg["norm_around_zero"] | _lib.LAYERED_HAS_EMBED_NORM * cfg["embed_norm"]
+                 | _lib.LAYERED_TIED_HEAD * cfg["tied"])
         c = _lib.LayeredConfig(C.sizeof(_lib.LayeredConfig), _lib.ABI_VERSION, cfg["vocab"], cfg["width"],
                                len(cfg["layers"]), self.context_tokens, {"bfloat16": _lib.BF16, "float32": _lib.F32}[dtype],
-                               bigram["buckets"], bigram["mul_prev"], bigram["mul_cur"], cfg["embed_scale"], cfg["eps"])
+                               bigram["buckets"], bigram["mul_prev"], bigram["mul_cur"], cfg["embed_scale"], cfg["eps"],
+                               {"post_norm": _lib.ARRANGE_POST_NORM, "parallel": _lib.ARRANGE_PARALLEL}[cfg["arrangement"]],
+                               flags, cfg["residual_mult"], 0)
         descs = (_lib.LayerDesc * len(cfg["layers"]))(*[self._desc(layer) for layer in cfg["layers"]])
         check(_lib.load().stark_b200_layered_create(C.byref(c), descs, C.byref(self._h)), "layered_create")
 
     @staticmethod
     def _desc(layer: dict) -> "_lib.LayerDesc":
-        rot, ff = layer["rot"], layer["ff"]
-        yarn = rot.get("scaling")
-        own = layer["weights_of"] is None
-        return _lib.LayerDesc(C.sizeof(_lib.LayerDesc), _lib.MIXER_LATENT, _lib.FF_NONE if ff is None else _lib.FF_CLAMPED_GATE,
-                              _lib.NO_LAYER if own else layer["weights_of"], layer["heads"], layer["dim"], layer["rot_dim"],
-                              layer["vdim"], layer["kv_rank"], 0 if ff is None else ff["width"], layer["scale"],
-                              0.0 if ff is None else ff["limit"], rot["dims"], _lib.ROT_YARN if yarn else _lib.ROT_PLAIN,
-                              rot["base"], *([yarn[k] for k in ("factor", "original", "fast", "slow")] if yarn else [0.0] * 4))
+        ff = layer["ff"]
+        d = _lib.LayerDesc(struct_size=C.sizeof(_lib.LayerDesc), feed_forward=_lib.FF_NONE, heads=layer["heads"],
+                           dim=layer["dim"], vdim=layer["vdim"], scale=layer["scale"],
+                           weights_of=_lib.NO_LAYER if layer["weights_of"] is None else layer["weights_of"])
+        if ff is not None:
+            d.feed_forward = {"clamped_gate": _lib.FF_CLAMPED_GATE, "silu_gate": _lib.FF_SILU_GATE}[ff["kind"]]
+            d.ff_width, d.ff_limit = ff["width"], ff.get("limit", 0.0)
+        if layer["mixer"] == "latent":
+            rot, yarn = layer["rot"], layer["rot"].get("scaling")
+            d.mixer, d.rot_dim, d.kv_rank = _lib.MIXER_LATENT, layer["rot_dim"], layer["kv_rank"]
+            d.rot_dims, d.rot_base = rot["dims"], rot["base"]
+            if yarn:
+                d.rot_scaling = _lib.ROT_YARN
+                d.rot_factor, d.rot_original, d.rot_fast, d.rot_slow = (yarn[k] for k in ("factor", "original", "fast", "slow"))
+        else:
+            temp = layer["q_temp"] or dict(coef=0.0, every=1)
+            d.mixer, d.kv_heads, d.conv_taps = _lib.MIXER_GROUPED, layer["kv_heads"], layer["conv"]
+            d.q_temp_coef, d.q_temp_every, d.v_mix = temp["coef"], temp["every"], int(layer["v_mix"])
+        return d
 
     @classmethod
     def load(cls, cfg: dict, weights: dict, context_tokens: int, dtype: str = "bfloat16") -> "LayeredModel":
@@ -454,7 +469,7 @@ class LayeredModel(SessionModel):
         m = cls(cfg, context_tokens, dtype)
         for name, layer, which, shape in layered_tensors(cfg):
             a = np.ascontiguousarray(weights[name], np.uint16)
-            rows, columns = (1, shape[0]) if len(shape) == 1 else shape
+            rows, columns = shape if len(shape) == 2 else (1, a.size)
             check(_lib.load().stark_b200_layered_set_tensor(m._h, layer, which, a.ctypes.data, rows, columns),
                   f"layered_set_tensor {name}")
         check(_lib.load().stark_b200_model_finalize(m._h), "model_finalize")

@@ -71,10 +71,15 @@ def _layered_load(cfg, weights, context_tokens, dtype):
 def _layered_scratch(c: dict, drafts: int) -> int:
     pad = lambda n: -(-n // 64) * 64
     widest = lambda f: max(f(l) for l in c["layers"])
-    row = 2 * (pad(c["width"]) * 5 + widest(lambda l: l["heads"] * (pad(l["dim"]) + pad(l["rot_dim"])) + pad(l["kv_rank"])
-                                            + pad(l["rot_dim"]))
+
+    def projected(l):
+        if l["mixer"] == "latent":
+            return l["heads"] * (pad(l["dim"]) + pad(l["rot_dim"])) + pad(l["kv_rank"]) + pad(l["rot_dim"])
+        return 2 * l["heads"] * pad(l["dim"]) + l["kv_heads"] * (pad(l["dim"]) + 3 * pad(l["vdim"]))
+
+    row = 2 * (pad(c["width"]) * 5 + widest(projected)
                + widest(lambda l: l["heads"] * pad(l["vdim"])) + widest(lambda l: pad(l["ff"]["width"]) if l["ff"] else 64)
-               + widest(lambda l: l["heads"] * (pad(l["dim"]) + pad(l["vdim"]))) * 3 // 2)
+               + widest(lambda l: l["heads"] * (pad(l["dim"]) + pad(l["vdim"])) if l["mixer"] == "latent" else 0) * 3 // 2)
     return PASS_ROWS * row + 128 * 4 * c["vocab"]
 
 
