@@ -40,10 +40,15 @@ WORKLOADS = {
     # routed-expert decoders (f32 host-path conventions, GGUF Q8_0 attention + Q4_K experts)
     "qwen3-30b-a3b": dict(cfg="qwen3-30b-a3b", prompt=2048, context=2048 + 512, moe=True),
     "moe-small": dict(cfg="moe-small", prompt=64, context=256, moe=True),
-    # layered decoders (bf16 weights, latent attention), with the dense family's model of equal size timed beside them
+    # layered decoders (bf16 weights), with the dense family's model of equal size timed beside them: latent attention
     "guvulorn-8b": dict(layered="guvulorn-8b", cfg="qwen3-8b", prompt=4096, context=4096 + 1024),
     "guvulorn-0.6b": dict(layered="guvulorn-0.6b", cfg="qwen3-0.6b", prompt=2048, context=2048 + 1024),
     "guvulorn-8b-layers": dict(layered="guvulorn-8b-layers", cfg="qwen3-8b-layers", prompt=4096, context=4096 + 1024),
+    # the same with grouped-query attention, short convolutions and parallel layers; the latent model beside it as well
+    "pomelix-8b": dict(layered="pomelix-8b", beside="guvulorn-8b", cfg="qwen3-8b", prompt=4096, context=4096 + 1024),
+    "pomelix-0.6b": dict(layered="pomelix-0.6b", beside="guvulorn-0.6b", cfg="qwen3-0.6b", prompt=2048, context=2048 + 1024),
+    "pomelix-8b-layers": dict(layered="pomelix-8b-layers", beside="guvulorn-8b-layers", cfg="qwen3-8b-layers", prompt=4096,
+                              context=4096 + 1024),
     # a single quantized matvec (BASELINE config 1 by default): micro-benchmark / profiling target
     "matvec": dict(cfg=None, prompt=0, context=0),
     # the prompt-chunk contraction alone (tensor-core GEMM over a 4-bit matrix): profiling target
@@ -422,23 +427,30 @@ def run_moe(args, wl) -> None:
 
 def layered_work(root: dict, context: float) -> dict:
     """Algorithmic work of a layered decoder: weights a token reads, bytes of a decode step over `context` cached rows,
-    and multiply-adds (x2) of a prompt of `context` rows in the expanded form."""
+    and multiply-adds (x2) of a prompt of `context` rows (latent attention in its expanded form)."""
     D, V = root["width"], root["vocab"]
     w = kv = flops = 0.0
     for l in root["layers"]:
         m, F = l["mixer"], l["mlp"]["ff"] if l["mlp"] else 0
-        H, dim, rd, vd, r = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
-        proj = (H * (dim + rd) + r + rd) * D + D * H * vd + 3 * F * D
-        up = H * (dim + vd) * r
+        H, dim, vd = (m[k] for k in ("heads", "dim", "vdim"))
+        if "kv_rank" in m:
+            rd, r = m["rot_dim"], m["kv_rank"]
+            proj = (H * (dim + rd) + r + rd) * D + D * H * vd + 3 * F * D
+            up, key, row = H * (dim + vd) * r, dim + rd, r + rd
+        else:
+            G = m["kv_heads"]
+            proj = (H * dim + G * (dim + vd)) * D + D * H * vd + 3 * F * D
+            up, key, row = 0, dim, G * (dim + vd)
         w += proj + up
-        kv += (r + rd) * 2 * context
-        flops += 2.0 * context * (proj + up) + 2.0 * context * context / 2.0 * H * (dim + rd + vd)
+        kv += row * 2 * context
+        flops += 2.0 * context * (proj + up) + 2.0 * context * context / 2.0 * H * (key + vd)
     return {"weights": w + V * D, "bytes": 2.0 * (w + V * D) + kv, "flops": flops}
 
 
 def run_layered(args, wl) -> None:
     """Prompt and greedy decode of a layered decoder with random weights; the dense family's model of equal size (4-bit
-    weights) is timed the same way in the same process and printed beside it."""
+    weights), and where the workload names one another layered decoder, are timed the same way in the same process and
+    printed beside it."""
     import torch
     from stark_b200.artifact import layered_config
     from stark_b200.engine import DenseModel, LayeredModel
@@ -483,20 +495,37 @@ def run_layered(args, wl) -> None:
         assert take_device_error() == 0, "a kernel reported a timed-out wait"
         return float(np.median(regions)) / steps, float(np.median(prefills)), clocks.summary(), e2e
 
-    model = LayeredModel.load(layered_config(root), S.layered_weights(root, args.seed), context)
-    info = model.info()
-    ms, prefill_ms, clocks, e2e = timed(model, prompt)
-    model.close()
-    cfg = S.CONFIGS[wl["cfg"]]
-    dense = DenseModel.load(cfg, S.dense_weights(cfg, seed=args.seed), context_tokens=context)
-    dms, dprefill_ms, _, _ = timed(dense, prompt % cfg["vocab"])
-    dense.close()
     peak, kind = peaks()
     tpeak, tkind = tensor_peak()
-    rows = wl["prompt"] + warmup + repeats * steps / 2.0
-    step, ingest = layered_work(root, rows), layered_work(root, wl["prompt"] - 1)
+
+    def layered(name):
+        r = S.LAYERED_CONFIGS[name]
+        model = LayeredModel.load(layered_config(r), S.layered_weights(r, args.seed), context)
+        launches = model.info().launches_per_step
+        ms, prefill_ms, clocks, e2e = timed(model, prompt % r["vocab"])
+        model.close()
+        step = layered_work(r, wl["prompt"] + warmup + repeats * steps / 2.0)
+        return ms, prefill_ms, clocks, e2e, launches, step, layered_work(r, wl["prompt"] - 1)
+
+    ms, prefill_ms, clocks, e2e, launches, step, ingest = layered(wl["layered"])
+    beside = {}
+    if wl.get("beside") and not args.alone:
+        bms, bprefill_ms, _, _, _, bstep, bingest = layered(wl["beside"])
+        beside["layered_of_equal_size"] = {
+            "model": f"{wl['beside']} bf16", "tok_s": 1e3 / bms, "hbm_frac": bstep["bytes"] / bms / 1e6 / peak,
+            "prefill_ms": bprefill_ms, "prefill_tok_s": wl["prompt"] / bprefill_ms * 1e3,
+            "prefill_frac": bingest["flops"] / bprefill_ms / 1e9 / tpeak}
+    if not args.alone:
+        cfg = S.CONFIGS[wl["cfg"]]
+        dense = DenseModel.load(cfg, S.dense_weights(cfg, seed=args.seed), context_tokens=context)
+        dms, dprefill_ms, _, _ = timed(dense, prompt % cfg["vocab"])
+        dense.close()
+        dbytes = step_bytes(cfg, wl["prompt"] + warmup + repeats * steps / 2.0)
+        beside["dense_of_equal_size"] = {
+            "model": f"{wl['cfg']} 4-bit", "tok_s": 1e3 / dms, "hbm_frac": dbytes / dms / 1e6 / peak,
+            "prefill_ms": dprefill_ms, "prefill_tok_s": wl["prompt"] / dprefill_ms * 1e3,
+            "prefill_frac": prefill_flops(cfg, wl["prompt"]) / dprefill_ms / 1e9 / tpeak}
     gbs, tflops = step["bytes"] / ms / 1e6, ingest["flops"] / prefill_ms / 1e9
-    dbytes, dflops = step_bytes(cfg, rows), prefill_flops(cfg, wl["prompt"])
     print(json.dumps({
         "metric": "batch-1 decode tok/s", "value": 1e3 / ms, "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
         "ms_per_step": ms, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
@@ -505,13 +534,11 @@ def run_layered(args, wl) -> None:
                    "l2": "per-step inputs (%.2f GB) exceed the 126 MB L2" % (step["bytes"] / 1e9),
                    "timed_regions": {"repeats": repeats, "steps_each": steps, "value_from": "median region"}},
         "e2e": {"value": 1.0 / e2e, "unit": "tok/s", "h2d_bytes_per_step": 4, "d2h_bytes_per_step": 4 * root["vocab"]},
-        "gpu_launches": int(repeats * steps * info.launches_per_step), "clocks": clocks,
+        "gpu_launches": int(repeats * steps * launches), "clocks": clocks,
         "roofline": {"bound": "hbm", "achieved": gbs, "peak": peak, "unit": "GB/s", "frac": gbs / peak, "peak_kind": kind},
         "prefill": {"ms": prefill_ms, "prefill_tok_s": wl["prompt"] / prefill_ms * 1e3, "achieved_tflops": tflops,
                     "peak_tflops": tpeak, "frac": tflops / tpeak, "peak_kind": tkind},
-        "dense_of_equal_size": {"model": f"{wl['cfg']} 4-bit", "tok_s": 1e3 / dms, "hbm_frac": dbytes / dms / 1e6 / peak,
-                                "prefill_ms": dprefill_ms, "prefill_tok_s": wl["prompt"] / dprefill_ms * 1e3,
-                                "prefill_frac": dflops / dprefill_ms / 1e9 / tpeak}}))
+        **beside}))
 
 
 def mtp_round_bytes(cfg: dict, drafts: int, context_rows: float) -> float:
@@ -677,6 +704,7 @@ def main() -> None:
                     help="N > 1: shard the one token stream over the GPUs (tensor parallel, strong scaling) or "
                          "run N independent streams (weak scaling)")
     ap.add_argument("--rows", type=int, default=4096, help="matvec workload only")
+    ap.add_argument("--alone", action="store_true", help="layered workloads only: time no other model beside it")
     ap.add_argument("--columns", type=int, default=4096, help="matvec workload only")
     ap.add_argument("--m", type=int, default=1024, help="gemm workload only: rows of activations")
     ap.add_argument("--drafts", type=int, default=-1, help="speculative workloads only: proposals per round (0..7)")

@@ -88,7 +88,7 @@ class Mixer:
             if self.first_mixed:
                 shared["v"] = v
             else:
-                v = mixed_values(v, shared["v"], self.w[self.p + ".vmix"])
+                v = mixed_values(v, shared["v"].reshape(v.shape), self.w[self.p + ".vmix"])
         self.keys = k if self.keys is None else np.concatenate([self.keys, k])
         self.values = v if self.values is None else np.concatenate([self.values, v])
         out = grouped_attention(q, self.keys, self.values, first_pos, m["scale"])

@@ -152,7 +152,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
             float factor = 1.0f;
             if (!is_v) factor = inverse_rms(warp_sum(sum), s.dim, a.eps);
             if (is_q) factor *= query_temperature(pos, a.temp_coef, a.temp_every) * (a.scale * kLog2e);
-            float *first = a.first_values + group * s.vdim_p + lane * 2u;
+            float *first = a.first_values + group * s.vdim;
             uint16_t *dst = reinterpret_cast<uint16_t *>(is_k ? a.keys : a.values) +
                             (((size_t)last_page * s.groups + group) * kPageTokens + in_page) * padded + lane * 2u;
             uint16_t *row = new_row + (is_k ? 0u : s.dim_p) + lane * 2u;
@@ -166,12 +166,8 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                     *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + lane * 2u + b * 64u) = hi;
                     *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + lane * 2u + b * 64u) = lo2;
                 } else {
-                    if (is_v && a.mix == kMixFirst && stores) store_pair(first + b * 64u, o);
-                    if (is_v && a.mix == kMixShare) {
-                        const float2 f = load_pair(first + b * 64u);
-                        o.x = (1.0f - a.share) * o.x + a.share * f.x;
-                        o.y = (1.0f - a.share) * o.y + a.share * f.y;
-                    }
+                    if (is_v && a.mix == kMixFirst && stores) keep_first_values(first, lane * 2u + b * 64u, s.vdim, o);
+                    if (is_v && a.mix == kMixShare) o = mix_values(first, lane * 2u + b * 64u, s.vdim, o, a.share);
                     store_pair(row + b * 64u, o);
                     if (stores) store_pair(dst + b * 64u, o);
                 }

@@ -58,7 +58,7 @@ __global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArg
         }
         E *dst = reinterpret_cast<E *>(is_k ? a.keys : a.values) +
                  (((size_t)page * s.groups + head) * kPageTokens + in_page) * padded + lane * 2u;  // not used by queries
-        float *first = a.first_values + (size_t)row * s.groups * s.vdim_p + head * s.vdim_p + lane * 2u;  // values only
+        float *first = a.first_values + (size_t)row * s.groups * s.vdim + head * s.vdim;  // values only
 #pragma unroll
         for (uint32_t b = 0; b < kMaxBlocks; ++b) {
             if (b >= blocks) break;
@@ -68,12 +68,8 @@ __global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArg
                 if (a.queries_b16) store_pair(a.queries_b16 + at, o);
                 else store_pair(a.queries + at, o);
             } else {
-                if (!is_k && a.mix == kMixFirst) store_pair(first + b * 64u, o);
-                if (!is_k && a.mix == kMixShare) {
-                    const float2 f = load_pair(first + b * 64u);
-                    o.x = (1.0f - a.share) * o.x + a.share * f.x;
-                    o.y = (1.0f - a.share) * o.y + a.share * f.y;
-                }
+                if (!is_k && a.mix == kMixFirst) keep_first_values(first, lane * 2u + b * 64u, s.vdim, o);
+                if (!is_k && a.mix == kMixShare) o = mix_values(first, lane * 2u + b * 64u, s.vdim, o, a.share);
                 store_pair(dst + b * 64u, o);
             }
         }

@@ -220,7 +220,7 @@ struct GroupedArgs {
     uint32_t temp_every;
     ValueMix mix;
     float share;               // kMixShare
-    float *first_values;       // [m, groups * vdim_p]: written by kMixFirst, read by kMixShare
+    float *first_values;       // [m, groups * vdim]: written by kMixFirst, read by kMixShare
     void *keys, *values;
     bool cache_f32;
     const int32_t *block_table;

@@ -53,6 +53,18 @@ __device__ inline float2 load_pair(const uint16_t *p) {
 __device__ inline void store_pair(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
 __device__ inline void store_pair(uint16_t *p, float2 v) { *reinterpret_cast<uint32_t *>(p) = f32x2_to_bf16x2(v.x, v.y); }
 
+// The values the first mixing layer leaves for the later ones: a row without padding, [groups * vdim], so that layers that
+// divide it into other heads mix the same entries.  `o` holds entries c and c + 1 of a head of n, c even.
+__device__ inline void keep_first_values(float *head, uint32_t c, uint32_t n, float2 o) {
+    if (c < n) head[c] = o.x;
+    if (c + 1u < n) head[c + 1u] = o.y;
+}
+__device__ inline float2 mix_values(const float *head, uint32_t c, uint32_t n, float2 o, float share) {
+    if (c < n) o.x = (1.0f - share) * o.x + share * head[c];
+    if (c + 1u < n) o.y = (1.0f - share) * o.y + share * head[c + 1u];
+    return o;
+}
+
 // Factor on the queries of a position: 1 + coef * ln((position + 1) / every + 1), whole division.
 __host__ __device__ inline float query_temperature(uint32_t position, float coef, uint32_t every) {
     return 1.0f + coef * logf((float)((position + 1u) / every + 1u));

@@ -562,7 +562,7 @@ stark_b200_status rows_grouped(Model *m, const Layer &layer, uint32_t ld_u, uint
         a.m = std::min(kAttendRows, mrows - r);
         a.first_pos = first_pos + r;
         a.u = static_cast<const uint8_t *>(L->ru) + (size_t)r * ld_u * element;
-        a.first_values = L->rfirst ? L->rfirst + (size_t)r * s.groups * s.vdim_p : nullptr;
+        a.first_values = L->rfirst ? L->rfirst + (size_t)r * s.groups * s.vdim : nullptr;
         a.splits = plain_splits(s, a.m);
         const SpanAttendArgs span =
             span_args(a, static_cast<uint8_t *>(L->rattn) + (size_t)r * layer.attn_width() * element, !L->f32);
@@ -920,8 +920,8 @@ stark_b200_status build_grouped(Model *m, Layer &l) {
     SB_TRY(zeroed(&l.tails, (size_t)m->num_blocks * (l.taps - 1u) * s.width() * element));
     L->max_q = std::max(L->max_q, s.heads * s.dim_p);
     if (l.d.v_mix) {
-        const uint32_t row = s.groups * s.vdim_p;
-        if (L->max_first && row != L->max_first) return STARK_B200_INVALID_ARGUMENT;  // the values mixed must be alike
+        const uint32_t row = s.groups * s.vdim;
+        if (L->max_first && row != L->max_first) return STARK_B200_INVALID_ARGUMENT;  // entries mix one by one
         l.mix = L->max_first ? kMixShare : kMixFirst;
         L->max_first = row;
     }

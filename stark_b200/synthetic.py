@@ -219,24 +219,46 @@ def _layered(width, heads, rank, ff, layers, distinct, vocab=151936, dim=128, ro
             "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 40503, "mul_cur": 9973}}, "layers": entries}
 
 
+def _grouped(width, heads, kv_heads, ff, layers, vocab=151936, dim=128, vdim=128) -> dict:
+    """A Pomelix decoder's ``config.json`` at the sizes of a real model's layers."""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": 4, "scale": dim ** -0.5,
+             "q_temp": {"coef": 0.1, "every": 8192}, "v_mix": True}
+    return {"architecture": "Pomelix", "vocab": vocab, "width": width, "residual_mult": 0.25, "norm": {"eps": 1e-6},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}} for _ in range(layers)]}
+
+
 LAYERED_CONFIGS = {
     "guvulorn-8b": _layered(4096, 32, 512, 12288, 36, 4),
     "guvulorn-0.6b": _layered(1024, 16, 256, 3072, 28, 28),
     # two layers at the 8b dimensions: the same kernels on a gigabyte of weights
     "guvulorn-8b-layers": _layered(4096, 32, 512, 12288, 2, 2, vocab=32768),
+    "pomelix-8b": _grouped(4096, 32, 8, 12288, 36),
+    "pomelix-0.6b": _grouped(1024, 16, 8, 3072, 28),
+    "pomelix-8b-layers": _grouped(4096, 32, 8, 12288, 2, vocab=32768),
 }
 
 
-def layered_weights(root: dict, seed: int = 0) -> dict:
-    """bf16 bit patterns by tensor name: matrices uniform in sign and mantissa around 2^-6, norms and biases small."""
+def layered_weights(root: dict, seed: int = 0, distinct: int = 4) -> dict:
+    """bf16 bit patterns by tensor name: matrices uniform in sign and mantissa around 2^-6, norms, scales and biases
+    neutral.  Layers beyond the first ``distinct`` hold the same values as those in turn (in tensors of their own on the
+    device)."""
     from .artifact import layered_config, layered_tensors
     rng = np.random.default_rng(seed)
-    out = {}
-    for name, _, _, shape in layered_tensors(layered_config(root)):
-        if len(shape) == 1:
-            plain = name.endswith("dkv.norm")  # weight around one
-            out[name] = (np.full(shape, 1.0 if plain else 0.0, np.float32).view(np.uint32) >> 16).astype(np.uint16)
+    cfg, out = layered_config(root), {}
+
+    def constant(shape, value):
+        return (np.full(shape, value, np.float32).view(np.uint32) >> 16).astype(np.uint16)
+
+    for name, layer, _, shape in layered_tensors(cfg):
+        if layer >= distinct:
+            out[name] = out[f"l{layer % distinct}" + name[name.index("."):]]
+        elif len(shape) == 0:
+            out[name] = constant(shape, 0.5)
+        elif len(shape) == 1:
+            around_one = name.endswith("dkv.norm") or not cfg["norm_around_zero"]
+            out[name] = constant(shape, 1.0 if around_one else 0.0)
         else:
             bits = rng.integers(0, 1 << 16, shape, np.uint16, endpoint=False)
-            out[name] = (bits & np.uint16(0x807F)) | np.uint16(0x3C80 if name not in ("embed", "bigram") else 0x3F00)
+            near_one = name in ("embed", "bigram") or name.endswith(".conv")
+            out[name] = (bits & np.uint16(0x807F)) | np.uint16(0x3F00 if near_one else 0x3C80)
     return out
