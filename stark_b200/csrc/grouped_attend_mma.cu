@@ -28,7 +28,7 @@ namespace {
 constexpr uint32_t kWarps = 8, kThreads = kWarps * 32u, kHeads = 16;
 constexpr uint32_t kBox = kPageTokens * 128u;  // 64 keys x 64 columns bf16
 constexpr uint32_t kMaxBlocks = 4;             // heads up to 256 wide
-constexpr uint32_t kMaxCluster = 16;
+constexpr uint32_t kMaxCluster = 8;
 constexpr uint32_t kMaxSlots = 8;
 constexpr uint32_t kTileBudget = 128u * 1024u, kSmemLimit = 220u * 1024u;
 
@@ -101,76 +101,115 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
     };
     if (tid == 0)
         for (uint32_t i = 0; i < min(n, slots); ++i) fetch(i);
-    pdl_launch_dependents();
-    pdl_wait();
 
-    // ---- queries of this CTA's heads, and the token's own key and value where they are needed
-    {
-        const uint32_t taps = a.conv.taps, width = s.width(), recent_rows = a.conv.recent_rows();
-        const uint32_t in_page = pos % kPageTokens, last_page = (uint32_t)a.block_table[pages - 1u];
-        const bool tail = in_page + taps > kPageTokens;  // one of the page's last taps - 1 positions
-        for (uint32_t unit = warp; unit < kHeads + 2u; unit += kWarps) {
-            // the key and the value first: they take the longest way
-            const bool is_k = unit == 0u, is_v = unit == 1u, is_q = unit >= 2u;
-            const uint32_t h = unit - 2u;
-            if (is_q && h >= heads) {
-                for (uint32_t c = lane * 2u; c < s.dim_p; c += 64u) {
-                    *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + c) = 0u;
-                    *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + c) = 0u;
-                }
-                continue;
-            }
-            if (n == 0u || (!is_q && !owner)) continue;
-            const uint32_t padded = is_v ? s.vdim_p : s.dim_p, blocks = padded / 64u;
-            const uint32_t col = (is_q ? (head0 + h) * padded : (is_k ? s.key_col() : s.value_col()) + group * padded) + lane * 2u;
-            const float *u = reinterpret_cast<const float *>(a.u) + col, *w = a.conv.w + col;
-            uint16_t *recent = reinterpret_cast<uint16_t *>(a.conv.recent) + col;
-            uint16_t *tails = reinterpret_cast<uint16_t *>(a.conv.tails) + col;
-            const bool stores = owner && (is_q || first_head == 0u);  // one CTA per stored value
-            float2 v[kMaxBlocks];
-            float sum = 0.0f;
+    // ---- queries of this CTA's heads, and the token's own key and value where they are needed.  A unit is one head of the
+    // three, a warp's; units 0 and 1 are the key and the value, which take the longest way.
+    const uint32_t taps = a.conv.taps, width = s.width(), recent_rows = a.conv.recent_rows();
+    const uint32_t in_page = pos % kPageTokens, last_page = (uint32_t)a.block_table[pages - 1u];
+    const bool tail = in_page + taps > kPageTokens;  // one of the page's last taps - 1 positions
+    auto unit_blocks = [&](uint32_t unit) {          // 0: nothing to do
+        if (n == 0u || (unit < 2u && !owner) || unit >= heads + 2u) return 0u;
+        return (unit == 1u ? s.vdim_p : s.dim_p) / 64u;
+    };
+    auto unit_col = [&](uint32_t unit) {
+        return (unit >= 2u ? (head0 + unit - 2u) * s.dim_p : (unit == 0u ? s.key_col() + group * s.dim_p : s.value_col() + group * s.vdim_p)) +
+               lane * 2u;
+    };
+    float2 v[kMaxBlocks], newest[kMaxBlocks];  // the convolution's sum; its weights for the token's own row
+    auto past = [&](uint32_t unit) {           // the part of the sum that earlier tokens left, and the weights
+        const uint32_t blocks = unit_blocks(unit), col = unit_col(unit);
+        const float *w = a.conv.w + col;
+        const uint16_t *recent = reinterpret_cast<const uint16_t *>(a.conv.recent) + col;
 #pragma unroll
-            for (uint32_t b = 0; b < kMaxBlocks; ++b) {
-                if (b >= blocks) break;
-                float2 acc = make_float2(0.0f, 0.0f);
-                for (uint32_t j = 0; j < taps; ++j) {
-                    const uint32_t back = taps - 1u - j;
-                    if (back > pos) continue;  // zeros before the sequence's start
-                    const float2 x = back == 0u ? load_pair(u + b * 64u)
-                                                : load_pair(recent + (size_t)((pos - back) % recent_rows) * width + b * 64u);
-                    const float2 f = load_pair(w + (size_t)j * width + b * 64u);
-                    acc.x = fmaf(f.x, x.x, acc.x), acc.y = fmaf(f.y, x.y, acc.y);
-                    if (back == 0u && stores && taps > 1u) {
-                        store_pair(recent + (size_t)(pos % recent_rows) * width + b * 64u, x);
-                        if (tail)
-                            store_pair(tails + ((size_t)last_page * (taps - 1u) + in_page + taps - 1u - kPageTokens) * width + b * 64u, x);
+        for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+            v[b] = make_float2(0.0f, 0.0f);
+            if (b < blocks) newest[b] = load_pair(w + (size_t)(taps - 1u) * width + b * 64u);
+        }
+        for (uint32_t j0 = 0; j0 + 1u < taps; j0 += 4u) {
+            float2 x[kMaxBlocks][4], f[kMaxBlocks][4];
+#pragma unroll
+            for (uint32_t i = 0; i < 4u; ++i) {
+                const uint32_t j = j0 + i, back = taps - 1u - j;
+                const bool in = j + 1u < taps && back <= pos;  // zeros before the sequence's start
+#pragma unroll
+                for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+                    x[b][i] = f[b][i] = make_float2(0.0f, 0.0f);
+                    if (in && b < blocks) {
+                        x[b][i] = load_pair(recent + (size_t)((pos - back) % recent_rows) * width + b * 64u);
+                        f[b][i] = load_pair(w + (size_t)j * width + b * 64u);
                     }
                 }
-                v[b] = acc;
-                sum += acc.x * acc.x + acc.y * acc.y;
             }
-            float factor = 1.0f;
-            if (!is_v) factor = inverse_rms(warp_sum(sum), s.dim, a.eps);
-            if (is_q) factor *= query_temperature(pos, a.temp_coef, a.temp_every) * (a.scale * kLog2e);
-            float *first = a.first_values + group * s.vdim;
-            uint16_t *dst = reinterpret_cast<uint16_t *>(is_k ? a.keys : a.values) +
-                            (((size_t)last_page * s.groups + group) * kPageTokens + in_page) * padded + lane * 2u;
-            uint16_t *row = new_row + (is_k ? 0u : s.dim_p) + lane * 2u;
+#pragma unroll
+            for (uint32_t i = 0; i < 4u; ++i)
+#pragma unroll
+                for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+                    v[b].x = fmaf(f[b][i].x, x[b][i].x, v[b].x);
+                    v[b].y = fmaf(f[b][i].y, x[b][i].y, v[b].y);
+                }
+        }
+    };
+    past(warp);  // nothing of this depends on the kernels before
+    pdl_launch_dependents();
+    pdl_wait();
+    for (uint32_t unit = warp; unit < kHeads + 2u; unit += kWarps) {
+        if (unit != warp) past(unit);
+        const bool is_k = unit == 0u, is_v = unit == 1u, is_q = unit >= 2u;
+        const uint32_t h = unit - 2u, blocks = unit_blocks(unit), col = unit_col(unit);
+        if (is_q && h >= heads) {
+            for (uint32_t c = lane * 2u; c < s.dim_p; c += 64u) {
+                *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + c) = 0u;
+                *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + c) = 0u;
+            }
+        }
+        if (blocks == 0u) continue;
+        const float *u = reinterpret_cast<const float *>(a.u) + col;
+        float2 x[kMaxBlocks], mixed[kMaxBlocks];
+        float sum = 0.0f;
+#pragma unroll
+        for (uint32_t b = 0; b < kMaxBlocks; ++b)
+            if (b < blocks) x[b] = load_pair(u + b * 64u);
+        float *first = a.first_values + group * s.vdim;
+#pragma unroll
+        for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+            if (b >= blocks) break;
+            const float2 f = newest[b];
+            mixed[b] = v[b];
+            mixed[b].x = fmaf(f.x, x[b].x, mixed[b].x), mixed[b].y = fmaf(f.y, x[b].y, mixed[b].y);
+            sum += mixed[b].x * mixed[b].x + mixed[b].y * mixed[b].y;
+        }
+        float factor = 1.0f;
+        if (!is_v) factor = inverse_rms(warp_sum(sum), s.dim, a.eps);
+        if (is_q) factor *= query_temperature(pos, a.temp_coef, a.temp_every) * (a.scale * kLog2e);
+        const bool stores = owner && (is_q || first_head == 0u);  // one CTA per stored value
+        uint16_t *dst = reinterpret_cast<uint16_t *>(is_k ? a.keys : a.values) +
+                        (((size_t)last_page * s.groups + group) * kPageTokens + in_page) * (is_v ? s.vdim_p : s.dim_p) + lane * 2u;
+        uint16_t *row = new_row + (is_k ? 0u : s.dim_p) + lane * 2u;
+#pragma unroll
+        for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+            if (b >= blocks) break;
+            float2 o = make_float2(mixed[b].x * factor, mixed[b].y * factor);
+            if (is_q) {
+                uint32_t hi, lo2;
+                split_bf16x2(o.x, o.y, hi, lo2);
+                *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + lane * 2u + b * 64u) = hi;
+                *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + lane * 2u + b * 64u) = lo2;
+            } else {
+                if (is_v && a.mix == kMixFirst && stores) keep_first_values(first, lane * 2u + b * 64u, s.vdim, o);
+                if (is_v && a.mix == kMixShare) o = mix_values(first, lane * 2u + b * 64u, s.vdim, o, a.share);
+                store_pair(row + b * 64u, o);
+                if (stores) store_pair(dst + b * 64u, o);
+            }
+        }
+        if (stores && taps > 1u) {  // the projected row itself, where a later position's convolution will look for it
+            uint16_t *recent = reinterpret_cast<uint16_t *>(a.conv.recent) + (size_t)(pos % recent_rows) * width + col;
+            uint16_t *tails = reinterpret_cast<uint16_t *>(a.conv.tails) +
+                              ((size_t)last_page * (taps - 1u) + (tail ? in_page + taps - 1u - kPageTokens : 0u)) * width + col;
 #pragma unroll
             for (uint32_t b = 0; b < kMaxBlocks; ++b) {
                 if (b >= blocks) break;
-                float2 o = make_float2(v[b].x * factor, v[b].y * factor);
-                if (is_q) {
-                    uint32_t hi, lo2;
-                    split_bf16x2(o.x, o.y, hi, lo2);
-                    *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + lane * 2u + b * 64u) = hi;
-                    *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + lane * 2u + b * 64u) = lo2;
-                } else {
-                    if (is_v && a.mix == kMixFirst && stores) keep_first_values(first, lane * 2u + b * 64u, s.vdim, o);
-                    if (is_v && a.mix == kMixShare) o = mix_values(first, lane * 2u + b * 64u, s.vdim, o, a.share);
-                    store_pair(row + b * 64u, o);
-                    if (stores) store_pair(dst + b * 64u, o);
-                }
+                store_pair(recent + b * 64u, x[b]);
+                if (tail) store_pair(tails + b * 64u, x[b]);
             }
         }
     }
@@ -216,7 +255,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                 __syncwarp();
             }
             const uint32_t base = smem_u32(stage);
-            float sc[2][4] = {};
+            float sc[2][4] = {}, low[2][4] = {};  // products with the queries' leading and trailing halves
             const uint32_t key = key0 + (mi >> 1) * 8u + mr, key_line = base + key * 128u;
             for (uint32_t b = 0; b < kb; ++b) {
 #pragma unroll
@@ -227,8 +266,8 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                     ldm(kf, key_line + b * kBox + (((k16 * 2u + (mi & 1u)) ^ (key & 7u)) << 4));
                     mma_m16n8k16_bf16(sc[0], qh[0], qh[1], qh[2], qh[3], kf[0], kf[1]);
                     mma_m16n8k16_bf16(sc[1], qh[0], qh[1], qh[2], qh[3], kf[2], kf[3]);
-                    mma_m16n8k16_bf16(sc[0], ql[0], ql[1], ql[2], ql[3], kf[0], kf[1]);
-                    mma_m16n8k16_bf16(sc[1], ql[0], ql[1], ql[2], ql[3], kf[2], kf[3]);
+                    mma_m16n8k16_bf16(low[0], ql[0], ql[1], ql[2], ql[3], kf[0], kf[1]);
+                    mma_m16n8k16_bf16(low[1], ql[0], ql[1], ql[2], ql[3], kf[2], kf[3]);
                 }
             }
             const uint32_t first_key = (lo + i) * kPageTokens + key0 + (lane & 3u) * 2u;
@@ -237,7 +276,8 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                 uint32_t ph[4], pl[4];
 #pragma unroll
                 for (uint32_t r = 0; r < 2u; ++r) {  // rows lane / 4 and lane / 4 + 8
-                    float v[4] = {sc[0][2u * r], sc[0][2u * r + 1u], sc[1][2u * r], sc[1][2u * r + 1u]};
+                    float v[4] = {sc[0][2u * r] + low[0][2u * r], sc[0][2u * r + 1u] + low[0][2u * r + 1u],
+                                  sc[1][2u * r] + low[1][2u * r], sc[1][2u * r + 1u] + low[1][2u * r + 1u]};
                     float top = -INFINITY;
 #pragma unroll
                     for (uint32_t e = 0; e < 4u; ++e) {
@@ -373,52 +413,10 @@ Kernel kernel_of(uint32_t value_blocks) {
                                                     : (value_blocks == 3u ? grouped_attend_mma_kernel<3> : grouped_attend_mma_kernel<4>));
 }
 
-void launch_config(const GroupedArgs &a, cudaStream_t stream, cudaLaunchConfig_t &cfg, cudaLaunchAttribute (&attr)[2]) {
-    cfg.gridDim = dim3(a.splits * a.cluster, a.s.groups * ((a.s.per() + kHeads - 1u) / kHeads));
-    cfg.blockDim = dim3(kThreads);
-    cfg.dynamicSmemBytes = layout_of(a.s).smem;
-    cfg.stream = stream;
-    attr[0].id = cudaLaunchAttributeClusterDimension;
-    attr[0].val.clusterDim.x = a.cluster;
-    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
-    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[1].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = a.pdl ? 2 : 1;
-}
-
-stark_b200_status opt_in(uint32_t value_blocks) {
-    static SmemOptIn once[kMaxBlocks], wide[kMaxBlocks];
-    Kernel kernel = kernel_of(value_blocks);
-    if (stark_b200_status st = ensure_dynamic_smem(kernel, (int)kSmemLimit, once[value_blocks - 1u])) return st;
-    int dev = 0;
-    SB_CUDA(cudaGetDevice(&dev));
-    const uint64_t bit = 1ull << (dev & 63);
-    if (wide[value_blocks - 1u].devices.load(std::memory_order_acquire) & bit) return STARK_B200_OK;
-    SB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
-    wide[value_blocks - 1u].devices.fetch_or(bit, std::memory_order_release);
-    return STARK_B200_OK;
-}
-
 }  // namespace
 
 bool grouped_attend_mma_supports(const GroupedShape &s) {
     return s.dim_p <= kMaxBlocks * 64u && s.vdim_p <= kMaxBlocks * 64u && layout_of(s).smem <= kSmemLimit && encode_tiled() != nullptr;
-}
-
-// 16 where the device can hold such a cluster of this kernel, else the portable 8.
-uint32_t grouped_attend_mma_max_cluster(const GroupedShape &s) {
-    if (opt_in(s.vdim_p / 64u) != STARK_B200_OK) return 8u;
-    GroupedArgs a{};
-    a.s = s;
-    a.splits = 1, a.cluster = kMaxCluster;
-    cudaLaunchConfig_t cfg{};
-    cudaLaunchAttribute attr[2];
-    launch_config(a, nullptr, cfg, attr);
-    int clusters = 0;
-    const cudaError_t e = cudaOccupancyMaxActiveClusters(&clusters, reinterpret_cast<const void *>(kernel_of(s.vdim_p / 64u)), &cfg);
-    if (e != cudaSuccess) cudaGetLastError();
-    return e == cudaSuccess && clusters > 0 ? kMaxCluster : 8u;
 }
 
 stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t stream) {
@@ -429,7 +427,9 @@ stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t s
         a.cluster > kMaxCluster || (a.cluster & (a.cluster - 1u)) || a.splits == 0 || a.splits > kMaxSplits ||
         (a.splits == 1u ? !a.out : !a.partials))
         return STARK_B200_INVALID_ARGUMENT;
-    if (stark_b200_status st = opt_in(s.vdim_p / 64u)) return st;
+    const Kernel kernel = kernel_of(s.vdim_p / 64u);
+    static SmemOptIn once[kMaxBlocks];
+    if (stark_b200_status st = ensure_dynamic_smem(kernel, (int)kSmemLimit, once[s.vdim_p / 64u - 1u])) return st;
     CUtensorMap k_map, v_map;
     auto make = [&](CUtensorMap *map, void *base, uint32_t columns) {
         const cuuint64_t dims[2] = {columns, (cuuint64_t)a.num_blocks * s.groups * kPageTokens}, strides[1] = {(cuuint64_t)columns * 2u};
@@ -441,9 +441,19 @@ stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t s
     if (!make(&k_map, a.keys, s.dim_p) || !make(&v_map, a.values, s.vdim_p)) return STARK_B200_DEVICE_FAILURE;
     const Layout l = layout_of(s);
     cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(a.splits * a.cluster, s.groups * ((s.per() + kHeads - 1u) / kHeads));
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = l.smem;
+    cfg.stream = stream;
     cudaLaunchAttribute attr[2];
-    launch_config(a, stream, cfg, attr);
-    SB_CUDA(cudaLaunchKernelEx(&cfg, kernel_of(s.vdim_p / 64u), k_map, v_map, a, l.slots, l.tile_bytes));
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = a.cluster;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = a.pdl ? 2 : 1;
+    SB_CUDA(cudaLaunchKernelEx(&cfg, kernel, k_map, v_map, a, l.slots, l.tile_bytes));
     return STARK_B200_OK;
 }
 

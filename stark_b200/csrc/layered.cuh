@@ -230,7 +230,7 @@ struct GroupedArgs {
     float *queries;            // grouped_rows: [m, heads, dim_p] scaled by scale * log2(e) ...
     uint16_t *queries_b16;     // ... or unscaled, rounded
     float *partials;           // grouped_attend_mma: [heads, splits, vdim_p + 4] where splits > 1
-    uint32_t splits, cluster;  // partials per head; spans of the cache merged into each (1, 2, 4, 8 or 16)
+    uint32_t splits, cluster;  // partials per head; spans of the cache merged into each (1, 2, 4 or 8)
     float *out;                // grouped_attend_mma: [heads * vdim_p] where splits == 1
     uint32_t *error_word;
     bool pdl;
@@ -240,7 +240,6 @@ bool grouped_shape_supported(const GroupedShape &s, uint32_t taps);
 stark_b200_status grouped_rows_launch(const GroupedArgs &a, cudaStream_t stream);
 // One token: the same and its attention in one launch, over a bf16 cache on the tensor cores.
 bool grouped_attend_mma_supports(const GroupedShape &s);
-uint32_t grouped_attend_mma_max_cluster(const GroupedShape &s);
 stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t stream);
 // The recent rows as they were before position `position` (a page's start), from the page tails.
 stark_b200_status short_conv_restore_launch(const GroupedArgs &a, uint32_t position, cudaStream_t stream);

@@ -86,7 +86,6 @@ struct LayeredState {
     // widest rows over the layers
     uint32_t max_in = 0, max_mixer = 0, max_attn = 0, max_ff = 0, max_joint = 0, max_expand = 0, max_q = 0, max_first = 0;
     size_t query_floats = 0, partial_floats = 0;
-    uint32_t max_cluster = 8;  // of the grouped decode attention
     // one token; attn: attention output with the gated activation behind it
     float *x[2] = {nullptr, nullptr}, *y = nullptr, *u = nullptr, *attn = nullptr;
     float *queries = nullptr, *partials = nullptr, *first_values = nullptr;
@@ -210,8 +209,7 @@ LatentArgs latent_args(Model *m, const Layer &layer) {
 // context is long.
 void divide_grouped(const Model *m, GroupedArgs &a) {
     const uint32_t tiles = a.s.groups * ((a.s.per() + 15u) / 16u), pages = m->num_blocks;
-    uint32_t most = m->layered->max_cluster;
-    if (tunables().grouped_cluster) most = std::min(most, tunables().grouped_cluster);
+    const uint32_t most = tunables().grouped_cluster ? tunables().grouped_cluster : 8u;
     a.cluster = 1;
     while (a.cluster * 2u <= most && a.cluster * 2u * tiles <= 148u && a.cluster < pages) a.cluster *= 2u;
     a.splits = std::max(1u, std::min({148u / (a.cluster * tiles), pages / (a.cluster * 16u), kMaxSplits}));
@@ -929,7 +927,6 @@ stark_b200_status build_grouped(Model *m, Layer &l) {
     for (uint32_t r = 1; r <= kAttendRows; ++r)
         L->partial_floats = std::max(L->partial_floats, span_partial_floats(s.heads, s.vdim_p, r, plain_splits(s, r)));
     L->partial_floats = std::max(L->partial_floats, span_partial_floats(s.heads, s.vdim_p, 1u, kMaxSplits));
-    if (!L->f32 && grouped_attend_mma_supports(s)) L->max_cluster = std::max(L->max_cluster, grouped_attend_mma_max_cluster(s));
     return STARK_B200_OK;
 }
 

@@ -35,7 +35,7 @@ const Entry kEntries[] = {
     {"gemm_half_tiles", "STARK_B200_GEMM_HALF_TILES", &Tunables::gemm_half_tiles, 1u, 0u, 2u},
     {"latent_spans", "STARK_B200_LATENT_SPANS", &Tunables::latent_spans, 0u, 0u, 64u},
     {"latent_cluster", "STARK_B200_LATENT_CLUSTER", &Tunables::latent_cluster, 4u, 1u, 8u},
-    {"grouped_cluster", "STARK_B200_GROUPED_CLUSTER", &Tunables::grouped_cluster, 0u, 0u, 16u},
+    {"grouped_cluster", "STARK_B200_GROUPED_CLUSTER", &Tunables::grouped_cluster, 0u, 0u, 8u},
     {"grouped_splits", "STARK_B200_GROUPED_SPLITS", &Tunables::grouped_splits, 0u, 0u, 64u},
     {"tp_rows_push", "STARK_B200_TP_ROWS_PUSH", &Tunables::tp_rows_push, 2u, 0u, 2u},
 };

@@ -29,7 +29,7 @@ struct Tunables {
     uint32_t rows_matvec;         // STARK_B200_ROWS_MATVEC      1: up to 8 rows go through the several-rows matvec, 0: through the tensor-core tile kernels
     uint32_t latent_spans;        // STARK_B200_LATENT_SPANS     spans of the latent cache a decode step attends to in parallel (0 = chosen from the head count, at most 64)
     uint32_t latent_cluster;      // STARK_B200_LATENT_CLUSTER   spans merged through distributed shared memory (1, 2, 4 or 8)
-    uint32_t grouped_cluster;     // STARK_B200_GROUPED_CLUSTER  spans of a key / value head merged through distributed shared memory in the grouped decode attention (0 = chosen from the head count; 1, 2, 4, 8 or 16)
+    uint32_t grouped_cluster;     // STARK_B200_GROUPED_CLUSTER  spans of a key / value head merged through distributed shared memory in the grouped decode attention (0 = chosen from the head count; 1, 2, 4 or 8)
     uint32_t grouped_splits;      // STARK_B200_GROUPED_SPLITS   clusters per key / value head there (0 = chosen; more than one costs a merging launch)
 };
 

@@ -195,7 +195,7 @@ def test_rewind_restores_the_convolutions(dtype):
 
 
 @pytest.mark.parametrize("settings", [dict(grouped_cluster=1), dict(grouped_cluster=2, grouped_splits=3), dict(grouped_cluster=8),
-                                      dict(grouped_cluster=16), dict(grouped_cluster=4, grouped_splits=9), dict(pdl=0)])
+                                      dict(grouped_cluster=4, grouped_splits=9), dict(pdl=0)])
 def test_spans_of_the_decode_attention(settings):
     """Recorded anew in the middle of a sequence with other divisions of the cache: more spans than pages, one span."""
     root = P.model([P.layer(P.mixer(heads=3, kv_heads=1, conv=5)), P.layer(P.mixer(heads=20, kv_heads=1, dim=64))])
