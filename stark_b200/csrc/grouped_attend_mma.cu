@@ -1,15 +1,17 @@
 // One token of grouped-query attention with short convolutions, in one launch over a bf16 cache: what a decode step runs.
 //
-// A CTA owns up to 16 query heads of one key / value head (the M side of mma.sync.m16n8k16) over one span of pages:
+// A CTA owns up to 8 query heads of one key / value head over one span of pages:
 //   pages       keys [64][dim_p] and values [64][vdim_p] by TMA, 128-byte swizzled boxes of 64 columns.  Every page was
 //               complete before this token began except for the token's own row, so all of them are fetched before the wait
-//               on the previous kernel
-//   own rows    after the wait every CTA forms its queries from the projected row and the recent ones (convolution, norm,
-//               temperature; bf16 hi + lo in shared memory).  The CTAs whose span ends with the token's own page also form
-//               its key and value, patch them into the fetched tile, and store them, the mixed-from values and the
-//               projected row for later positions
-//   attention   eight warps, each 16 keys of a page of its own pair (even and odd pages): f32 scores, running maximum and
-//               sum per head, weights as bf16 hi + lo straight from the score registers, weighted values in registers
+//               on the previous kernel, and the part of the convolutions that earlier tokens left is summed there too
+//   own rows    after the wait every CTA forms its queries from the projected row (convolution, norm, temperature; bf16
+//               hi + lo in shared memory).  The CTAs whose span ends with the token's own page also form its key and
+//               value, patch them into the fetched tile, and store them, the values to mix with and the projected row for
+//               later layers and positions
+//   attention   eight warps, each 32 keys of every fourth page.  Keys are the M side of mma.sync.m16n8k16, heads the N side:
+//               eight heads, or four whose hi and lo halves sit side by side (PACK), so that one product serves both.  f32
+//               scores, running maximum and sum per head; the weights, hi + lo likewise, go from the score registers into
+//               the second product (values transposed on the M side) through a register transpose
 //   merge       warps through shared memory, the spans of a cluster through distributed shared memory, each CTA taking a
 //               share of the columns; clusters beyond one leave partials for span_merge
 // so scores and weights keep f32 accuracy against the bf16 cache.  Every wait is bounded; a wait that runs out sets the
@@ -25,7 +27,8 @@ namespace sb {
 
 namespace {
 
-constexpr uint32_t kWarps = 8, kThreads = kWarps * 32u, kHeads = 16;
+constexpr uint32_t kWarps = 8, kThreads = kWarps * 32u, kHeads = kGroupedHeadTile;
+constexpr uint32_t kRound = 4;                 // pages read at a time, two warps each (two where tiles are so large)
 constexpr uint32_t kBox = kPageTokens * 128u;  // 64 keys x 64 columns bf16
 constexpr uint32_t kMaxBlocks = 4;             // heads up to 256 wide
 constexpr uint32_t kMaxCluster = 8;
@@ -52,17 +55,24 @@ __device__ inline float4 peer_load4(uint32_t addr) {
     return v;
 }
 
-__device__ inline float quad_max(float v) {
-    v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
-    return fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
+// Ends the kernel's use of distributed shared memory: only that everybody has come this far matters, not what was written.
+__device__ inline void cluster_leave() {
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;\n\tbarrier.cluster.wait.aligned;" ::: "memory");
 }
-__device__ inline float quad_sum(float v) {
-    v += __shfl_xor_sync(0xffffffffu, v, 1);
-    return v + __shfl_xor_sync(0xffffffffu, v, 2);
+// Over the lanes that hold the same columns of a product: lane / 4 varies.
+__device__ inline float rows_max(float v) {
+    v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 4));
+    v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 8));
+    return fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 16));
+}
+__device__ inline float rows_sum(float v) {
+    v += __shfl_xor_sync(0xffffffffu, v, 4);
+    v += __shfl_xor_sync(0xffffffffu, v, 8);
+    return v + __shfl_xor_sync(0xffffffffu, v, 16);
 }
 
-// blockIdx: (span, head tile of a key / value head); VB: value blocks of 64 columns
-template <uint32_t VB>
+// blockIdx: (span, head tile of a key / value head); VB: value blocks of 64 columns; PACK: at most four heads a tile
+template <uint32_t VB, bool PACK>
 __global__ void __launch_bounds__(kThreads, 1)
 grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const GroupedArgs a,
                           const uint32_t slots, const uint32_t tile_bytes) {
@@ -73,8 +83,9 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
     const GroupedShape &s = a.s;
     const uint32_t kb = s.dim_p / 64u, stage_bytes = (kb + VB) * kBox, q_pitch = s.dim_p + 8u;
     uint8_t *tile = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(grouped_smem) + 1023u) & ~(uintptr_t)1023u);
-    uint16_t *q_hi = reinterpret_cast<uint16_t *>(tile + tile_bytes), *q_lo = q_hi + kHeads * q_pitch;  // [head][q_pitch]
-    uint16_t *new_row = q_lo + kHeads * q_pitch;                                                       // key, then value
+    constexpr uint32_t kLow = PACK ? 4u : 8u;  // rows of the lo halves behind those of the hi halves
+    uint16_t *q_rows = reinterpret_cast<uint16_t *>(tile + tile_bytes);  // [2 * kLow][q_pitch]
+    uint16_t *new_row = q_rows + 2u * kLow * q_pitch;                    // key, then value
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
     const uint32_t head_tiles = (s.per() + kHeads - 1u) / kHeads;
     const uint32_t span_i = blockIdx.x, group = blockIdx.y / head_tiles, first_head = blockIdx.y % head_tiles * kHeads;
@@ -150,18 +161,14 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
         }
     };
     past(warp);  // nothing of this depends on the kernels before
+    const float q_factor = query_temperature(pos, a.temp_coef, a.temp_every) * (a.scale * kLog2e);
+    for (uint32_t i = heads * q_pitch + tid; i < kLow * q_pitch; i += kThreads) q_rows[i] = q_rows[kLow * q_pitch + i] = 0u;
     pdl_launch_dependents();
     pdl_wait();
-    for (uint32_t unit = warp; unit < kHeads + 2u; unit += kWarps) {
+    for (uint32_t unit = warp; unit < heads + 2u; unit += kWarps) {
         if (unit != warp) past(unit);
         const bool is_k = unit == 0u, is_v = unit == 1u, is_q = unit >= 2u;
         const uint32_t h = unit - 2u, blocks = unit_blocks(unit), col = unit_col(unit);
-        if (is_q && h >= heads) {
-            for (uint32_t c = lane * 2u; c < s.dim_p; c += 64u) {
-                *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + c) = 0u;
-                *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + c) = 0u;
-            }
-        }
         if (blocks == 0u) continue;
         const float *u = reinterpret_cast<const float *>(a.u) + col;
         float2 x[kMaxBlocks], mixed[kMaxBlocks];
@@ -180,7 +187,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
         }
         float factor = 1.0f;
         if (!is_v) factor = inverse_rms(warp_sum(sum), s.dim, a.eps);
-        if (is_q) factor *= query_temperature(pos, a.temp_coef, a.temp_every) * (a.scale * kLog2e);
+        if (is_q) factor *= q_factor;
         const bool stores = owner && (is_q || first_head == 0u);  // one CTA per stored value
         uint16_t *dst = reinterpret_cast<uint16_t *>(is_k ? a.keys : a.values) +
                         (((size_t)last_page * s.groups + group) * kPageTokens + in_page) * (is_v ? s.vdim_p : s.dim_p) + lane * 2u;
@@ -192,8 +199,8 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
             if (is_q) {
                 uint32_t hi, lo2;
                 split_bf16x2(o.x, o.y, hi, lo2);
-                *reinterpret_cast<uint32_t *>(q_hi + h * q_pitch + lane * 2u + b * 64u) = hi;
-                *reinterpret_cast<uint32_t *>(q_lo + h * q_pitch + lane * 2u + b * 64u) = lo2;
+                *reinterpret_cast<uint32_t *>(q_rows + h * q_pitch + lane * 2u + b * 64u) = hi;
+                *reinterpret_cast<uint32_t *>(q_rows + (kLow + h) * q_pitch + lane * 2u + b * 64u) = lo2;
             } else {
                 if (is_v && a.mix == kMixFirst && stores) keep_first_values(first, lane * 2u + b * 64u, s.vdim, o);
                 if (is_v && a.mix == kMixShare) o = mix_values(first, lane * 2u + b * 64u, s.vdim, o, a.share);
@@ -215,14 +222,24 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
     }
     __syncthreads();
 
-    // ---- attention: warps 0-3 take the span's even pages, 4-7 the odd ones, 16 keys each
-    const uint32_t half = warp >> 2, key0 = (warp & 3u) * 16u;
+    // ---- attention: warps 2j and 2j + 1 take pages j, j + 4, ... of the span, half the keys each
+    const uint32_t key0 = (warp & 1u) * 32u;
     const uint32_t mi = lane >> 3, mr = lane & 7u;  // ldmatrix: which 8 x 8 matrix this lane addresses, which row of it
-    const uint32_t q_at = smem_u32(q_hi) + (((lane & 7u) + ((lane >> 3) & 1u) * 8u) * q_pitch + (lane >> 4) * 8u) * 2u;
-    const uint32_t q_lo_at = q_at + kHeads * q_pitch * 2u;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f}, out[VB * 8u][4];
+    const uint32_t col = (lane & 3u) * 2u;          // this lane's columns of a product: two heads (PACK: modulo 4)
+    uint32_t qf[kMaxBlocks * 4u][2], ql[PACK ? 1u : kMaxBlocks * 4u][2];
 #pragma unroll
-    for (uint32_t i = 0; i < VB * 8u; ++i)
+    for (uint32_t i = 0; i < kMaxBlocks * 4u; ++i) {
+        if (i >= kb * 4u) break;
+        const uint16_t *src = q_rows + (lane >> 2) * q_pitch + i * 16u + col;
+        qf[i][0] = *reinterpret_cast<const uint32_t *>(src), qf[i][1] = *reinterpret_cast<const uint32_t *>(src + 8u);
+        if constexpr (!PACK) {
+            ql[i][0] = *reinterpret_cast<const uint32_t *>(src + kLow * q_pitch);
+            ql[i][1] = *reinterpret_cast<const uint32_t *>(src + kLow * q_pitch + 8u);
+        }
+    }
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f}, out[VB * 4u][4];  // l: this lane's keys only
+#pragma unroll
+    for (uint32_t i = 0; i < VB * 4u; ++i)
 #pragma unroll
         for (uint32_t e = 0; e < 4u; ++e) out[i][e] = 0.0f;
     auto ldm = [](uint32_t (&r)[4], uint32_t addr) {
@@ -237,9 +254,10 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                      : "r"(addr)
                      : "memory");
     };
-    for (uint32_t i0 = 0; i0 < n; i0 += 2u) {
-        const uint32_t i = i0 + half;
-        bool ok = i < n;
+    const uint32_t round = min(kRound, slots);
+    for (uint32_t i0 = 0; i0 < n; i0 += round) {
+        const uint32_t i = i0 + (warp >> 1);
+        bool ok = i < n && (warp >> 1) < round && (lo + i) * kPageTokens + key0 <= pos;  // something to see; the same for the whole warp
         if (ok && !(ok = mbar_wait_bounded(&full[i % slots], (i / slots) & 1u, &abort_flag))) {
             abort_flag = 1;
             if (lane == 0) atomicOr(a.error_word, kErrMbarTimeout);
@@ -248,104 +266,123 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
         if (ok) {
             uint8_t *stage = tile + (i % slots) * stage_bytes;
             const uint32_t row = pos % kPageTokens;
-            if (lo + i + 1u == pages && (row & ~15u) == key0) {  // this warp's keys include the token's own
+            if (lo + i + 1u == pages && (row & ~31u) == key0) {  // this warp's keys include the token's own
                 const uint4 *src = reinterpret_cast<const uint4 *>(new_row);
                 for (uint32_t c = lane; c < (kb + VB) * 8u; c += 32u)
                     *reinterpret_cast<uint4 *>(stage + (c >> 3) * kBox + row * 128u + (((c & 7u) ^ (row & 7u)) << 4)) = src[c];
                 __syncwarp();
             }
             const uint32_t base = smem_u32(stage);
-            float sc[2][4] = {}, low[2][4] = {};  // products with the queries' leading and trailing halves
-            const uint32_t key = key0 + (mi >> 1) * 8u + mr, key_line = base + key * 128u;
-            for (uint32_t b = 0; b < kb; ++b) {
+            float sc[2][4] = {}, low[2][4] = {};  // [16 keys][keys lane / 4 and + 8, two heads each]
+            const uint32_t key = key0 + (mi & 1u) * 8u + mr, key_line = base + key * 128u;
+#pragma unroll
+            for (uint32_t b = 0; b < kMaxBlocks; ++b) {
+                if (b >= kb) break;
 #pragma unroll
                 for (uint32_t k16 = 0; k16 < 4u; ++k16) {  // 16 columns
-                    uint32_t qh[4], ql[4], kf[4];
-                    ldm(qh, q_at + (b * 64u + k16 * 16u) * 2u);
-                    ldm(ql, q_lo_at + (b * 64u + k16 * 16u) * 2u);
-                    ldm(kf, key_line + b * kBox + (((k16 * 2u + (mi & 1u)) ^ (key & 7u)) << 4));
-                    mma_m16n8k16_bf16(sc[0], qh[0], qh[1], qh[2], qh[3], kf[0], kf[1]);
-                    mma_m16n8k16_bf16(sc[1], qh[0], qh[1], qh[2], qh[3], kf[2], kf[3]);
-                    mma_m16n8k16_bf16(low[0], ql[0], ql[1], ql[2], ql[3], kf[0], kf[1]);
-                    mma_m16n8k16_bf16(low[1], ql[0], ql[1], ql[2], ql[3], kf[2], kf[3]);
+#pragma unroll
+                    for (uint32_t g = 0; g < 2u; ++g) {    // 16 keys
+                        uint32_t kf[4];
+                        ldm(kf, key_line + g * 2048u + b * kBox + (((k16 * 2u + (mi >> 1)) ^ (key & 7u)) << 4));
+                        mma_m16n8k16_bf16(sc[g], kf[0], kf[1], kf[2], kf[3], qf[b * 4u + k16][0], qf[b * 4u + k16][1]);
+                        if constexpr (!PACK)
+                            mma_m16n8k16_bf16(low[g], kf[0], kf[1], kf[2], kf[3], ql[b * 4u + k16][0], ql[b * 4u + k16][1]);
+                    }
                 }
             }
-            const uint32_t first_key = (lo + i) * kPageTokens + key0 + (lane & 3u) * 2u;
-            if (first_key - (lane & 3u) * 2u <= pos) {  // the same for the whole warp
-                float keep[2];
-                uint32_t ph[4], pl[4];
+            const uint32_t first_key = (lo + i) * kPageTokens + key0 + (lane >> 2);
+            float keep[2];
+            uint32_t pf[2][2], pl[2][2];  // weights as the second product wants them: [16 keys][8 of them]
+            {
+                float w[2][4], top[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-                for (uint32_t r = 0; r < 2u; ++r) {  // rows lane / 4 and lane / 4 + 8
-                    float v[4] = {sc[0][2u * r] + low[0][2u * r], sc[0][2u * r + 1u] + low[0][2u * r + 1u],
-                                  sc[1][2u * r] + low[1][2u * r], sc[1][2u * r + 1u] + low[1][2u * r + 1u]};
-                    float top = -INFINITY;
+                for (uint32_t g = 0; g < 2u; ++g)
 #pragma unroll
                     for (uint32_t e = 0; e < 4u; ++e) {
-                        if (first_key + (e & 1u) + (e >> 1) * 8u > pos) v[e] = -INFINITY;
-                        top = fmaxf(top, v[e]);
+                        w[g][e] = sc[g][e] + (PACK ? __shfl_xor_sync(0xffffffffu, sc[g][e], 2) : low[g][e]);
+                        if (first_key + g * 16u + (e >> 1) * 8u > pos) w[g][e] = -INFINITY;
+                        top[e & 1u] = fmaxf(top[e & 1u], w[g][e]);
                     }
-                    top = fmaxf(m[r], quad_max(top));
-                    keep[r] = exp2f(m[r] - top);  // 0 at first
-                    m[r] = top;
-                    float sum = 0.0f;
 #pragma unroll
-                    for (uint32_t e = 0; e < 4u; ++e) {
-                        v[e] = exp2f(v[e] - top);
-                        sum += v[e];
-                    }
-                    l[r] = l[r] * keep[r] + quad_sum(sum);
-                    split_bf16x2(v[0], v[1], ph[r], pl[r]);
-                    split_bf16x2(v[2], v[3], ph[2u + r], pl[2u + r]);
+                for (uint32_t e = 0; e < 2u; ++e) {
+                    top[e] = fmaxf(m[e], rows_max(top[e]));
+                    keep[e] = exp2f(m[e] - top[e]);  // 0 at first
+                    m[e] = top[e];
+                    l[e] *= keep[e];
                 }
-                const uint32_t vkey = key0 + (mi & 1u) * 8u + mr, value_line = base + kb * kBox + vkey * 128u;
 #pragma unroll
-                for (uint32_t b = 0; b < VB; ++b)
+                for (uint32_t g = 0; g < 2u; ++g)
 #pragma unroll
-                    for (uint32_t n2 = 0; n2 < 4u; ++n2) {  // 16 columns
-                        uint32_t vf[4];
-                        ldm_trans(vf, value_line + b * kBox + (((n2 * 2u + (mi >> 1)) ^ (vkey & 7u)) << 4));
-#pragma unroll
-                        for (uint32_t t = 0; t < 2u; ++t) {
-                            float(&o)[4] = out[b * 8u + n2 * 2u + t];
-                            o[0] *= keep[0], o[1] *= keep[0], o[2] *= keep[1], o[3] *= keep[1];
-                            mma_m16n8k16_bf16(o, ph[0], ph[1], ph[2], ph[3], vf[2u * t], vf[2u * t + 1u]);
-                            mma_m16n8k16_bf16(o, pl[0], pl[1], pl[2], pl[3], vf[2u * t], vf[2u * t + 1u]);
+                    for (uint32_t e = 0; e < 4u; e += 2u) {
+                        const float w0 = exp2f(w[g][e] - top[0]), w1 = exp2f(w[g][e + 1u] - top[1]);
+                        l[0] += w0, l[1] += w1;
+                        uint32_t hi, lo2;
+                        split_bf16x2(w0, w1, hi, lo2);
+                        if constexpr (PACK) {
+                            pf[g][e >> 1] = movmatrix_trans(col < 4u ? hi : lo2);
+                        } else {
+                            pf[g][e >> 1] = movmatrix_trans(hi);
+                            pl[g][e >> 1] = movmatrix_trans(lo2);
                         }
                     }
             }
+            const uint32_t vkey = key0 + (mi >> 1) * 8u + mr, value_line = base + kb * kBox + vkey * 128u;
+#pragma unroll
+            for (uint32_t v16 = 0; v16 < VB * 4u; ++v16) {  // 16 columns
+                float(&o)[4] = out[v16];
+                o[0] *= keep[0], o[1] *= keep[1], o[2] *= keep[0], o[3] *= keep[1];
+#pragma unroll
+                for (uint32_t g = 0; g < 2u; ++g) {
+                    uint32_t vf[4];
+                    ldm_trans(vf, value_line + g * 2048u + (v16 >> 2) * kBox + ((((v16 & 3u) * 2u + (mi & 1u)) ^ (vkey & 7u)) << 4));
+                    mma_m16n8k16_bf16(o, vf[0], vf[1], vf[2], vf[3], pf[g][0], pf[g][1]);
+                    if constexpr (!PACK) mma_m16n8k16_bf16(o, vf[0], vf[1], vf[2], vf[3], pl[g][0], pl[g][1]);
+                }
+            }
         }
-        if (i0 + slots < n) {  // the two pages just read make room for two more
+        if (i0 + slots < n) {  // the pages just read make room for more
             __syncthreads();
             if (tid == 0)
-                for (uint32_t j = i0 + slots; j < min(n, i0 + slots + 2u); ++j) fetch(j);
+                for (uint32_t j = i0 + slots; j < min(n, i0 + slots + round); ++j) fetch(j);
         }
     }
 
     // ---- merge of the warps: statistics, then weighted values, rows pitch apart
     const uint32_t pitch = s.vdim_p + 8u;
     float *state = reinterpret_cast<float *>(tile);  // [warp][head][pitch]; the sum ends up in warp 0's part
-    if ((lane & 3u) == 0u) {
 #pragma unroll
-        for (uint32_t r = 0; r < 2u; ++r) warp_m[warp][(lane >> 2) + 8u * r] = m[r], warp_l[warp][(lane >> 2) + 8u * r] = l[r];
+    for (uint32_t e = 0; e < 2u; ++e) {
+        l[e] = rows_sum(l[e]);
+        if (lane < (PACK ? 2u : 4u)) warp_m[warp][col + e] = m[e], warp_l[warp][col + e] = l[e];
     }
     __syncthreads();  // everybody is through with the tiles as well
+    {
+        float mine[2];
 #pragma unroll
-    for (uint32_t r = 0; r < 2u; ++r) {
-        const uint32_t h = (lane >> 2) + 8u * r;
-        if (h >= heads) continue;
-        float top = -INFINITY, sum = 0.0f;
+        for (uint32_t e = 0; e < 2u; ++e) {
+            const uint32_t h = (PACK ? col & 2u : col) + e;
+            float top = -INFINITY;
 #pragma unroll
-        for (uint32_t w = 0; w < kWarps; ++w) top = fmaxf(top, warp_m[w][h]);
-        const float mine = m[r] == -INFINITY ? 0.0f : exp2f(m[r] - top);
-        float *dst = state + ((size_t)warp * heads + h) * pitch + (lane & 3u) * 2u;
+            for (uint32_t w = 0; w < kWarps; ++w) top = fmaxf(top, warp_m[w][h]);
+            mine[e] = m[e] == -INFINITY ? 0.0f : exp2f(m[e] - top);
+        }
 #pragma unroll
-        for (uint32_t i = 0; i < VB * 8u; ++i)
-            *reinterpret_cast<float2 *>(dst + i * 8u) = make_float2(out[i][2u * r] * mine, out[i][2u * r + 1u] * mine);
-        if (warp == 0u && (lane & 3u) == 0u) {
+        for (uint32_t v16 = 0; v16 < VB * 4u; ++v16)
+#pragma unroll
+            for (uint32_t e = 0; e < 4u; ++e) {  // columns lane / 4 and + 8 of 16, two heads each
+                float o = out[v16][e] * mine[e & 1u];
+                if constexpr (PACK) o += __shfl_xor_sync(0xffffffffu, o, 2);
+                const uint32_t h = col + (e & 1u);
+                if (h < heads) state[((size_t)warp * heads + h) * pitch + v16 * 16u + (e >> 1) * 8u + (lane >> 2)] = o;
+            }
+        if (tid < heads) {
+            float top = -INFINITY, sum = 0.0f;
+#pragma unroll
+            for (uint32_t w = 0; w < kWarps; ++w) top = fmaxf(top, warp_m[w][tid]);
 #pragma unroll
             for (uint32_t w = 0; w < kWarps; ++w)
-                if (warp_m[w][h] != -INFINITY) sum = fmaf(exp2f(warp_m[w][h] - top), warp_l[w][h], sum);
-            run_m[h] = top, run_l[h] = sum;
+                if (warp_m[w][tid] != -INFINITY) sum = fmaf(exp2f(warp_m[w][tid] - top), warp_l[w][tid], sum);
+            run_m[tid] = top, run_l[tid] = sum;
         }
     }
     __syncthreads();
@@ -390,7 +427,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
             *reinterpret_cast<float4 *>(dst + 4u + q * 4u) = v;
         }
     }
-    if (a.cluster > 1u) cluster_sync();  // nobody leaves while another CTA may read its shared memory
+    if (a.cluster > 1u) cluster_leave();  // nobody leaves while another CTA may read its shared memory
 }
 
 struct Layout {
@@ -400,17 +437,19 @@ Layout layout_of(const GroupedShape &s) {
     const uint32_t stage = (s.dim_p + s.vdim_p) / 64u * kBox, heads = std::min(kHeads, s.per());
     Layout l{};
     l.slots = std::min(kMaxSlots, std::max(2u, kTileBudget / stage));
+    if (l.slots < kRound) l.slots = 2u;
     l.tile_bytes = std::max(l.slots * stage, kWarps * heads * (s.vdim_p + 8u) * 4u);
     l.tile_bytes = (l.tile_bytes + 127u) & ~127u;
-    l.smem = l.tile_bytes + 2u * kHeads * (s.dim_p + 8u) * 2u + (s.dim_p + s.vdim_p) * 2u + 1024u;
+    l.smem = l.tile_bytes + 2u * (heads <= 4u ? 4u : 8u) * (s.dim_p + 8u) * 2u + (s.dim_p + s.vdim_p) * 2u + 1024u;
     return l;
 }
 
 using Kernel = void (*)(const CUtensorMap, const CUtensorMap, const GroupedArgs, uint32_t, uint32_t);
+template <bool PACK>
 Kernel kernel_of(uint32_t value_blocks) {
-    return value_blocks == 1u ? grouped_attend_mma_kernel<1>
-                              : (value_blocks == 2u ? grouped_attend_mma_kernel<2>
-                                                    : (value_blocks == 3u ? grouped_attend_mma_kernel<3> : grouped_attend_mma_kernel<4>));
+    return value_blocks == 1u ? grouped_attend_mma_kernel<1, PACK>
+                              : (value_blocks == 2u ? grouped_attend_mma_kernel<2, PACK>
+                                                    : (value_blocks == 3u ? grouped_attend_mma_kernel<3, PACK> : grouped_attend_mma_kernel<4, PACK>));
 }
 
 }  // namespace
@@ -427,9 +466,10 @@ stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t s
         a.cluster > kMaxCluster || (a.cluster & (a.cluster - 1u)) || a.splits == 0 || a.splits > kMaxSplits ||
         (a.splits == 1u ? !a.out : !a.partials))
         return STARK_B200_INVALID_ARGUMENT;
-    const Kernel kernel = kernel_of(s.vdim_p / 64u);
-    static SmemOptIn once[kMaxBlocks];
-    if (stark_b200_status st = ensure_dynamic_smem(kernel, (int)kSmemLimit, once[s.vdim_p / 64u - 1u])) return st;
+    const bool pack = s.per() <= 4u;
+    const Kernel kernel = pack ? kernel_of<true>(s.vdim_p / 64u) : kernel_of<false>(s.vdim_p / 64u);
+    static SmemOptIn once[2][kMaxBlocks];
+    if (stark_b200_status st = ensure_dynamic_smem(kernel, (int)kSmemLimit, once[pack][s.vdim_p / 64u - 1u])) return st;
     CUtensorMap k_map, v_map;
     auto make = [&](CUtensorMap *map, void *base, uint32_t columns) {
         const cuuint64_t dims[2] = {columns, (cuuint64_t)a.num_blocks * s.groups * kPageTokens}, strides[1] = {(cuuint64_t)columns * 2u};

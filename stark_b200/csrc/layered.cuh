@@ -239,6 +239,7 @@ bool grouped_shape_supported(const GroupedShape &s, uint32_t taps);
 // Convolutions, norms, temperature and mixing of m rows; keys and values into the cache, the convolutions' state kept.
 stark_b200_status grouped_rows_launch(const GroupedArgs &a, cudaStream_t stream);
 // One token: the same and its attention in one launch, over a bf16 cache on the tensor cores.
+constexpr uint32_t kGroupedHeadTile = 8;  // query heads of a key / value head a CTA takes there
 bool grouped_attend_mma_supports(const GroupedShape &s);
 stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t stream);
 // The recent rows as they were before position `position` (a page's start), from the page tails.

@@ -204,11 +204,11 @@ LatentArgs latent_args(Model *m, const Layer &layer) {
     return a;
 }
 
-// Spans of the grouped decode attention: a cluster of CTAs per key / value head (and 16 of its query heads), as large as
+// Spans of the grouped decode attention: a cluster of CTAs per key / value head (and 8 of its query heads), as large as
 // the SMs allow and the context has pages; more clusters, merged by a launch of their own, where heads are few and the
 // context is long.
 void divide_grouped(const Model *m, GroupedArgs &a) {
-    const uint32_t tiles = a.s.groups * ((a.s.per() + 15u) / 16u), pages = m->num_blocks;
+    const uint32_t tiles = a.s.groups * ((a.s.per() + kGroupedHeadTile - 1u) / kGroupedHeadTile), pages = m->num_blocks;
     const uint32_t most = tunables().grouped_cluster ? tunables().grouped_cluster : 8u;
     a.cluster = 1;
     while (a.cluster * 2u <= most && a.cluster * 2u * tiles <= 148u && a.cluster < pages) a.cluster *= 2u;
