@@ -3,6 +3,7 @@
 // y = W x is bound by the bytes of W.  A CTA's warps each take pairs of rows (the gate and the up row of one unit, or
 // two neighbours) and stream them with eight 16-byte loads in flight per lane; two 256-thread CTAs per SM keep 64 KB
 // in flight.  The first batch of loads is issued before the wait on the previous kernel: weights depend on nothing.
+// Where there are too few pairs for the SMs' warps, several warps of a CTA share a pair, each taking its batches of columns.
 // The input row stays f32 throughout (a bf16 weight times an f32 activation, f32 accumulation), so the one-row path has
 // no rounding of activations at all and serves the 32-bit mode unchanged.
 // The input row is formed by every CTA in its prologue: plain, its norm, or the residual add of a normed sublayer output,
@@ -56,6 +57,7 @@ struct MatvecParams {
     float *stored_out;
     const float *residual, *scale_a, *scale_b;
     uint32_t split_col;
+    uint32_t share;         // warps of a CTA that share a pair: 1, 2, 4 or 8
 };
 
 template <uint32_t PRO, uint32_t EPI>
@@ -66,8 +68,10 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
     __shared__ uint32_t best_i[kWarps];
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
     const uint32_t chunks = (p.cols + kChunk - 1u) / kChunk;
-    const uint32_t stride = gridDim.x * kWarps;
-    uint32_t pair = blockIdx.x * kWarps + warp;
+    __shared__ float parts[2][kWarps][4];  // of a shared pair's sums
+    const uint32_t share = EPI == kRowLogits ? 1u : p.share, slot = warp / share, sub = warp % share, per_cta = kWarps / share;
+    const uint32_t stride = gridDim.x * per_cta, first_chunk = sub * kUnroll;
+    uint32_t pair = blockIdx.x * per_cta + slot;
 
     // rows of a pair: gate and up 16 apart, or neighbours
     auto is_gate = [&](uint32_t pr) { return EPI == kRowGate && pr >= p.stored_pairs; };
@@ -91,7 +95,7 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
             }
         }
     };
-    fetch(buf[0], pair, 0u);
+    fetch(buf[0], pair, first_chunk);
 
     pdl_launch_dependents();
     pdl_wait();
@@ -151,7 +155,8 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
     float top = -INFINITY;
     uint32_t top_i = 0xffffffffu;
     bool bad = false;
-    uint32_t chunk = 0, cur = 0;
+    uint32_t chunk = first_chunk, cur = 0, turn = 0;
+    const uint32_t lead = share > 1u ? slot : 0u;  // warps that share pairs go on until the CTA's first one has none
     float acc[2] = {0.0f, 0.0f}, behind[2] = {0.0f, 0.0f};  // behind: columns from split_col on
     float res[2], sa[2], sb[2];
     auto fetch_residual = [&](uint32_t pr) {  // asked for when a pair begins, used when it ends
@@ -167,9 +172,9 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
         }
     };
     fetch_residual(pair);
-    while (pair < p.pairs) {
-        uint32_t next_pair = pair, next_chunk = chunk + kUnroll;
-        if (next_chunk >= chunks) next_chunk = 0, next_pair = pair + stride;
+    while (pair - lead < p.pairs) {
+        uint32_t next_pair = pair, next_chunk = chunk + kUnroll * share;
+        if (next_chunk >= chunks) next_chunk = first_chunk, next_pair = pair + stride;
         auto consume = [&](uint4 (&now)[kUnroll][2], uint4 (&then)[kUnroll][2]) {
             fetch(then, next_pair, next_chunk);
 #pragma unroll
@@ -198,14 +203,27 @@ __global__ void __launch_bounds__(kThreads, 2) matvec_b16_kernel(const MatvecPar
         if (next_pair != pair) {
             float v0 = warp_sum(acc[0]), v1 = warp_sum(acc[1]);
             acc[0] = acc[1] = 0.0f;
+            float w0 = 0.0f, w1 = 0.0f;
             if constexpr (EPI == kRowResidual) {
-                const float w0 = warp_sum(behind[0]), w1 = warp_sum(behind[1]);
+                w0 = warp_sum(behind[0]), w1 = warp_sum(behind[1]);
                 behind[0] = behind[1] = 0.0f;
+            }
+            if (EPI != kRowLogits && share > 1u) {  // the same number of times in every warp
+                float *mine = parts[turn][warp];
+                if (lane == 0) mine[0] = v0, mine[1] = v1, mine[2] = w0, mine[3] = w1;
+                __syncthreads();
+                for (uint32_t i = 1; i < share; ++i) {  // the first of the sharing warps has the sum
+                    const float *other = parts[turn][slot * share + i];
+                    v0 += other[0], v1 += other[1], w0 += other[2], w1 += other[3];
+                }
+                turn ^= 1u;
+            }
+            if constexpr (EPI == kRowResidual) {
                 v0 = fmaf(sb[0], w0, fmaf(sa[0], v0, res[0]));
                 v1 = fmaf(sb[1], w1, fmaf(sa[1], v1, res[1]));
                 fetch_residual(next_pair);
             }
-            if (lane == 0) {
+            if (lane == 0 && sub == 0u && pair < p.pairs) {
                 const uint32_t r = row0(pair), step = apart(pair);
                 if (p.bias) v0 += p.bias[r], v1 += r + step < p.rows ? p.bias[r + step] : 0.0f;
                 if (is_gate(pair)) {
@@ -318,7 +336,11 @@ stark_b200_status matvec_b16_launch(const MatvecArgs &a, cudaStream_t stream) {
     p.stored_pairs = a.epilogue == kRowGate ? a.stored_rows / 2u : 0u, p.stored_out = a.stored_out;
     p.residual = a.residual, p.scale_a = a.scale_a, p.scale_b = a.scale_b, p.split_col = a.split_col;
     const uint32_t smem = matvec_smem(a.w);
-    const uint32_t grid = std::min<uint32_t>((p.pairs + kWarps - 1u) / kWarps, 148u * (smem <= 100u * 1024u ? 2u : 1u));
+    const uint32_t most = 148u * (smem <= 100u * 1024u ? 2u : 1u), batches = (a.w.cols + kChunk * kUnroll - 1u) / (kChunk * kUnroll);
+    p.share = 1;
+    while (a.epilogue != kRowLogits && p.share < kWarps && p.share * 2u <= batches && (p.pairs * p.share * 2u + kWarps - 1u) / kWarps <= most)
+        p.share *= 2u;
+    const uint32_t grid = std::min<uint32_t>((p.pairs * p.share + kWarps - 1u) / kWarps, most);
     MatvecKernel kernel = a.prologue == kRowPlain
                               ? pick<kRowPlain>(a.epilogue)
                               : (a.prologue == kRowAddNorm

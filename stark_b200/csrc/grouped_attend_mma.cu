@@ -33,7 +33,7 @@ constexpr uint32_t kBox = kPageTokens * 128u;  // 64 keys x 64 columns bf16
 constexpr uint32_t kMaxBlocks = 4;             // heads up to 256 wide
 constexpr uint32_t kMaxCluster = 8;
 constexpr uint32_t kMaxSlots = 8;
-constexpr uint32_t kTileBudget = 128u * 1024u, kSmemLimit = 220u * 1024u;
+constexpr uint32_t kSmemLimit = 220u * 1024u;  // dynamic; of 227 KB an SM has for its CTAs
 
 __device__ inline void cluster_sync() {
     asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -102,16 +102,15 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
         mbar_fence_init();
     }
     __syncthreads();
-    auto fetch = [&](uint32_t i) {  // one thread
-        const uint32_t slot = i % slots;
+    auto fetch = [&](uint32_t slot, uint32_t page) {  // one thread
         mbar_arrive_expect_tx(&full[slot], stage_bytes);
-        const uint32_t y = ((uint32_t)a.block_table[lo + i] * s.groups + group) * kPageTokens;
+        const uint32_t y = (page * s.groups + group) * kPageTokens;
         uint8_t *dst = tile + slot * stage_bytes;
         for (uint32_t b = 0; b < kb; ++b) tma_load_2d(dst + b * kBox, &k_map, b * 64u, y, &full[slot]);
         for (uint32_t b = 0; b < VB; ++b) tma_load_2d(dst + (kb + b) * kBox, &v_map, b * 64u, y, &full[slot]);
     };
     if (tid == 0)
-        for (uint32_t i = 0; i < min(n, slots); ++i) fetch(i);
+        for (uint32_t i = 0; i < min(n, slots); ++i) fetch(i, (uint32_t)a.block_table[lo + i]);
 
     // ---- queries of this CTA's heads, and the token's own key and value where they are needed.  A unit is one head of the
     // three, a warp's; units 0 and 1 are the key and the value, which take the longest way.
@@ -255,16 +254,24 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                      : "memory");
     };
     const uint32_t round = min(kRound, slots);
+    uint32_t slot0 = 0, phase0 = 0;  // of page i0
     for (uint32_t i0 = 0; i0 < n; i0 += round) {
         const uint32_t i = i0 + (warp >> 1);
+        const bool wraps = slot0 + (warp >> 1) >= slots;
+        const uint32_t slot = slot0 + (warp >> 1) - (wraps ? slots : 0u), phase = phase0 ^ (wraps ? 1u : 0u);
+        uint32_t coming[kRound];  // pages that take the places of those read now
+        if (tid == 0)
+#pragma unroll
+            for (uint32_t j = 0; j < kRound; ++j)
+                coming[j] = j < round && i0 + slots + j < n ? (uint32_t)a.block_table[lo + i0 + slots + j] : UINT32_MAX;
         bool ok = i < n && (warp >> 1) < round && (lo + i) * kPageTokens + key0 <= pos;  // something to see; the same for the whole warp
-        if (ok && !(ok = mbar_wait_bounded(&full[i % slots], (i / slots) & 1u, &abort_flag))) {
+        if (ok && !(ok = mbar_wait_bounded(&full[slot], phase, &abort_flag))) {
             abort_flag = 1;
             if (lane == 0) atomicOr(a.error_word, kErrMbarTimeout);
         }
         ok = __all_sync(0xffffffffu, ok);
         if (ok) {
-            uint8_t *stage = tile + (i % slots) * stage_bytes;
+            uint8_t *stage = tile + slot * stage_bytes;
             const uint32_t row = pos % kPageTokens;
             if (lo + i + 1u == pages && (row & ~31u) == key0) {  // this warp's keys include the token's own
                 const uint4 *src = reinterpret_cast<const uint4 *>(new_row);
@@ -340,11 +347,18 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                 }
             }
         }
-        if (i0 + slots < n) {  // the pages just read make room for more
+        if (i0 + slots < n) {
             __syncthreads();
-            if (tid == 0)
-                for (uint32_t j = i0 + slots; j < min(n, i0 + slots + round); ++j) fetch(j);
+            if (tid == 0) {
+                uint32_t into = slot0;
+#pragma unroll
+                for (uint32_t j = 0; j < kRound; ++j) {
+                    if (coming[j] != UINT32_MAX) fetch(into, coming[j]);
+                    if (++into == slots) into = 0u;
+                }
+            }
         }
+        if ((slot0 += round) >= slots) slot0 -= slots, phase0 ^= 1u;
     }
 
     // ---- merge of the warps: statistics, then weighted values, rows pitch apart
@@ -403,20 +417,25 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
     const uint32_t me = span_i % a.cluster, split_i = span_i / a.cluster;
     for (uint32_t t = me + a.cluster * tid; t < heads * quads; t += a.cluster * kThreads) {
         const uint32_t h = t / quads, q = t % quads;
-        float weight[kMaxCluster], top = -INFINITY, sum = 0.0f;
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        float weight[kMaxCluster], sums[kMaxCluster], top = -INFINITY, sum = 0.0f;
+        float4 x[kMaxCluster], v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+        for (uint32_t c = 0; c < kMaxCluster; ++c) {  // all on their way before the first is used
+            const uint32_t from = c < a.cluster ? c : 0u;
+            weight[c] = peer_load(peer_smem(&run_m[h], from));
+            sums[c] = peer_load(peer_smem(&run_l[h], from));
+            x[c] = peer_load4(peer_smem(state + h * pitch + q * 4u, from));
+        }
 #pragma unroll
         for (uint32_t c = 0; c < kMaxCluster; ++c) {
-            weight[c] = c < a.cluster ? peer_load(peer_smem(&run_m[h], c)) : -INFINITY;
+            if (c >= a.cluster) weight[c] = -INFINITY;
             top = fmaxf(top, weight[c]);
         }
 #pragma unroll
         for (uint32_t c = 0; c < kMaxCluster; ++c) {
-            if (c >= a.cluster) break;
             const float k = weight[c] == -INFINITY ? 0.0f : exp2f(weight[c] - top);
-            sum = fmaf(k, peer_load(peer_smem(&run_l[h], c)), sum);
-            const float4 x = peer_load4(peer_smem(state + h * pitch + q * 4u, c));
-            v.x = fmaf(k, x.x, v.x), v.y = fmaf(k, x.y, v.y), v.z = fmaf(k, x.z, v.z), v.w = fmaf(k, x.w, v.w);
+            sum = fmaf(k, sums[c], sum);
+            v.x = fmaf(k, x[c].x, v.x), v.y = fmaf(k, x[c].y, v.y), v.z = fmaf(k, x[c].z, v.z), v.w = fmaf(k, x[c].w, v.w);
         }
         if (a.splits == 1u) {
             const float inv = 1.0f / sum;
@@ -433,14 +452,17 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
 struct Layout {
     uint32_t slots, tile_bytes, smem;
 };
-Layout layout_of(const GroupedShape &s) {
+// `beside`: shared memory of an SM to leave for the CTAs of the kernels around this one.
+Layout layout_of(const GroupedShape &s, uint32_t beside) {
     const uint32_t stage = (s.dim_p + s.vdim_p) / 64u * kBox, heads = std::min(kHeads, s.per());
+    const uint32_t rows = 2u * (heads <= 4u ? 4u : 8u) * (s.dim_p + 8u) * 2u + (s.dim_p + s.vdim_p) * 2u + 1024u;
+    const uint32_t room = kSmemLimit - std::min(beside, kSmemLimit / 2u);
     Layout l{};
-    l.slots = std::min(kMaxSlots, std::max(2u, kTileBudget / stage));
+    l.slots = std::min(kMaxSlots, std::max(2u, (room - std::min(rows, room)) / stage));
     if (l.slots < kRound) l.slots = 2u;
     l.tile_bytes = std::max(l.slots * stage, kWarps * heads * (s.vdim_p + 8u) * 4u);
     l.tile_bytes = (l.tile_bytes + 127u) & ~127u;
-    l.smem = l.tile_bytes + 2u * (heads <= 4u ? 4u : 8u) * (s.dim_p + 8u) * 2u + (s.dim_p + s.vdim_p) * 2u + 1024u;
+    l.smem = l.tile_bytes + rows;
     return l;
 }
 
@@ -455,7 +477,7 @@ Kernel kernel_of(uint32_t value_blocks) {
 }  // namespace
 
 bool grouped_attend_mma_supports(const GroupedShape &s) {
-    return s.dim_p <= kMaxBlocks * 64u && s.vdim_p <= kMaxBlocks * 64u && layout_of(s).smem <= kSmemLimit && encode_tiled() != nullptr;
+    return s.dim_p <= kMaxBlocks * 64u && s.vdim_p <= kMaxBlocks * 64u && layout_of(s, kSmemLimit).smem <= kSmemLimit && encode_tiled() != nullptr;
 }
 
 stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t stream) {
@@ -479,7 +501,7 @@ stark_b200_status grouped_attend_mma_launch(const GroupedArgs &a, cudaStream_t s
                CUDA_SUCCESS;
     };
     if (!make(&k_map, a.keys, s.dim_p) || !make(&v_map, a.values, s.vdim_p)) return STARK_B200_DEVICE_FAILURE;
-    const Layout l = layout_of(s);
+    const Layout l = layout_of(s, a.beside_smem);
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(a.splits * a.cluster, s.groups * ((s.per() + kHeads - 1u) / kHeads));
     cfg.blockDim = dim3(kThreads);

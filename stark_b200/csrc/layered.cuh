@@ -231,6 +231,7 @@ struct GroupedArgs {
     uint16_t *queries_b16;     // ... or unscaled, rounded
     float *partials;           // grouped_attend_mma: [heads, splits, vdim_p + 4] where splits > 1
     uint32_t splits, cluster;  // partials per head; spans of the cache merged into each (1, 2, 4 or 8)
+    uint32_t beside_smem;      // grouped_attend_mma: shared memory of an SM it leaves for the CTAs of the kernels around it
     float *out;                // grouped_attend_mma: [heads * vdim_p] where splits == 1
     uint32_t *error_word;
     bool pdl;

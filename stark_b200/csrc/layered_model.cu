@@ -204,14 +204,15 @@ LatentArgs latent_args(Model *m, const Layer &layer) {
     return a;
 }
 
-// Spans of the grouped decode attention: a cluster of CTAs per key / value head (and 8 of its query heads), as large as
-// the SMs allow and the context has pages; more clusters, merged by a launch of their own, where heads are few and the
-// context is long.
+// Spans of the grouped decode attention: a cluster of up to eight CTAs (8 query heads of a key / value head each), which
+// merges them; several clusters, merged by a launch of their own, where heads are few and the context is long.
 void divide_grouped(const Model *m, GroupedArgs &a) {
     const uint32_t tiles = a.s.groups * ((a.s.per() + kGroupedHeadTile - 1u) / kGroupedHeadTile), pages = m->num_blocks;
-    const uint32_t most = tunables().grouped_cluster ? tunables().grouped_cluster : 8u;
+    // the contraction before it: two CTAs an SM, an input row and some words each
+    a.beside_smem = 2u * ((m->layered->width_p + 255u) / 256u * 1024u + 2048u);
     a.cluster = 1;
-    while (a.cluster * 2u <= most && a.cluster * 2u * tiles <= 148u && a.cluster < pages) a.cluster *= 2u;
+    while (a.cluster < 8u && a.cluster * 2u * tiles <= 148u && a.cluster < pages) a.cluster *= 2u;
+    if (tunables().grouped_cluster) a.cluster = tunables().grouped_cluster;
     a.splits = std::max(1u, std::min({148u / (a.cluster * tiles), pages / (a.cluster * 16u), kMaxSplits}));
     if (tunables().grouped_splits) a.splits = tunables().grouped_splits;
 }
