@@ -1,7 +1,6 @@
 // Grouped-query attention with short convolutions: what happens to projected rows before they attend, for any number of
 // rows, and the state the convolutions keep.  A unit is one head of the queries, keys or values; a warp owns one unit of a
-// few rows, two neighbouring channels a lane and 64 channels at a time.  Everything is f32 between the projected values and
-// what is stored.
+// few rows.  Everything is f32 between the projected values and what is stored.
 #include "layered.cuh"
 #include "layered_math.cuh"
 
@@ -9,9 +8,9 @@ namespace sb {
 
 namespace {
 
-constexpr uint32_t kThreads = 256, kWarpRows = 8, kCtaRows = kThreads / 32u * kWarpRows;
+constexpr uint32_t kThreads = 256, kWarpRows = 4, kCtaRows = kThreads / 32u * kWarpRows;
 constexpr uint32_t kMaxBlocks = 8;  // heads up to 512 wide
-constexpr uint32_t kWindowTaps = 4, kWindowBlocks = 2;
+constexpr uint32_t kWindowTaps = 4, kRun = 8;  // grouped_window_kernel: taps; rows in a run
 
 // What a unit's channels are called in the projected row, and where its row goes.
 struct Unit {
@@ -81,107 +80,108 @@ __device__ inline void keep_row(const GroupedArgs &a, const Unit &t, uint32_t po
     }
 }
 
-// Sums over the warp's lanes of eight values each, by halves: afterwards lane l holds the sum of value (l >> 2) with its
-// three bits in reverse, which is row_of_lane(l).
-__device__ inline uint32_t row_of_lane(uint32_t lane) { return ((lane >> 4) & 1u) | ((lane >> 2) & 2u) | (lane & 4u); }
-__device__ inline uint32_t lane_of_row(uint32_t row) { return ((row & 1u) << 4) | ((row & 2u) << 2) | (row & 4u); }
-__device__ inline float sum_eight(const float (&v)[8], uint32_t lane) {
-    float a[4], b[2], c;
+__device__ inline void unpack8(const uint4 &r, float (&v)[8]) {
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll
-    for (uint32_t i = 0; i < 4u; ++i) {
-        const bool up = (lane & 16u) != 0u;
-        const float send = up ? v[2u * i] : v[2u * i + 1u], keep = up ? v[2u * i + 1u] : v[2u * i];
-        a[i] = keep + __shfl_xor_sync(0xffffffffu, send, 16);
-    }
-#pragma unroll
-    for (uint32_t i = 0; i < 2u; ++i) {
-        const bool up = (lane & 8u) != 0u;
-        const float send = up ? a[2u * i] : a[2u * i + 1u], keep = up ? a[2u * i + 1u] : a[2u * i];
-        b[i] = keep + __shfl_xor_sync(0xffffffffu, send, 8);
-    }
-    const bool up = (lane & 4u) != 0u;
-    c = (up ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, up ? b[0] : b[1], 4);
-    c += __shfl_xor_sync(0xffffffffu, c, 2);
-    return c + __shfl_xor_sync(0xffffffffu, c, 1);
+    for (int i = 0; i < 4; ++i) v[2 * i] = __uint_as_float(w[i] << 16), v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
 }
 
-// Up to kWindowTaps taps and heads of kWindowBlocks blocks: a warp holds the rows its convolution reaches in registers, all
-// of them asked for at once, so that a projected value is read once (and the few rows in front of a warp's first one again);
-// the norms of its eight rows are reduced together and each row's factor is worked out by the lanes that end up with it.
-// U: type of the projected rows; E: type of the cache and of the convolutions' state.  blockIdx: (rows, unit)
-template <typename U, typename E>
+// Runs of kRun rows of a bf16 pass, up to kWindowTaps taps and heads up to 256 wide: what prompts go through.  A lane has
+// eight neighbouring channels, as many lanes as the unit needs walk one run (a warp two or four runs of narrow units), the
+// rows the convolution reaches stay in registers and every projected value is read once.  blockIdx: (rows, unit)
 __global__ void __launch_bounds__(kThreads) grouped_window_kernel(const GroupedArgs a) {
     pdl_launch_dependents();
     pdl_wait();
-    using RawU = RawPair<U>;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, taps = a.conv.taps, width = a.s.width();
-    const Unit t = unit_of(a.s, blockIdx.y, lane);
-    const uint32_t row0 = blockIdx.x * kCtaRows + warp * kWarpRows;
-    if (row0 >= a.m) return;
-    const uint32_t first_pos = a.state ? a.state->position : a.first_pos, rows = min(kWarpRows, a.m - row0);
-    const U *u = reinterpret_cast<const U *>(a.u) + (size_t)row0 * a.ld_u + t.col;
-    constexpr uint32_t kBack = kWindowTaps - 1u;
-    typename RawU::type x[kBack + kWarpRows][kWindowBlocks];
-    float2 f[kWindowTaps][kWindowBlocks];  // f[j] weighs the row kBack - j back
+    const GroupedShape &s = a.s;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, taps = a.conv.taps, width = s.width();
+    Unit t = unit_of(s, blockIdx.y, 0u);
+    const uint32_t lanes = t.padded / 8u, runs = 32u / lanes, sub = lane / lanes, channel = lane % lanes * 8u;
+    const bool idle = sub >= runs;  // 192 wide: eight lanes over
+    const uint32_t warp_row0 = (blockIdx.x * (kThreads / 32u) + warp) * runs * kRun, row0 = warp_row0 + sub * kRun;
+    if (warp_row0 >= a.m) return;
+    t.col += channel;
+    const uint16_t *u = reinterpret_cast<const uint16_t *>(a.u) + t.col;
+    uint16_t *recent = reinterpret_cast<uint16_t *>(a.conv.recent) + t.col, *tails = reinterpret_cast<uint16_t *>(a.conv.tails) + t.col;
+    const uint32_t rows = idle || row0 >= a.m ? 0u : min(kRun, a.m - row0);
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    uint4 raw[kRun], front[kWindowTaps - 1u];
 #pragma unroll
-    for (uint32_t i = 0; i < kWarpRows; ++i)
+    for (uint32_t r = 0; r < kRun; ++r)
+        raw[r] = r < rows ? *reinterpret_cast<const uint4 *>(u + (size_t)(row0 + r) * a.ld_u) : zero;
+    // the rows in front of the run: of this pass, or recent ones, or zeros before the sequence's start
 #pragma unroll
-        for (uint32_t b = 0; b < kWindowBlocks; ++b)
-            x[kBack + i][b] = i < rows && b < t.blocks
-                                  ? *reinterpret_cast<const typename RawU::type *>(u + (size_t)i * a.ld_u + b * 64u)
-                                  : RawU::zero();
-    // the rows in front: of this pass, or recent ones, or zeros before the sequence's start
-    float2 front[kBack][kWindowBlocks];
-#pragma unroll
-    for (uint32_t i = 0; i < kBack; ++i) {
-        const uint32_t back = kBack - i;
-        const bool in = back < taps && back <= first_pos + row0;
-        const E *recent = reinterpret_cast<const E *>(a.conv.recent) + (size_t)((first_pos + row0 - (in ? back : 0u)) % a.conv.recent_rows()) * width + t.col;
-#pragma unroll
-        for (uint32_t b = 0; b < kWindowBlocks; ++b) {
-            front[i][b] = make_float2(0.0f, 0.0f);
-            if (in && b < t.blocks) front[i][b] = back <= row0 ? load_pair(u - (size_t)back * a.ld_u + b * 64u) : load_pair(recent + b * 64u);
-        }
+    for (uint32_t i = 0; i < kWindowTaps - 1u; ++i) {
+        const uint32_t back = kWindowTaps - 1u - i;
+        front[i] = zero;
+        if (rows && back < taps && back <= a.first_pos + row0)
+            front[i] = *reinterpret_cast<const uint4 *>(
+                back <= row0 ? u + (size_t)(row0 - back) * a.ld_u
+                             : recent + (size_t)((a.first_pos + row0 - back) % a.conv.recent_rows()) * width);
     }
+    float f[kWindowTaps][8];  // f[j] weighs the row kWindowTaps - 1 - j back
 #pragma unroll
-    for (uint32_t j = 0; j < kWindowTaps; ++j)
+    for (uint32_t j = 0; j < kWindowTaps; ++j) {
+        const bool in = !idle && j + taps >= kWindowTaps;
+        const float4 *w = reinterpret_cast<const float4 *>(a.conv.w + (size_t)(in ? j + taps - kWindowTaps : 0u) * width + t.col);
+        const float4 lo = in ? w[0] : make_float4(0.f, 0.f, 0.f, 0.f), hi = in ? w[1] : make_float4(0.f, 0.f, 0.f, 0.f);
+        f[j][0] = lo.x, f[j][1] = lo.y, f[j][2] = lo.z, f[j][3] = lo.w, f[j][4] = hi.x, f[j][5] = hi.y, f[j][6] = hi.z, f[j][7] = hi.w;
+    }
+    // lane i: the page of the warp's row i, and its factor apart from the norm
+    const uint32_t my_row = warp_row0 + lane, my_pos = a.first_pos + my_row;
+    const bool mine = lane < runs * kRun && my_row < a.m;
+    const uint32_t my_page = mine ? (uint32_t)a.block_table[my_pos / kPageTokens] : 0u;
+    const float my_factor = t.is_q ? query_temperature(my_pos, a.temp_coef, a.temp_every) * (a.queries_b16 ? 1.0f : a.scale * kLog2e) : 1.0f;
+    const float inverse_dim = 1.0f / (float)s.dim;
+    float x[kWindowTaps][8];  // the window, by row modulo kWindowTaps
 #pragma unroll
-        for (uint32_t b = 0; b < kWindowBlocks; ++b)
-            f[j][b] = j + taps >= kWindowTaps && b < t.blocks ? load_pair(a.conv.w + (size_t)(j + taps - kWindowTaps) * width + t.col + b * 64u)
-                                                              : make_float2(0.0f, 0.0f);
-    // lane r < kWarpRows: the page of row r
-    const uint32_t my_page = lane < rows ? (uint32_t)a.block_table[(first_pos + row0 + lane) / kPageTokens] : 0u;
-    float2 v[kWarpRows][kWindowBlocks];
-    float squares[kWarpRows];
+    for (uint32_t i = 0; i < kWindowTaps - 1u; ++i) unpack8(front[i], x[i]);
 #pragma unroll
-    for (uint32_t r = 0; r < kWarpRows; ++r) {
-        squares[r] = 0.0f;
+    for (uint32_t r = 0; r < kRun; ++r) {
+        const uint32_t row = row0 + r, pos = a.first_pos + row;
+        unpack8(raw[r], x[(r + kWindowTaps - 1u) % kWindowTaps]);
+        float v[8], sum = 0.0f;
 #pragma unroll
-        for (uint32_t b = 0; b < kWindowBlocks; ++b) {
-            float2 acc = make_float2(0.0f, 0.0f);
+        for (uint32_t e = 0; e < 8u; ++e) {
+            v[e] = 0.0f;
 #pragma unroll
-            for (uint32_t j = 0; j < kWindowTaps; ++j) {
-                const float2 at = r + j < kBack ? front[r + j][b] : RawU::value(x[r + j][b]);
-                acc.x = fmaf(f[j][b].x, at.x, acc.x), acc.y = fmaf(f[j][b].y, at.y, acc.y);
+            for (uint32_t j = 0; j < kWindowTaps; ++j) v[e] = fmaf(f[j][e], x[(r + j) % kWindowTaps][e], v[e]);
+            sum = fmaf(v[e], v[e], sum);
+        }
+        const uint32_t page = __shfl_sync(0xffffffffu, my_page, sub * kRun + r);
+        if (t.is_q || t.is_k) {
+            // over the run's lanes; all of the warp where they are no power of two (the idle ones hold zeros)
+            for (uint32_t o = lanes == 24u ? 16u : lanes / 2u; o > 0u; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            const float factor = __shfl_sync(0xffffffffu, my_factor, sub * kRun + r) * rsqrtf(sum * inverse_dim + a.eps);
+#pragma unroll
+            for (uint32_t e = 0; e < 8u; ++e) v[e] *= factor;
+        }
+        if (r >= rows) continue;
+        uint16_t *dst;
+        if (t.is_q) {
+            dst = a.queries_b16 + ((size_t)row * s.heads + t.head) * s.dim_p + channel;
+        } else {
+            dst = reinterpret_cast<uint16_t *>(t.is_k ? a.keys : a.values) +
+                  (((size_t)page * s.groups + t.head) * kPageTokens + pos % kPageTokens) * t.padded + channel;
+            if (!t.is_k && a.mix != kMixNone) {
+                float *first = a.first_values + ((size_t)row * s.groups + t.head) * s.vdim;
+#pragma unroll
+                for (uint32_t e = 0; e < 8u; e += 2u) {
+                    if (a.mix == kMixFirst) {
+                        keep_first_values(first, channel + e, s.vdim, make_float2(v[e], v[e + 1u]));
+                    } else {
+                        const float2 o = mix_values(first, channel + e, s.vdim, make_float2(v[e], v[e + 1u]), a.share);
+                        v[e] = o.x, v[e + 1u] = o.y;
+                    }
+                }
             }
-            v[r][b] = acc;
-            squares[r] += acc.x * acc.x + acc.y * acc.y;
         }
-    }
-    float my_factor = 1.0f;
-    if (t.is_q || t.is_k) my_factor = row_factor(a, t, sum_eight(squares, lane), first_pos + row0 + row_of_lane(lane));
-#pragma unroll
-    for (uint32_t r = 0; r < kWarpRows; ++r) {
-        if (r >= rows) break;
-        const uint32_t pos = first_pos + row0 + r, page = __shfl_sync(0xffffffffu, my_page, r);
-        const float factor = __shfl_sync(0xffffffffu, my_factor, lane_of_row(r));
-        store_row<E, kWindowBlocks>(a, t, row0 + r, pos, page, lane, v[r], factor);
-        if (taps > 1u && (a.m <= kConvSpare || pos % kPageTokens + taps > kPageTokens)) {
-            float2 raw[kWindowBlocks];
-#pragma unroll
-            for (uint32_t b = 0; b < kWindowBlocks; ++b) raw[b] = RawU::value(x[r + kBack][b]);
-            keep_row<E, kWindowBlocks>(a, t, pos, page, raw);
-        }
+        *reinterpret_cast<uint4 *>(dst) = make_uint4(f32x2_to_bf16x2(v[0], v[1]), f32x2_to_bf16x2(v[2], v[3]),
+                                                     f32x2_to_bf16x2(v[4], v[5]), f32x2_to_bf16x2(v[6], v[7]));
+        // the projected row itself, where a later position's convolution will look for it
+        const uint32_t in_page = pos % kPageTokens;
+        if (taps > 1u && a.m <= kConvSpare) *reinterpret_cast<uint4 *>(recent + (size_t)(pos % a.conv.recent_rows()) * width) = raw[r];
+        if (taps > 1u && in_page + taps > kPageTokens)
+            *reinterpret_cast<uint4 *>(tails + ((size_t)page * (taps - 1u) + in_page + taps - 1u - kPageTokens) * width) = raw[r];
     }
 }
 
@@ -252,13 +252,18 @@ stark_b200_status grouped_rows_launch(const GroupedArgs &a, cudaStream_t stream)
         (a.state && a.m != 1u) || !a.temp_every || (a.mix != kMixNone && !a.first_values) ||
         (a.queries == nullptr) == (a.queries_b16 == nullptr) || (a.u_b16 && a.cache_f32) || a.ld_u < a.s.width() || a.ld_u % 2u)
         return STARK_B200_INVALID_ARGUMENT;
-    const bool window = a.conv.taps <= kWindowTaps && std::max(a.s.dim_p, a.s.vdim_p) <= kWindowBlocks * 64u;
-    auto kernel = window ? (a.u_b16 ? grouped_window_kernel<uint16_t, uint16_t>
-                                    : (a.cache_f32 ? grouped_window_kernel<float, float> : grouped_window_kernel<float, uint16_t>))
-                         : (a.u_b16 ? grouped_rows_kernel<uint16_t, uint16_t>
-                                    : (a.cache_f32 ? grouped_rows_kernel<float, float> : grouped_rows_kernel<float, uint16_t>));
-    const dim3 grid((a.m + kCtaRows - 1u) / kCtaRows, a.s.heads + 2u * a.s.groups);
-    if (stark_b200_status st = launch_chained(kernel, grid, dim3(kThreads), 0, a.pdl, stream, a)) return st;
+    const uint32_t units = a.s.heads + 2u * a.s.groups, widest = std::max(a.s.dim_p, a.s.vdim_p);
+    if (a.u_b16 && a.queries_b16 && a.conv.taps <= kWindowTaps && widest <= 256u && a.ld_u % 8u == 0) {
+        const uint32_t cta_rows = kThreads / 32u * (256u / widest) * kRun;  // of the units with the fewest runs to a warp
+        if (stark_b200_status st = launch_chained(grouped_window_kernel, dim3((a.m + cta_rows - 1u) / cta_rows, units), dim3(kThreads), 0,
+                                                  a.pdl, stream, a))
+            return st;
+    } else {
+        auto kernel = a.u_b16 ? grouped_rows_kernel<uint16_t, uint16_t>
+                              : (a.cache_f32 ? grouped_rows_kernel<float, float> : grouped_rows_kernel<float, uint16_t>);
+        if (stark_b200_status st = launch_chained(kernel, dim3((a.m + kCtaRows - 1u) / kCtaRows, units), dim3(kThreads), 0, a.pdl, stream, a))
+            return st;
+    }
     if (a.m <= kConvSpare || a.conv.taps == 1u) return STARK_B200_OK;
     auto keep = a.u_b16 ? short_conv_keep_kernel<uint16_t, uint16_t>
                         : (a.cache_f32 ? short_conv_keep_kernel<float, float> : short_conv_keep_kernel<float, uint16_t>);

@@ -50,21 +50,6 @@ __device__ inline float2 load_pair(const uint16_t *p) {
     const uint32_t w = *reinterpret_cast<const uint32_t *>(p);
     return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u));
 }
-// The same as it lies in memory, and what it holds.
-template <typename T>
-struct RawPair;
-template <>
-struct RawPair<float> {
-    using type = float2;
-    static __device__ inline float2 value(float2 r) { return r; }
-    static __device__ inline float2 zero() { return make_float2(0.0f, 0.0f); }
-};
-template <>
-struct RawPair<uint16_t> {
-    using type = uint32_t;
-    static __device__ inline float2 value(uint32_t r) { return make_float2(__uint_as_float(r << 16), __uint_as_float(r & 0xffff0000u)); }
-    static __device__ inline uint32_t zero() { return 0u; }
-};
 __device__ inline void store_pair(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
 __device__ inline void store_pair(uint16_t *p, float2 v) { *reinterpret_cast<uint32_t *>(p) = f32x2_to_bf16x2(v.x, v.y); }
 
