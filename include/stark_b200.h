@@ -675,7 +675,7 @@ typedef struct stark_b200_layer_desc {
     double rot_base;
     double rot_factor, rot_original, rot_fast, rot_slow; /* STARK_B200_ROT_YARN */
     /* STARK_B200_MIXER_GROUPED */
-    uint32_t kv_heads;     /* key / value heads; query head h uses h / (heads / kv_heads) */
+    uint32_t kv_heads;     /* key / value heads, each shared by heads / kv_heads neighbouring query heads */
     uint32_t conv_taps;    /* taps of the causal convolution over time on queries, keys and values (0: none) */
     uint32_t q_temp_every; /* queries times 1 + q_temp_coef * ln((position + 1) / q_temp_every + 1), whole division */
     float q_temp_coef;

@@ -38,8 +38,8 @@ def mixed_values(v, first, share):
 
 
 def grouped_attention(q, keys, values, first_pos, scale):
-    """q [rows, heads, dim] at positions first_pos.. over keys [n, groups, dim] and values [n, groups, vdim]; query head
-    h uses key/value head h // (heads / groups).  Softmax over every key up to the row's own position."""
+    """q [rows, heads, dim] at positions first_pos.. over keys [n, groups, dim] and values [n, groups, vdim]; heads /
+    groups neighbouring query heads share a group.  A row attends to the keys up to and including its own position."""
     per = q.shape[1] // keys.shape[1]
     out = np.zeros((q.shape[0], q.shape[1], values.shape[2]), q.dtype)
     for h in range(q.shape[1]):

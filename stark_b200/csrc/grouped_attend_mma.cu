@@ -79,7 +79,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
     extern __shared__ uint8_t grouped_smem[];
     __shared__ uint64_t full[kMaxSlots];
     __shared__ float warp_m[kWarps][kHeads], warp_l[kWarps][kHeads], run_m[kHeads], run_l[kHeads];
-    __shared__ uint32_t abort_flag;
+    __shared__ volatile uint32_t abort_flag;
     const GroupedShape &s = a.s;
     const uint32_t kb = s.dim_p / 64u, stage_bytes = (kb + VB) * kBox, q_pitch = s.dim_p + 8u;
     uint8_t *tile = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(grouped_smem) + 1023u) & ~(uintptr_t)1023u);
@@ -140,7 +140,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
 #pragma unroll
             for (uint32_t i = 0; i < 4u; ++i) {
                 const uint32_t j = j0 + i, back = taps - 1u - j;
-                const bool in = j + 1u < taps && back <= pos;  // zeros before the sequence's start
+                const bool in = j + 1u < taps && back <= pos;  // nothing precedes the first token
 #pragma unroll
                 for (uint32_t b = 0; b < kMaxBlocks; ++b) {
                     x[b][i] = f[b][i] = make_float2(0.0f, 0.0f);
@@ -254,7 +254,7 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                      : "memory");
     };
     const uint32_t round = min(kRound, slots);
-    uint32_t slot0 = 0, phase0 = 0;  // of page i0
+    uint32_t slot0 = 0, phase0 = 0, fetched = min(n, slots);  // slot and phase of page i0; pages asked for (thread 0)
     for (uint32_t i0 = 0; i0 < n; i0 += round) {
         const uint32_t i = i0 + (warp >> 1);
         const bool wraps = slot0 + (warp >> 1) >= slots;
@@ -353,12 +353,17 @@ grouped_attend_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __gri
                 uint32_t into = slot0;
 #pragma unroll
                 for (uint32_t j = 0; j < kRound; ++j) {
-                    if (coming[j] != UINT32_MAX) fetch(into, coming[j]);
+                    if (coming[j] != UINT32_MAX && !abort_flag) fetch(into, coming[j]), ++fetched;
                     if (++into == slots) into = 0u;
                 }
             }
         }
         if ((slot0 += round) >= slots) slot0 -= slots, phase0 ^= 1u;
+    }
+
+    if (tid == 0 && abort_flag) {  // what is still on its way must not land in the words below
+        const uint32_t go_on = 0u;
+        for (uint32_t i = fetched - min(fetched, slots); i < fetched; ++i) mbar_wait_bounded(&full[i % slots], (i / slots) & 1u, &go_on);
     }
 
     // ---- merge of the warps: statistics, then weighted values, rows pitch apart

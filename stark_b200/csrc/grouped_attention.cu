@@ -108,7 +108,7 @@ __global__ void __launch_bounds__(kThreads) grouped_window_kernel(const GroupedA
 #pragma unroll
     for (uint32_t r = 0; r < kRun; ++r)
         raw[r] = r < rows ? *reinterpret_cast<const uint4 *>(u + (size_t)(row0 + r) * a.ld_u) : zero;
-    // the rows in front of the run: of this pass, or recent ones, or zeros before the sequence's start
+    // the rows in front of the run: of this pass, or recent ones, or nothing (zeros) in front of the first token
 #pragma unroll
     for (uint32_t i = 0; i < kWindowTaps - 1u; ++i) {
         const uint32_t back = kWindowTaps - 1u - i;
@@ -206,7 +206,7 @@ __global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArg
             float2 acc = make_float2(0.0f, 0.0f);
             for (uint32_t j = 0; j < taps; ++j) {
                 const uint32_t back = taps - 1u - j;
-                if (back > pos) continue;  // zeros before the sequence's start
+                if (back > pos) continue;  // nothing precedes the first token
                 x[b] = back <= row ? load_pair(u + (size_t)(row - back) * a.ld_u + b * 64u)
                                    : load_pair(recent + (size_t)((pos - back) % a.conv.recent_rows()) * width + b * 64u);
                 const float2 f = load_pair(w + (size_t)j * width + b * 64u);

@@ -214,6 +214,25 @@ def test_spans_of_the_decode_attention(settings):
         m.close()
 
 
+@pytest.mark.parametrize("dim,vdim", [(16, 16), (128, 128), (180, 70), (250, 250)])
+def test_spans_longer_than_the_pages_in_flight(dim, vdim):
+    """One CTA reads the whole cache: pages take the places of pages already read, whatever number of them fits."""
+    root = P.model([P.layer(P.mixer(heads=5, kv_heads=1, dim=dim, vdim=vdim, scale=1.0 / np.sqrt(dim)), ff=None)])
+    w = P.weights(root, seed=25)
+    ids = P.tokens(root, 900)
+    want = P.oracle(root, w).feed(ids)
+    m = P.engine(root, w, 900, "bfloat16")
+    try:
+        m.recapture(grouped_cluster=1, grouped_splits=1)
+        for at in (60, 190, 250, 330, 640, 885):
+            m.reset()
+            m.prefill(ids[:at])
+            close(feed(m, ids[at:at + 12], [1] * 12), want[at:at + 12], "bfloat16")
+    finally:
+        m.recapture(grouped_cluster=0, grouped_splits=0)
+        m.close()
+
+
 def needle_model(scale=0.75, coef=0.3, every=16):
     """Every query asks for one direction, which only the needle token's key has: entry 0 of the embedding marks the needle,
     entry 1 is in every other token."""
