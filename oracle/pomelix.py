@@ -19,7 +19,7 @@ def norm(x, w, eps):
 
 def short_convolution(u, w, past):
     """Causal convolution over time per channel: row t is sum_j w[:, j] u[t - taps + 1 + j].  ``past`` holds the
-    taps - 1 rows before ``u`` (zeros before a sequence's start)."""
+    taps - 1 rows that came before ``u``, zeros where there were none."""
     taps = w.shape[1]
     rows = np.concatenate([past, u])
     out = np.zeros_like(u)
